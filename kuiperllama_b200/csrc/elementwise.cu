@@ -67,7 +67,7 @@ __global__ void swiglu_kernel(const float* __restrict__ x1, const float* __restr
   if (i < n) out[i] = swiglu_ref(x1[i], x3[i]);
 }
 
-// rope_kernel.cu:38-49 / 84-95 / 124-135: same expression, same libdevice calls, and -- like the
+// rope_kernel.cu:38-49 / 84-95 / 124-135: same expression, same math calls, and -- like the
 // reference -- a LITERAL base per flavour so the compiler sees the same powf call site.
 template <int kFlavour>
 __global__ void sincos_kernel(int head_size, int seq_len, float* sin_cache, float* cos_cache) {

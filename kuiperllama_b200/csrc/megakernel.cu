@@ -545,7 +545,7 @@ __device__ __forceinline__ void accum_w8_dp4a(const uint32_t (&w)[NR], const uin
 // The integer dot-product unit runs at a quarter of the FP32 rate on sm_100 (measured: the dp4a rows above are
 // bound by it, 12 IDP.4A per 16 weights), so where a ring stage holds several rows that share the input
 // vector -- every matrix with 4096-byte rows -- the 64-element groups go through mma.sync m16n8k32 (s8 x s8 ->
-// s32, SASS IMMA.16832.S8.S8) instead:
+// s32) instead:
 //     A (16 x 32, row major)  rows 0..7 = the (up to 8) weight rows of the stage, rows 8..15 mirror them
 //     B (32 x 8, column major) columns 0, 1, 2 = the three digit planes of x, columns 3..7 = 0
 //     D (16 x 8, s32)          D[r][k] = sum_i w[r][i] * l_k[i]  -- the exact integers D_k of the dp4a form

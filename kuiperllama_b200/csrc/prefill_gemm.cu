@@ -11,10 +11,10 @@
 //
 // Structure (one CTA per 128 weight rows x one block of BN tokens, 6 warps):
 //   warp 0   TMA producer: cp.async.bulk.tensor 2-D tiles of w [128 x 32 fp32] and x [BN x 32 fp32],
-//            128-byte swizzle, into a 4-stage shared-memory ring (SASS: UTMALDG)
+//            128-byte swizzle, into a 4-stage shared-memory ring
 //   warp 1   MMA issuer: one thread, 4 x tcgen05.mma.kind::tf32 (M 128, N BN, K 8) per stage, D in
-//            TMEM; tcgen05.commit frees the stage / signals the epilogue (SASS: UTCHMMA / UTCBAR)
-//   warps 2-5 epilogue: tcgen05.ld 32 lanes x 32 columns per warp (SASS: LDTM), transposed store
+//            TMEM; tcgen05.commit frees the stage / signals the epilogue
+//   warps 2-5 epilogue: tcgen05.ld 32 lanes x 32 columns per warp, transposed store
 #include <cuda.h>
 #include <cuda_runtime.h>
 
