@@ -33,7 +33,7 @@ extern "C" {
 #define KLLM_SEQ_MIXER_SSD 6       /* state-space duality: short convolution, one input-dependent decay per head, a matrix state per head */
 #define KLLM_SEQ_FF_NONE 0
 #define KLLM_SEQ_FF_MOE 1   /* routed experts (softmax or sigmoid router), optional gated shared expert */
-#define KLLM_SEQ_FF_DENSE 2 /* down(act(up h)) */
+#define KLLM_SEQ_FF_DENSE 2 /* down(act(up h)), or down(act(gate h) * up h) */
 
 #define KLLM_SEQ_NORM_LAYER 0 /* (v - mean) / sqrt(var + eps) * w + b */
 #define KLLM_SEQ_NORM_RMS 1   /* v / sqrt(mean(v^2) + eps) * w */
@@ -48,6 +48,13 @@ extern "C" {
 #define KLLM_SEQ_QKNORM_NONE 0
 #define KLLM_SEQ_QKNORM_WEIGHTED 1 /* RMS norm over dim with q_norm_w / k_norm_w, before the rotation */
 #define KLLM_SEQ_QKNORM_UNIT 2     /* x / sqrt(mean(x^2) + eps) without weights, after the rotation */
+#define KLLM_SEQ_QKNORM_PROJECTION 3 /* ONE RMS norm over all query rows and one over all key rows, before they are split into
+                                        heads (q_norm_w [heads*dim], k_norm_w [kv_heads*dim]), before the rotation */
+
+/* values blended with those of an earlier layer (kllm_seq_attention.v_blend) */
+#define KLLM_SEQ_VBLEND_NONE 0
+#define KLLM_SEQ_VBLEND_SOURCE 1 /* this layer's values are the ones later layers blend with */
+#define KLLM_SEQ_VBLEND_MIX 2    /* v <- (1 - v_lambda) v + v_lambda * the source's values of the same token */
 
 /* activations of a feed-forward's inner layer */
 #define KLLM_SEQ_ACT_SWIGLU 0 /* silu(gate h) * (up h): the weights hold gate rows, then up rows */
@@ -55,6 +62,7 @@ extern "C" {
 #define KLLM_SEQ_ACT_XIELU 2  /* z > 0: a z^2 + z / 2;  z <= 0: b (exp(z) - 1 - z) + z / 2 */
 #define KLLM_SEQ_ACT_RELU_GATE 3    /* max(gate h, 0) * (up h): gate rows, then up rows */
 #define KLLM_SEQ_ACT_CLAMP_SWIGLU 4 /* g = min(gate h, limit), u = clamp(up h, -limit, limit): g * sigmoid(alpha g) * (u + 1) */
+#define KLLM_SEQ_ACT_GELU_GATE 5    /* gelu(gate h) * (up h), the tanh form of gelu: gate rows, then up rows */
 
 #define KLLM_SEQ_ROUTER_SOFTMAX 0 /* scores = softmax(z); weights = chosen scores / their sum * scale */
 #define KLLM_SEQ_ROUTER_SIGMOID 1 /* scores = sigmoid(z); chosen by score + correction, inside the best groups; weights = score * scale */
@@ -78,8 +86,8 @@ typedef struct kllm_seq_attention {
   int32_t gate;                       /* KLLM_SEQ_GATE_*: sigmoid output gate; its rows close w_in */
   const void* w_in;  /* [heads*dim + kv_heads*dim + kv_heads*vdim (+ gate rows), width]: q | k | v (| gate) rows, compute type
                         (differential: 2*heads*dim query rows and 2*kv_heads*dim key rows) */
-  const float* q_norm_w; /* [dim] */
-  const float* k_norm_w; /* [dim] */
+  const float* q_norm_w; /* [dim]; KLLM_SEQ_QKNORM_PROJECTION: [heads*dim] */
+  const float* k_norm_w; /* [dim]; KLLM_SEQ_QKNORM_PROJECTION: [kv_heads*dim] */
   const void* w_out;     /* [width, heads*vdim], compute type */
   int32_t window;        /* position i sees j <= i with i - j < window or j < keep_first; 0: every earlier position */
   int32_t keep_first;    /* the first keep_first positions stay visible behind the window (at their true positions) */
@@ -103,26 +111,38 @@ typedef struct kllm_seq_attention {
    * o / sqrt(mean(o^2) + eps) * diff_out_scale over its vdim values. */
   int32_t differential;
   float diff_lambda, diff_out_scale;
+  const float* out_bias; /* [width] fp32 added to the output projection, or NULL */
+  /* KLLM_SEQ_VBLEND_*: the source's values are taken as projected (bias included), in fp32; what a MIX layer caches is the
+   * blend.  The latest source ahead of a MIX layer in the run order must have the same kv_heads * vdim. */
+  int32_t v_blend;
+  float v_lambda;
 } kllm_seq_attention;
 
-/* Attention through a latent.  Queries: cq = RMSnorm(W_dq h), q = W_uq cq, per head [dim plain | rot_dim rotated].
+/* Attention through a latent.  Queries: cq = RMSnorm(W_dq h), q = W_uq cq -- or q = W_q h itself (q_rank == 0) --, per head
+ * [dim plain | rot_dim rotated].
  * Keys / values: W_dkv h = [kv_rank | rot_dim]; c = RMSnorm(first part) is the latent, the second part, rotated, is a key
  * part shared by all heads.  Per head k = [W_uk c | rotated part], v = W_uv c.  Only c and the rotated part are cached:
  * the engine scores with W_uk^T q against c and applies W_uv after the weighted sum of latents. */
 typedef struct kllm_seq_latent {
-  int32_t heads, dim, rot_dim, vdim, q_rank, kv_rank;
+  int32_t heads, dim, rot_dim, vdim;
+  int32_t q_rank;     /* 0: the queries are projected directly */
+  int32_t kv_rank;
   float scale;        /* score = (q . k) * scale */
   int32_t window;     /* position i sees j with 0 <= i - j < window; 0: all earlier positions */
-  int32_t rope_dims;  /* rotary positions on the first rope_dims coordinates of the rotated part, coordinate i paired with i + rope_dims / 2 */
+  int32_t rope_dims;  /* rotary positions on the first rope_dims coordinates of the rotated part (rope_pairing) */
   float rope_base;    /* angle = position * rope_base^(-2 i / rope_dims) */
-  const void* w_in;   /* [q_rank + kv_rank + rot_dim + heads, width]: W_dq | W_dkv | gate rows, compute type */
-  const float* q_norm_w;  /* [q_rank] */
+  const void* w_in;   /* [q_rank + kv_rank + rot_dim (+ heads), width]: W_dq | W_dkv (| gate rows), compute type;
+                         q_rank == 0: heads * (dim + rot_dim) rows of W_q take the place of W_dq */
+  const float* q_norm_w;  /* [q_rank]; not read when q_rank == 0 */
   const float* kv_norm_w; /* [kv_rank] */
-  const void* w_uq;   /* [heads * (dim + rot_dim), q_rank] */
+  const void* w_uq;   /* [heads * (dim + rot_dim), q_rank]; not read when q_rank == 0 */
   const void* w_uk;   /* [heads * dim, kv_rank] */
-  const void* w_uv;   /* [heads * vdim, kv_rank] */
+  const void* w_uv;   /* [heads * vdim, kv_rank]; when it follows w_uk in memory, a prompt expands its latents in one product */
   const float* sink;  /* [heads]: exp(sink) joins the softmax denominator (no key, no value), or NULL */
   const void* w_out;  /* [width, heads * vdim] */
+  int32_t gate;           /* KLLM_SEQ_GATE_NONE / KLLM_SEQ_GATE_HEAD: one sigmoid gate per (token, head) */
+  int32_t rope_pairing;   /* KLLM_SEQ_ROPE_* */
+  const float* rope_freq; /* [rope_dims / 2] fp32: angle of pair i = position * rope_freq[i], or NULL: rope_base^(-2 i / rope_dims) */
 } kllm_seq_latent;
 
 /* Linear attention: q, k, v = silu(W h); per head S <- decay * S + k v^T, o = S^T q; the heads together are RMS-normed,
@@ -187,7 +207,7 @@ typedef struct kllm_seq_ssd {
 } kllm_seq_ssd;
 
 typedef struct kllm_seq_dense {
-  int32_t ff, act;    /* inner size; KLLM_SEQ_ACT_* (XIELU, RELU2, or RELU_GATE: then `up` holds ff gate rows followed by ff up rows) */
+  int32_t ff, act;    /* inner size; KLLM_SEQ_ACT_* (XIELU, RELU2, or RELU_GATE / GELU_GATE: then `up` holds ff gate rows followed by ff up rows) */
   float act_a, act_b; /* the two coefficients of KLLM_SEQ_ACT_XIELU */
   const void* up;     /* [ff, width] */
   const void* down;   /* [width, ff] */
@@ -212,6 +232,15 @@ typedef struct kllm_seq_moe {
   float act_limit, act_alpha; /* KLLM_SEQ_ACT_CLAMP_SWIGLU: the routed experts' clamp and the sigmoid's slope */
   float shared_act_limit;     /* the shared expert's clamp (same activation and slope) */
 } kllm_seq_moe;
+
+/* Hyper-connections of one sublayer.  With kllm_seq_desc.streams == S > 0 the residual is S streams x_1 .. x_S (all equal to
+ * the embedding output at the start): the sublayer reads u = sum_s in[s] x_s (through its pre-norm), and its output y joins
+ * every stream at once, x_t <- sum_s mix[s][t] x_s + out[t] y.  After the last layer x is the sum of the streams. */
+typedef struct kllm_seq_hyper {
+  const float* in;  /* [S] */
+  const float* out; /* [S] */
+  const float* mix; /* [S][S], indexed [from][to] */
+} kllm_seq_hyper;
 
 typedef struct kllm_seq_layer {
   int32_t mixer_kind; /* KLLM_SEQ_MIXER_* */
@@ -240,6 +269,7 @@ typedef struct kllm_seq_layer {
   kllm_seq_ssd ssd;
   /* RMS norms over the model width on each mixer's own output, before the mixers' weighted sum (w == NULL: none) */
   kllm_seq_norm mixer_out_norm, mixer2_out_norm;
+  kllm_seq_hyper hyper_mixer, hyper_ff; /* read when the description has streams */
 } kllm_seq_layer;
 
 typedef struct kllm_seq_desc {
@@ -267,6 +297,9 @@ typedef struct kllm_seq_desc {
   float logit_scale;         /* logits = head(...) * logit_scale; 0 means 1 */
   float embed_scale;         /* the embedding rows are multiplied by it (before embed_norm); 0 means 1 */
   float logit_softcap;       /* logits <- cap * tanh(logits / cap), after logit_scale; 0: none */
+  int32_t streams;           /* residual streams joined by hyper-connections (kllm_seq_hyper); 0: one plain residual.  Streams
+                                take no post-norms, token shift, second mixer, feed-forward beside the mixer, routed experts
+                                or additions before a run */
 } kllm_seq_desc;
 
 typedef struct kllm_seq_engine kllm_seq_engine;

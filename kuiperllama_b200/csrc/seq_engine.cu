@@ -141,6 +141,7 @@ struct kllm_seq_engine {
   DevBuf lat_c, lat_kr, lat_kp, lat_vp, lat_q, lat_k, lat_v;  // a prompt step's latents expanded into per-head keys / values
   DevBuf x0, hn, qf, qa, ol;  // embedding output; fp32 normed rows ahead of a token shift; latent / linear attention scratch
   DevBuf y3, y4;              // outputs of a second mixer and of a feed-forward that runs beside the mixer
+  DevBuf xs, vfirst;          // residual streams [T][streams][width]; the values of the step that later layers blend with
   DevBuf rec_a, rec_b, rec_c; // fp32 scratch of the selective scan (filtered rows, low-rank rows) and the delta rule (prepared rows)
   float* logits_pinned = nullptr;
   size_t logits_pinned_cap = 0;
@@ -173,7 +174,7 @@ struct kllm_seq_engine {
   }
   // limits over the layers
   int max_proj = 0, max_q = 0, max_att = 0, max_gates = 0, max_ws_heads = 0, max_top = 0, max_ff = 0, max_sff = 0;
-  int max_qf = 0, max_qa = 0, max_ol = 0, max_rec_a = 0, max_rec_b = 0, max_rec_c = 0;
+  int max_qf = 0, max_qa = 0, max_ol = 0, max_rec_a = 0, max_rec_b = 0, max_rec_c = 0, max_blend = 0;
   bool any_mixer2 = false, any_parallel_ff = false;
   bool any_shift = false, any_run_embed = false;
   std::vector<int32_t> run_embed;
@@ -210,6 +211,11 @@ static int attn_proj_rows(const kllm_seq_attention& A) {
   return s.heads * A.dim + s.kv_heads * A.dim + (A.values_are_keys ? 0 : A.kv_heads * A.vdim) + gate_floats(s);
 }
 
+static LatentShape latent_shape(const kllm_seq_latent& A) {
+  return LatentShape{A.heads, A.dim, A.rot_dim, A.vdim, A.q_rank, A.kv_rank, A.rope_dims, A.rope_base, A.gate, A.rope_pairing, A.rope_freq};
+}
+// an inner layer of gate rows and up rows joined by the activation
+static bool dense_gated(const kllm_seq_dense& f) { return f.act == KLLM_SEQ_ACT_RELU_GATE || f.act == KLLM_SEQ_ACT_GELU_GATE; }
 static bool has_cache(int kind) { return kind == KLLM_SEQ_MIXER_ATTENTION || kind == KLLM_SEQ_MIXER_LATENT; }
 
 static int validate_mixer(const kllm_seq_layer& L, int kind) {
@@ -217,24 +223,28 @@ static int validate_mixer(const kllm_seq_layer& L, int kind) {
     const kllm_seq_attention& a = L.attn;
     if (a.heads <= 0 || a.kv_heads <= 0 || a.heads % a.kv_heads || a.dim <= 0 || a.vdim <= 0 || !a.w_in || !a.w_out)
       return KLLM_E_INVALID;
-    if (a.qk_norm == KLLM_SEQ_QKNORM_WEIGHTED && (!a.q_norm_w || !a.k_norm_w)) return KLLM_E_INVALID;
-    if (a.qk_norm < 0 || a.qk_norm > KLLM_SEQ_QKNORM_UNIT || a.gate < 0 || a.gate > KLLM_SEQ_GATE_ELEMENT) return KLLM_E_INVALID;
+    if ((a.qk_norm == KLLM_SEQ_QKNORM_WEIGHTED || a.qk_norm == KLLM_SEQ_QKNORM_PROJECTION) && (!a.q_norm_w || !a.k_norm_w))
+      return KLLM_E_INVALID;
+    if (a.qk_norm < 0 || a.qk_norm > KLLM_SEQ_QKNORM_PROJECTION || a.gate < 0 || a.gate > KLLM_SEQ_GATE_ELEMENT) return KLLM_E_INVALID;
     // the two maps of a differential head are joined without a sink; the filtered form has one map
     if (a.differential && (a.sink || a.values_are_keys)) return KLLM_E_UNSUPPORTED;
+    if (a.v_blend < 0 || a.v_blend > KLLM_SEQ_VBLEND_MIX) return KLLM_E_INVALID;
+    if (a.differential && a.qk_norm == KLLM_SEQ_QKNORM_PROJECTION) return KLLM_E_UNSUPPORTED;
     if (a.vdim > 256 || a.dim > 512) return KLLM_E_UNSUPPORTED;
     if (a.window < 0 || a.keep_first < 0 || a.softcap < 0.f || a.conv_taps < 0 || a.rope_dims < 0 || a.rope_dims > a.dim ||
         (a.rope_dims & 1) || (a.rope_dims > 0 && a.rope_base <= 0.f))
       return KLLM_E_INVALID;
     if (a.values_are_keys && a.vdim != a.dim) return KLLM_E_INVALID;
     // the filtered, rotated form has its own preparation kernel: no head norms, temperature or gate there
-    const bool prep2 = a.values_are_keys || a.conv_taps > 1 || a.conv_w || a.in_bias;
-    if (prep2 && (!a.values_are_keys || a.qk_norm || a.gate || a.temp_every || a.rope_freq)) return KLLM_E_UNSUPPORTED;
+    const bool prep2 = a.values_are_keys || a.conv_taps > 1 || a.conv_w;
+    if (prep2 && (!a.values_are_keys || a.qk_norm || a.gate || a.temp_every || a.rope_freq || a.v_blend)) return KLLM_E_UNSUPPORTED;
   } else if (kind == KLLM_SEQ_MIXER_LATENT) {
     const kllm_seq_latent& a = L.latent;
-    if (a.heads <= 0 || a.dim <= 0 || a.rot_dim < 0 || a.vdim <= 0 || a.q_rank <= 0 || a.kv_rank <= 0 || a.window < 0 ||
+    if (a.heads <= 0 || a.dim <= 0 || a.rot_dim < 0 || a.vdim <= 0 || a.q_rank < 0 || a.kv_rank <= 0 || a.window < 0 ||
         a.rope_dims < 0 || a.rope_dims > a.rot_dim || (a.rope_dims & 1) || (a.rope_dims > 0 && a.rope_base <= 0.f) ||
-        !a.w_in || !a.q_norm_w || !a.kv_norm_w || !a.w_uq || !a.w_uk || !a.w_uv || !a.w_out)
+        !a.w_in || (a.q_rank > 0 && (!a.q_norm_w || !a.w_uq)) || !a.kv_norm_w || !a.w_uk || !a.w_uv || !a.w_out)
       return KLLM_E_INVALID;
+    if (a.gate != KLLM_SEQ_GATE_NONE && a.gate != KLLM_SEQ_GATE_HEAD) return KLLM_E_UNSUPPORTED;
     // the latent is the value of the paged attention kernel, latent + rotated part its key
     if (a.kv_rank > 256 || a.kv_rank + a.rot_dim > 512) return KLLM_E_UNSUPPORTED;
   } else if (kind == KLLM_SEQ_MIXER_LINEAR) {
@@ -306,10 +316,30 @@ static int validate(const kllm_seq_desc* d) {
       const kllm_seq_dense& f = L.dense;
       if (f.ff <= 0 || !f.up || !f.down || (!L.pre_ff.w && L.pre_ff.kind != KLLM_SEQ_NORM_NONE && !L.parallel_ff))
         return KLLM_E_INVALID;
-      if (f.act != KLLM_SEQ_ACT_XIELU && f.act != KLLM_SEQ_ACT_RELU2 && f.act != KLLM_SEQ_ACT_RELU_GATE) return KLLM_E_UNSUPPORTED;
+      if (f.act != KLLM_SEQ_ACT_XIELU && f.act != KLLM_SEQ_ACT_RELU2 && !dense_gated(f)) return KLLM_E_UNSUPPORTED;
     } else if (L.ff_kind != KLLM_SEQ_FF_NONE) {
       return KLLM_E_UNSUPPORTED;
     }
+    if (d->streams > 0) {  // the step between two sublayers is the streams' kernel: what it does not know is refused
+      const bool ff = L.ff_kind != KLLM_SEQ_FF_NONE;
+      for (const kllm_seq_hyper* h : {&L.hyper_mixer, ff ? &L.hyper_ff : &L.hyper_mixer})
+        if (!h->in || !h->out || !h->mix) return KLLM_E_INVALID;
+      if (L.post_mixer.w || L.post_ff.w || L.shift || L.mixer2_kind != 0 || L.parallel_ff || L.ff_kind == KLLM_SEQ_FF_MOE ||
+          L.mixer_out_norm.w)
+        return KLLM_E_UNSUPPORTED;
+    }
+  }
+  if (d->streams < 0) return KLLM_E_INVALID;
+  if (d->streams > kMaxStreams) return KLLM_E_UNSUPPORTED;
+  // every blend has a source ahead of it with the same value row
+  int source = -1;
+  for (int r = 0; r < d->n_runs; ++r) {
+    const kllm_seq_layer& L = d->layers[d->run_layer[r]];
+    if (d->streams > 0 && ((d->run_add && d->run_add[r] >= 0) || (d->run_embed && d->run_embed[r]))) return KLLM_E_UNSUPPORTED;
+    if (L.mixer_kind != KLLM_SEQ_MIXER_ATTENTION && L.mixer2_kind != KLLM_SEQ_MIXER_ATTENTION) continue;
+    const int row = L.attn.kv_heads * L.attn.vdim;
+    if (L.attn.v_blend == KLLM_SEQ_VBLEND_SOURCE) source = row;
+    if (L.attn.v_blend == KLLM_SEQ_VBLEND_MIX && source != row) return KLLM_E_INVALID;
   }
   return 0;
 }
@@ -412,11 +442,12 @@ extern "C" int kllm_seq_create(const kllm_seq_desc* desc, void* stream, kllm_seq
         e->max_q = std::max(e->max_q, a.heads * attn_maps(a) * a.dim);
         e->max_att = std::max(e->max_att, a.heads * a.vdim);
         e->max_gates = std::max(e->max_gates, gate_floats(attn_shape(a)));
+        if (a.v_blend == KLLM_SEQ_VBLEND_SOURCE) e->max_blend = std::max(e->max_blend, a.kv_heads * a.vdim);
       } else if (kind == KLLM_SEQ_MIXER_LATENT) {
         const kllm_seq_latent& a = L.latent;
-        e->max_proj = std::max(e->max_proj, a.q_rank + a.kv_rank + a.rot_dim + a.heads);
+        e->max_proj = std::max(e->max_proj, latent_proj_rows(latent_shape(a)));
         e->max_q = std::max(e->max_q, a.q_rank);
-        e->max_qf = std::max(e->max_qf, a.heads * (a.dim + a.rot_dim));
+        if (a.q_rank > 0) e->max_qf = std::max(e->max_qf, a.heads * (a.dim + a.rot_dim));
         e->max_qa = std::max(e->max_qa, a.heads * (a.kv_rank + a.rot_dim));
         e->max_ol = std::max(e->max_ol, a.heads * a.kv_rank);
         e->max_att = std::max(e->max_att, a.heads * a.vdim);
@@ -449,7 +480,7 @@ extern "C" int kllm_seq_create(const kllm_seq_desc* desc, void* stream, kllm_seq
       }
     }
     if (L.ff_kind == KLLM_SEQ_FF_DENSE) {
-      e->max_proj = std::max(e->max_proj, (L.dense.act == KLLM_SEQ_ACT_RELU_GATE ? 2 : 1) * L.dense.ff);
+      if (!dense_gated(L.dense)) e->max_proj = std::max(e->max_proj, L.dense.ff);  // the gated product writes its activations
       e->max_att = std::max(e->max_att, L.dense.ff);
     }
     if (L.ff_kind == KLLM_SEQ_FF_MOE) {
@@ -615,6 +646,8 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
   };
   const size_t Ts = static_cast<size_t>(T);
   RC(e->x.reserve(Ts * W * 4));
+  if (d.streams > 0) RC(e->xs.reserve(Ts * d.streams * W * 4));
+  if (e->max_blend > 0) RC(e->vfirst.reserve(Ts * e->max_blend * 4));
   RC(e->h.reserve(Ts * W * es));
   RC(e->proj.reserve(Ts * std::max({e->max_proj, 2 * e->max_sff, W}) * 4));
   RC(e->q.reserve(Ts * std::max(1, e->max_q) * es));
@@ -724,7 +757,8 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
       const PagedKV kv{e->k_pool[r], e->v_pool[r], e->table_dev, e->table_stride, e->page, shape.kv_heads * A.dim,
                        A.kv_heads * A.vdim};
       const int n_proj = attn_proj_rows(A);
-      RC(gemm(dtype, e->h.p, A.w_in, proj, T, W, n_proj, st));
+      // the filtered form adds its bias in its own preparation
+      RC(gemm(dtype, e->h.p, A.w_in, proj, T, W, n_proj, st, A.values_are_keys ? nullptr : A.in_bias));
       e->mark(KLLM_SEQ_PHASE_IN_PROJ);
       if (A.values_are_keys) {
         const AttnPrep prep{std::max(1, A.conv_taps), A.conv_w, e->attn_conv[r], A.in_bias, A.rope_dims, A.rope_pairing,
@@ -733,7 +767,8 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
       } else {
         const RopeArgs rope{A.rope_dims, A.rope_base, A.rope_freq, A.rope_mag, A.rope_pairing};
         RC(launch_qk_prepare(dtype, shape, rope, proj, A.q_norm_w, A.k_norm_w, d.norm_eps, d_seq, d_pos, e->q.p,
-                             static_cast<float*>(e->gates.p), kv, T, st));
+                             static_cast<float*>(e->gates.p), kv,
+                             ValueBlend{A.v_blend, A.v_lambda, static_cast<float*>(e->vfirst.p)}, T, st));
       }
       e->mark(KLLM_SEQ_PHASE_QK_PREPARE);
       RC(launch_attention(dtype, shape, e->q.p, static_cast<const float*>(e->gates.p), kv, n_entries, d_first, d_count,
@@ -744,37 +779,49 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
                              static_cast<const float*>(e->gates.p), A.diff_lambda, A.diff_out_scale, d.norm_eps, e->att.p, T,
                              st));
       e->mark(KLLM_SEQ_PHASE_ATTENTION);
-      RC(gemm(dtype, e->att.p, A.w_out, yout, T, A.heads * A.vdim, W, st));
+      RC(gemm(dtype, e->att.p, A.w_out, yout, T, A.heads * A.vdim, W, st, A.out_bias));
       e->mark(KLLM_SEQ_PHASE_OUT_PROJ);
     } else if (kind == KLLM_SEQ_MIXER_LATENT) {
       const kllm_seq_latent& A = L.latent;
-      const LatentShape ls{A.heads, A.dim, A.rot_dim, A.vdim, A.q_rank, A.kv_rank, A.rope_dims, A.rope_base};
+      const LatentShape ls = latent_shape(A);
       const int krow = A.kv_rank + A.rot_dim;
       const PagedKV kv{e->k_pool[r], e->k_pool[r], e->table_dev, e->table_stride, e->page, krow, krow};
-      float* gates = static_cast<float*>(e->gates.p);
-      RC(gemm(dtype, e->h.p, A.w_in, proj, T, W, A.q_rank + krow + A.heads, st));
+      float* gates = A.gate ? static_cast<float*>(e->gates.p) : nullptr;
+      const int n_proj = latent_proj_rows(ls);
+      RC(gemm(dtype, e->h.p, A.w_in, proj, T, W, n_proj, st));
       e->mark(KLLM_SEQ_PHASE_IN_PROJ);
+      // the queries: expanded from their own latent, or rows of the input projection
+      const float* queries = A.q_rank > 0 ? static_cast<const float*>(e->qf.p) : proj;
+      const int q_row = A.q_rank > 0 ? A.heads * (A.dim + A.rot_dim) : n_proj;
+      auto expand_queries = [&]() -> int {
+        return A.q_rank > 0 ? gemm(dtype, e->q.p, A.w_uq, static_cast<float*>(e->qf.p), T, A.q_rank, q_row, st) : 0;
+      };
       // Prompt steps whose sequences all start here: the step's own latents are all the keys there are, so they are
       // expanded into per-head keys and values (two products) and the tensor-core attention runs on those rows.  Every
       // other step scores against the cached latents (the absorbed form below).
       const int dqk = A.dim + A.rot_dim;
-      const AttnShape eshape{A.heads, A.heads, dqk, A.vdim, A.scale, 0.f, 0, 0, 1, A.window, A.sink, 0, 0, 0};
+      const AttnShape eshape{A.heads, A.heads, dqk, A.vdim, A.scale, 0.f, 0, 0, A.gate, A.window, A.sink, 0, 0, 0};
       if (fresh_prompt && attention_mma_usable(dtype, eshape, max_count)) {
         RC(e->lat_c.reserve(Ts * A.kv_rank * es));
         RC(e->lat_kr.reserve(Ts * std::max(1, A.rot_dim) * 4));
-        RC(e->lat_kp.reserve(Ts * A.heads * A.dim * 4));
-        RC(e->lat_vp.reserve(Ts * A.heads * A.vdim * 4));
+        // W_uk and W_uv side by side in memory are one product whose rows hold a token's keys, then its values
+        const int kn = A.heads * A.dim, vn = A.heads * A.vdim;
+        const bool stacked = static_cast<const char*>(A.w_uv) == static_cast<const char*>(A.w_uk) + static_cast<size_t>(kn) * A.kv_rank * es;
+        RC(e->lat_kp.reserve(Ts * (stacked ? kn + vn : kn) * 4));
+        if (!stacked) RC(e->lat_vp.reserve(Ts * vn * 4));
         RC(e->lat_q.reserve(Ts * A.heads * dqk * es));
         RC(e->lat_k.reserve(Ts * A.heads * dqk * es));
         RC(e->lat_v.reserve(Ts * A.heads * A.vdim * es));
         RC(launch_latent_prepare(dtype, ls, proj, A.q_norm_w, A.kv_norm_w, d.norm_eps, d_seq, d_pos, e->q.p, gates, kv,
                                  e->lat_c.p, static_cast<float*>(e->lat_kr.p), T, st));
-        RC(gemm(dtype, e->q.p, A.w_uq, static_cast<float*>(e->qf.p), T, A.q_rank, A.heads * dqk, st));
-        RC(launch_latent_pack_q(dtype, ls, static_cast<const float*>(e->qf.p), d_pos, e->lat_q.p, T, st));
-        RC(gemm(dtype, e->lat_c.p, A.w_uk, static_cast<float*>(e->lat_kp.p), T, A.kv_rank, A.heads * A.dim, st));
-        RC(gemm(dtype, e->lat_c.p, A.w_uv, static_cast<float*>(e->lat_vp.p), T, A.kv_rank, A.heads * A.vdim, st));
-        RC(launch_latent_pack_kv(dtype, ls, static_cast<const float*>(e->lat_kp.p), static_cast<const float*>(e->lat_kr.p),
-                                 static_cast<const float*>(e->lat_vp.p), e->lat_k.p, e->lat_v.p, T, st));
+        RC(expand_queries());
+        RC(launch_latent_pack_q(dtype, ls, queries, q_row, d_pos, e->lat_q.p, T, st));
+        float* kp = static_cast<float*>(e->lat_kp.p);
+        RC(gemm(dtype, e->lat_c.p, A.w_uk, kp, T, A.kv_rank, stacked ? kn + vn : kn, st));
+        if (!stacked) RC(gemm(dtype, e->lat_c.p, A.w_uv, static_cast<float*>(e->lat_vp.p), T, A.kv_rank, vn, st));
+        RC(launch_latent_pack_kv(dtype, ls, kp, stacked ? kn + vn : kn, static_cast<const float*>(e->lat_kr.p),
+                                 stacked ? kp + kn : static_cast<const float*>(e->lat_vp.p), stacked ? kn + vn : vn, e->lat_k.p,
+                                 e->lat_v.p, T, st));
         e->mark(KLLM_SEQ_PHASE_QK_PREPARE);
         const PagedKV rows{e->lat_k.p, e->lat_v.p, nullptr, 0, 1, A.heads * dqk, A.heads * A.vdim};
         RC(launch_attention(dtype, eshape, e->lat_q.p, gates, rows, n_entries, d_first, d_count, d_eseq, d_pos0, max_count,
@@ -785,13 +832,13 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
       } else {
       RC(launch_latent_prepare(dtype, ls, proj, A.q_norm_w, A.kv_norm_w, d.norm_eps, d_seq, d_pos, e->q.p, gates, kv, nullptr,
                                nullptr, T, st));
-      RC(gemm(dtype, e->q.p, A.w_uq, static_cast<float*>(e->qf.p), T, A.q_rank, A.heads * (A.dim + A.rot_dim), st));
-      RC(launch_latent_absorb(dtype, ls, static_cast<const float*>(e->qf.p), A.w_uk, d_pos, static_cast<float*>(e->qa.p), T, st));
+      RC(expand_queries());
+      RC(launch_latent_absorb(dtype, ls, queries, q_row, A.w_uk, d_pos, static_cast<float*>(e->qa.p), T, st));
       e->mark(KLLM_SEQ_PHASE_QK_PREPARE);
       // one shared key/value "head": keys [latent | rotated part], values the latent itself
       // steps of single tokens merge the key splits and apply W_uv in one kernel
       const bool fused_merge = single && T <= 32;
-      const AttnShape shape{A.heads, 1, krow, A.kv_rank, A.scale, 0.f, 0, 0, 1, A.window, A.sink, 1, 1, fused_merge ? 1 : 0};
+      const AttnShape shape{A.heads, 1, krow, A.kv_rank, A.scale, 0.f, 0, 0, A.gate, A.window, A.sink, 1, 1, fused_merge ? 1 : 0};
       const int lsplits = window_splits(A.window);
       RC(launch_attention(dtype, shape, e->qa.p, gates, kv, n_entries, d_first, d_count, d_eseq, d_pos0, max_count, max_ctx,
                           lsplits, static_cast<float*>(e->ws.p), e->ol.p, T, d_seq, d_pos, st));
@@ -869,9 +916,8 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
     *shared_out = false;
     if (L.ff_kind == KLLM_SEQ_FF_DENSE) {
       const kllm_seq_dense& F = L.dense;
-      if (F.act == KLLM_SEQ_ACT_RELU_GATE) {
-        RC(gemm(dtype, e->h.p, F.up, proj, T, W, 2 * F.ff, st));
-        RC(launch_gated_act(dtype, GatedAct{F.act, 0.f, 0.f}, proj, e->att.p, T, F.ff, st));
+      if (dense_gated(F)) {
+        RC(gemm_gated(dtype, e->h.p, F.up, e->att.p, T, W, F.ff, GatedAct{F.act, 0.f, 0.f}, st));
       } else {
         RC(gemm(dtype, e->h.p, F.up, proj, T, W, F.ff, st));
         RC(launch_activation(dtype, F.act, F.act_a, F.act_b, proj, e->att.p, Ts * F.ff, st));
@@ -937,8 +983,49 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
     }
     return 0;
   };
+  // Residual streams: every boundary between two sublayers is one kernel that ends the one before (its output y joins the
+  // streams through `done`) and starts the next (`next` reads the streams, its pre-norm writes h).
+  if (d.streams > 0) {
+    float* xs = static_cast<float*>(e->xs.p);
+    bool spread = false;  // false: every stream is still the embedding output in x
+    auto boundary = [&](const kllm_seq_hyper* done, const kllm_seq_hyper* next, const NormW& pre, void* out) {
+      StreamArgs a{};
+      a.src = spread ? xs : x, a.src_shared = spread ? 0 : 1;
+      if (done) a.dst = xs, a.y = y, a.mix = done->mix, a.out_w = done->out, spread = true;
+      if (next) a.in_w = next->in;
+      a.pre = pre, a.out = out, a.T = T, a.width = W, a.streams = d.streams, a.dtype = dtype, a.eps = d.norm_eps;
+      return a;
+    };
+    const kllm_seq_hyper* open = nullptr;  // a sublayer whose output is in y and has not joined the streams yet
+    for (int r = 0; r < d.n_runs; ++r) {
+      const kllm_seq_layer& L = e->layers[e->run_layer[r]];
+      RC(launch_streams(boundary(open, &L.hyper_mixer, nw(L.pre_mixer), e->h.p), st));
+      e->mark(KLLM_SEQ_PHASE_NORM);
+      RC(run_mixer(L, L.mixer_kind, r, y));
+      open = &L.hyper_mixer;
+      if (L.ff_kind != KLLM_SEQ_FF_NONE) {
+        RC(launch_streams(boundary(open, &L.hyper_ff, nw(L.pre_ff), e->h.p), st));
+        e->mark(KLLM_SEQ_PHASE_NORM);
+        bool shared = false;
+        RC(run_ff(L, y, &shared));
+        open = &L.hyper_ff;
+      }
+      if (tracing) {  // the sum of the streams after this run
+        StreamArgs a = boundary(open, nullptr, NormW{}, nullptr);
+        a.sum_out = y2;
+        RC(launch_streams(a, st));
+        open = nullptr;
+        CU(cudaMemcpyAsync(e->trace_host + static_cast<size_t>(r) * T * W, y2, Ts * W * 4, cudaMemcpyDeviceToHost, st));
+      }
+    }
+    if (n_want > 0) {  // the wanted rows only: nothing reads the streams after this
+      StreamArgs a = boundary(open, nullptr, nw(d.final_norm), e->hw.p);
+      a.dst = nullptr, a.rows = d_want, a.T = n_want;
+      RC(launch_streams(a, st));
+    }
+  }
   bool pre_done = false;  // the previous run's last kernel already produced this run's h
-  for (int r = 0; r < d.n_runs; ++r) {
+  for (int r = 0; d.streams == 0 && r < d.n_runs; ++r) {
     const kllm_seq_layer& L = e->layers[e->run_layer[r]];
     if (!pre_done) RC(launch_pre(ResidNormArgs{}, r, KLLM_SEQ_PHASE_NORM));
     pre_done = false;
@@ -996,10 +1083,12 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
 
   // ---- the wanted rows: final norm, classifier, greedy id -------------------------------------------------------
   if (n_want > 0) {
-    ResidNormArgs a{};
-    a.x = x, a.pre = nw(d.final_norm), a.out = e->hw.p, a.rows = d_want, a.T = n_want, a.width = W, a.dtype = dtype;
-    a.eps = d.norm_eps;
-    RC(launch_resid_norm(a, st));
+    if (d.streams == 0) {
+      ResidNormArgs a{};
+      a.x = x, a.pre = nw(d.final_norm), a.out = e->hw.p, a.rows = d_want, a.T = n_want, a.width = W, a.dtype = dtype;
+      a.eps = d.norm_eps;
+      RC(launch_resid_norm(a, st));
+    }
     float* lg = static_cast<float*>(e->logits.p);
     RC(gemm(dtype, e->hw.p, d.head, lg, n_want, W, d.vocab, st));
     if ((d.logit_scale != 0.f && d.logit_scale != 1.f) || d.logit_softcap > 0.f)

@@ -47,7 +47,7 @@ struct AttnShape {
   float scale;
   float temp_coef;  // query temperature 1 + coef * ln(floor((p + 1) / every) + 1); every == 0: none
   int temp_every;
-  int qk_norm;      // RMS norm of each query / key head with a shared weight vector
+  int qk_norm;      // KLLM_SEQ_QKNORM_*
   int gate;         // one sigmoid gate per (token, head) on the attention output
   int window;       // position i sees j with 0 <= i - j < window; 0: every earlier position
   const float* sink;  // [heads] or null: exp(sink) is added to the softmax denominator
@@ -87,6 +87,8 @@ __host__ __device__ inline float gated_act(const GatedAct& a, float g, float u) 
     return g / (1.0f + expf(-a.alpha * g)) * (u + 1.0f);
   }
   if (a.kind == KLLM_SEQ_ACT_RELU_GATE) return fmaxf(g, 0.f) * u;
+  if (a.kind == KLLM_SEQ_ACT_GELU_GATE)  // sqrt(2 / pi) (g + 0.044715 g^3)
+    return 0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u;
   return g / (1.0f + expf(-g)) * u;
 }
 
@@ -155,9 +157,16 @@ int launch_resid_norm(const ResidNormArgs& a, cudaStream_t s);
 // is written map-major inside each group of heads that share keys -- head h, map m of key group g goes to index
 // (g * v_share + m) * rep + h % rep, rep = query heads per key head -- so that the attention kernels find the rows of one
 // key head side by side.
+// KLLM_SEQ_QKNORM_PROJECTION norms all query rows together and all key rows together (weights of those sizes).
+// `blend`: the token's values are kept in blend.rows (SOURCE) or replaced by their blend with the rows kept there (MIX).
+struct ValueBlend {
+  int mode;      // KLLM_SEQ_VBLEND_*
+  float lambda;
+  float* rows;   // [T, value row] fp32
+};
 int launch_qk_prepare(int dtype, const AttnShape& a, const RopeArgs& rope, const float* qkvg, const float* qnorm_w,
                       const float* knorm_w, float eps, const int32_t* tok_seq, const int32_t* tok_pos, void* q, float* gates,
-                      const PagedKV& kv, int T, cudaStream_t s);
+                      const PagedKV& kv, const ValueBlend& blend, int T, cudaStream_t s);
 // Differential attention: joins the key splits of both maps of every head (a.no_merge left them in `ws`), then
 // o = a1 - lambda * a2, o / sqrt(mean(o^2) + eps) * out_scale over the head's vdim values, the output gate, and the
 // conversion: out [T, (heads / 2) * vdim] in the compute type.  `a` is the shape the attention ran with (v_share == 2).
@@ -190,9 +199,17 @@ struct LatentShape {
   int heads, dim, rot_dim, vdim, q_rank, kv_rank;
   int rope_dims;
   float rope_base;
+  int gate;                 // KLLM_SEQ_GATE_NONE / KLLM_SEQ_GATE_HEAD
+  int rope_pairing;         // KLLM_SEQ_ROPE_*
+  const float* rope_freq;   // [rope_dims / 2] or null (frequencies from the base)
 };
-// proj [T, q_rank + kv_rank + rot_dim + heads] fp32 -> cq [T, q_rank] (compute type, RMS-normed), the cache row
-// [kv_rank normed latent | rot_dim rotated key part] of every token, gates [T, heads] = sigmoid
+// rows of the input projection: query latent (or the queries themselves), key/value latent, rotated key part, gates
+inline __host__ __device__ int latent_query_rows(const LatentShape& a) { return a.q_rank > 0 ? a.q_rank : a.heads * (a.dim + a.rot_dim); }
+inline __host__ __device__ int latent_proj_rows(const LatentShape& a) {
+  return latent_query_rows(a) + a.kv_rank + a.rot_dim + (a.gate ? a.heads : 0);
+}
+// proj [T, latent_proj_rows()] fp32 -> cq [T, q_rank] (compute type, RMS-normed; nothing when q_rank == 0), the cache row
+// [kv_rank normed latent | rot_dim rotated key part] of every token, gates [T, heads] = sigmoid (when the shape has gates)
 int launch_latent_prepare(int dtype, const LatentShape& a, const float* proj, const float* q_norm_w, const float* kv_norm_w,
                           float eps, const int32_t* tok_seq, const int32_t* tok_pos, void* cq, float* gates,
                           const PagedKV& kv, void* c_rows, float* kr_rows, int T, cudaStream_t s);
@@ -200,12 +217,13 @@ int launch_latent_prepare(int dtype, const LatentShape& a, const float* proj, co
 // tensor-core attention on them: c_rows [T, kv_rank] (compute type) and kr_rows [T, rot_dim] (fp32, rotated) are the
 // step's latents as rows (optional outputs of latent_prepare); pack_q rotates and converts the queries; pack_kv joins
 // W_uk c with the shared rotated part and converts W_uv c.
-int launch_latent_pack_q(int dtype, const LatentShape& a, const float* q, const int32_t* tok_pos, void* out, int T,
+// Row strides: q_row floats between two tokens' queries, kp_row / vp_row between two tokens' expanded keys / values.
+int launch_latent_pack_q(int dtype, const LatentShape& a, const float* q, int q_row, const int32_t* tok_pos, void* out, int T,
                          cudaStream_t s);
-int launch_latent_pack_kv(int dtype, const LatentShape& a, const float* kp, const float* kr, const float* vp, void* k, void* v,
-                          int T, cudaStream_t s);
-// q [T, heads, dim + rot_dim] fp32 -> qa [T, heads, kv_rank + rot_dim] fp32: W_uk(head)^T q_plain | rotated q_rot
-int launch_latent_absorb(int dtype, const LatentShape& a, const float* q, const void* w_uk, const int32_t* tok_pos, float* qa,
+int launch_latent_pack_kv(int dtype, const LatentShape& a, const float* kp, int kp_row, const float* kr, const float* vp,
+                          int vp_row, void* k, void* v, int T, cudaStream_t s);
+// q [T, heads, dim + rot_dim] fp32 (rows q_row apart) -> qa [T, heads, kv_rank + rot_dim] fp32: W_uk(head)^T q_plain | rotated q_rot
+int launch_latent_absorb(int dtype, const LatentShape& a, const float* q, int q_row, const void* w_uk, const int32_t* tok_pos, float* qa,
                          int T, cudaStream_t s);
 // Single-token steps: the merge of the key splits (sink and gate included) and W_uv in one kernel, a CTA per (token, head).
 // ws: the partial results launch_attention left (AttnShape::no_merge) for value size kv_rank.
@@ -265,6 +283,27 @@ int launch_gated_act(int dtype, const GatedAct& act, const float* gu, void* out,
 // pairs ordered by expert in blocks of `block` rows (padded with -1), and the expert of every block.
 int launch_sort_pairs(const int32_t* top_idx, int n_pairs, int experts, int block, int32_t* counts /*[experts+1]*/,
                       int32_t* sorted_pair /*[cap]*/, int32_t* block_expert /*[cap/block]*/, int cap, cudaStream_t s);
+
+// ---- seq_streams.cu: residual streams joined by hyper-connections -------------------------------------------------------
+// Row t of S streams [T, S, width]: x_t <- sum_s mix[s][t] x_s + out_w[t] y (when y is given), then u = sum_s in_w[s] x_s (in_w
+// null: the plain sum) and out = N(u; pre) in the compute type.
+struct StreamArgs {
+  const float* src;      // [T, S, width], or [T, width] when src_shared: every stream is still that row
+  int src_shared;
+  float* dst;            // [T, S, width]: the new streams (may be src); null: they are not kept
+  const float* y;        // [T, width] output of the sublayer that ends here, or null
+  const float* mix;      // its hyper-connection, [S][S] and [S]
+  const float* out_w;
+  const float* in_w;     // of the sublayer that starts here, or null
+  NormW pre;
+  void* out;             // null: no normed rows
+  float* sum_out;        // [T, width] fp32 u before the norm, or null
+  const int32_t* rows;   // row i reads src / y row rows[i] (dst must be null), or null
+  int T, width, streams, dtype;
+  float eps;
+};
+constexpr int kMaxStreams = 32;
+int launch_streams(const StreamArgs& a, cudaStream_t s);
 
 // ---- seq_recurrent.cu: short convolutions with their state, query / key preparation behind one, selective scan, gated delta rule ----
 // Where the last taps - 1 inputs of a convolution live: [slots][taps - 1][channels] fp32, row i of a sequence of length n
@@ -343,8 +382,10 @@ int launch_ssd_out(int dtype, const kllm_seq_ssd& m, const float* y, const float
                    cudaStream_t s);
 
 // ---- seq_gemm.cu --------------------------------------------------------------------------------------------------
-// out[T, N] (fp32) = a[T, K] . w[N, K]^T, a and w in the compute type, fp32 accumulation.
-int gemm(int dtype, const void* a, const void* w, float* out, int T, int K, int N, cudaStream_t s);
+// out[T, N] (fp32) = a[T, K] . w[N, K]^T (+ bias[N]), a and w in the compute type, fp32 accumulation.
+int gemm(int dtype, const void* a, const void* w, float* out, int T, int K, int N, cudaStream_t s, const float* bias = nullptr);
+// out[T, ff] (compute type) = gated_act(a . wg^T, a . wu^T), w = [ff gate rows, then ff up rows][K]
+int gemm_gated(int dtype, const void* a, const void* w, void* out, int T, int K, int ff, const GatedAct& act, cudaStream_t s);
 // != 0 when a bounded wait inside a tensor-core product ran out since the last call (checked after a step's sync)
 int gemm_take_error();
 // Grouped form for the routed experts: block b (of `block` rows) multiplies rows a[row_of(b, i)] with the weights of

@@ -4,6 +4,8 @@
 //   rows_kernel     T <= 8 (decode steps): the weights are streamed once, a warp per output feature, all rows of `a`
 //                   against each 16-byte weight vector -- bound by the weight bytes
 //   tiled_kernel    any shape: 64 x 64 x 16 tiles through shared memory, 4 x 4 outputs per thread (fp32 FMA)
+// Every form adds an optional bias per output feature.  The gated form (gate rows, then up rows) joins the two products with
+// the activation in its epilogue and writes the compute type.
 //   umma_kernel     bf16, T >= 64, K % 8 == 0: 128 weight rows x BN tokens per CTA on tcgen05.mma (kind::f16, operands
 //                   by TMA with 128-byte swizzle, accumulator in TMEM)                      [seq_gemm_umma.cuh]
 //   grouped_kernel  the tiled kernel over row blocks that each belong to one expert (rows gathered by index, the
@@ -64,7 +66,8 @@ template <> struct Vec16<__nv_bfloat16> {
 // ---- a few rows against every weight row ----------------------------------------------------------------------------
 template <typename AT, int R, bool VEC>
 __global__ void __launch_bounds__(256)
-rows_kernel(const AT* __restrict__ a, const AT* __restrict__ w, float* __restrict__ out, int T, int K, int N) {
+rows_kernel(const AT* __restrict__ a, const AT* __restrict__ w, const float* __restrict__ bias, float* __restrict__ out, int T,
+            int K, int N) {
   constexpr int V = Vec16<AT>::N;
   const int lane = threadIdx.x & 31;
   const int n = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -100,7 +103,57 @@ rows_kernel(const AT* __restrict__ a, const AT* __restrict__ w, float* __restric
     float v = acc[r];
 #pragma unroll
     for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-    if (lane == 0 && r < T) out[static_cast<size_t>(r) * N + n] = v;
+    if (lane == 0 && r < T) out[static_cast<size_t>(r) * N + n] = bias ? v + bias[n] : v;
+  }
+}
+
+// The gated form: a warp owns feature f and streams its gate row and its up row together.
+template <typename AT, int R, bool VEC>
+__global__ void __launch_bounds__(256)
+rows_gated_kernel(const AT* __restrict__ a, const AT* __restrict__ w, AT* __restrict__ out, int T, int K, int N, GatedAct act) {
+  constexpr int V = Vec16<AT>::N;
+  const int lane = threadIdx.x & 31;
+  const int n = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (n >= N) return;
+  const AT* wg = w + static_cast<size_t>(n) * K;
+  const AT* wu = w + static_cast<size_t>(N + n) * K;
+  float g[R], u[R];
+#pragma unroll
+  for (int r = 0; r < R; ++r) g[r] = u[r] = 0.f;
+  if (VEC) {
+    for (int k = lane * V; k < K; k += 32 * V) {
+      float gf[V], uf[V];
+      Vec16<AT>::load_stream(wg + k, gf);
+      Vec16<AT>::load_stream(wu + k, uf);
+#pragma unroll
+      for (int r = 0; r < R; ++r) {
+        if (r < T) {
+          float af[V];
+          Vec16<AT>::load(a + static_cast<size_t>(r) * K + k, af);
+#pragma unroll
+          for (int i = 0; i < V; ++i) g[r] = fmaf(af[i], gf[i], g[r]), u[r] = fmaf(af[i], uf[i], u[r]);
+        }
+      }
+    }
+  } else {
+    for (int k = lane; k < K; k += 32) {
+      const float gv = ld_f(wg + k), uv = ld_f(wu + k);
+#pragma unroll
+      for (int r = 0; r < R; ++r)
+        if (r < T) {
+          const float av = ld_f(a + static_cast<size_t>(r) * K + k);
+          g[r] = fmaf(av, gv, g[r]), u[r] = fmaf(av, uv, u[r]);
+        }
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < R; ++r) {
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      g[r] += __shfl_xor_sync(0xffffffffu, g[r], o);
+      u[r] += __shfl_xor_sync(0xffffffffu, u[r], o);
+    }
+    if (lane == 0 && r < T) st_t(out + static_cast<size_t>(r) * N + n, gated_act(act, g[r], u[r]));
   }
 }
 
@@ -114,7 +167,7 @@ template <typename AT, bool GROUPED, int EPI>
 __global__ void __launch_bounds__(256)
 tiled_kernel(const AT* __restrict__ a, const AT* __restrict__ w, void* __restrict__ out_, int T, int K, int N,
              const int32_t* __restrict__ sorted_pair, const int32_t* __restrict__ block_expert, int a_row_div,
-             GatedAct act = GatedAct{KLLM_SEQ_ACT_SWIGLU, 0.f, 0.f}) {
+             GatedAct act = GatedAct{KLLM_SEQ_ACT_SWIGLU, 0.f, 0.f}, const float* __restrict__ bias = nullptr) {
   __shared__ float As[TK][TM + 4];
   __shared__ float Ws[EPI == 1 ? 2 : 1][TK][TN + 4];
   __shared__ int32_t rowsrc[TM], rowdst[TM];
@@ -194,14 +247,14 @@ tiled_kernel(const AT* __restrict__ a, const AT* __restrict__ w, void* __restric
         const float u = fmaxf(acc[0][i][j], 0.f);
         st_t(static_cast<AT*>(out_) + static_cast<size_t>(dst) * N + n, u * u);
       } else {
-        static_cast<float*>(out_)[static_cast<size_t>(dst) * N + n] = acc[0][i][j];
+        static_cast<float*>(out_)[static_cast<size_t>(dst) * N + n] = bias ? acc[0][i][j] + bias[n] : acc[0][i][j];
       }
     }
   }
 }
 
 template <typename AT>
-int gemm_t(const AT* a, const AT* w, float* out, int T, int K, int N, cudaStream_t s, bool* umma_used) {
+int gemm_t(const AT* a, const AT* w, const float* bias, float* out, int T, int K, int N, cudaStream_t s, bool* umma_used) {
   constexpr int V = Vec16<AT>::N;
   if (T <= 8) {
     const bool vec = (K % V) == 0 && (reinterpret_cast<uintptr_t>(a) & 15) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0;
@@ -209,8 +262,8 @@ int gemm_t(const AT* a, const AT* w, float* out, int T, int K, int N, cudaStream
     const dim3 grid((N + warps - 1) / warps);
 #define KLLM_ROWS(R)                                                                  \
   do {                                                                                \
-    if (vec) rows_kernel<AT, R, true><<<grid, warps * 32, 0, s>>>(a, w, out, T, K, N); \
-    else rows_kernel<AT, R, false><<<grid, warps * 32, 0, s>>>(a, w, out, T, K, N);    \
+    if (vec) rows_kernel<AT, R, true><<<grid, warps * 32, 0, s>>>(a, w, bias, out, T, K, N); \
+    else rows_kernel<AT, R, false><<<grid, warps * 32, 0, s>>>(a, w, bias, out, T, K, N);    \
   } while (0)
     if (T <= 1) KLLM_ROWS(1);
     else if (T <= 2) KLLM_ROWS(2);
@@ -222,10 +275,42 @@ int gemm_t(const AT* a, const AT* w, float* out, int T, int K, int N, cudaStream
   }
   if (umma::usable<AT>(a, w, T, K, N)) {
     *umma_used = true;
-    return umma::launch(a, w, out, T, K, N, s);
+    return umma::launch(a, w, bias, out, T, K, N, s);
   }
   const dim3 grid((N + TN - 1) / TN, (T + TM - 1) / TM);
-  tiled_kernel<AT, false, 0><<<grid, 256, 0, s>>>(a, w, out, T, K, N, nullptr, nullptr, 1);
+  tiled_kernel<AT, false, 0><<<grid, 256, 0, s>>>(a, w, out, T, K, N, nullptr, nullptr, 1,
+                                                 GatedAct{KLLM_SEQ_ACT_SWIGLU, 0.f, 0.f}, bias);
+  count_launch();
+  return cuda_rc(cudaGetLastError());
+}
+
+template <typename AT>
+int gemm_gated_t(const AT* a, const AT* w, AT* out, int T, int K, int N, const GatedAct& act, cudaStream_t s, bool* umma_used) {
+  constexpr int V = Vec16<AT>::N;
+  if (T <= 8) {
+    const bool vec = (K % V) == 0 && (reinterpret_cast<uintptr_t>(a) & 15) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0;
+    // a warp per feature; four warps per CTA spread a small inner size over more SMs
+    const int warps = 4;
+    const dim3 grid((N + warps - 1) / warps);
+#define KLLM_ROWS(R)                                                                                \
+  do {                                                                                              \
+    if (vec) rows_gated_kernel<AT, R, true><<<grid, warps * 32, 0, s>>>(a, w, out, T, K, N, act);    \
+    else rows_gated_kernel<AT, R, false><<<grid, warps * 32, 0, s>>>(a, w, out, T, K, N, act);       \
+  } while (0)
+    if (T <= 1) KLLM_ROWS(1);
+    else if (T <= 2) KLLM_ROWS(2);
+    else if (T <= 4) KLLM_ROWS(4);
+    else KLLM_ROWS(8);
+#undef KLLM_ROWS
+    count_launch();
+    return cuda_rc(cudaGetLastError());
+  }
+  if (umma::usable<AT>(a, w, T, K, N)) {
+    *umma_used = true;
+    return umma::launch_gated(a, w, out, T, K, N, act, s);
+  }
+  const dim3 grid((N + TN - 1) / TN, (T + TM - 1) / TM);
+  tiled_kernel<AT, false, 1><<<grid, 256, 0, s>>>(a, w, out, T, K, N, nullptr, nullptr, 1, act);
   count_launch();
   return cuda_rc(cudaGetLastError());
 }
@@ -250,11 +335,23 @@ int grouped_t(const GroupedArgs& g, cudaStream_t s) {
 }  // namespace
 
 static bool g_umma_used;
-int gemm(int dtype, const void* a, const void* w, float* out, int T, int K, int N, cudaStream_t s) {
+int gemm(int dtype, const void* a, const void* w, float* out, int T, int K, int N, cudaStream_t s, const float* bias) {
   if (!a || !w || !out || T <= 0 || K <= 0 || N <= 0) return KLLM_E_INVALID;
-  if (dtype == KLLM_SEQ_F32) return gemm_t(static_cast<const float*>(a), static_cast<const float*>(w), out, T, K, N, s, &g_umma_used);
+  if (dtype == KLLM_SEQ_F32)
+    return gemm_t(static_cast<const float*>(a), static_cast<const float*>(w), bias, out, T, K, N, s, &g_umma_used);
   if (dtype == KLLM_SEQ_BF16)
-    return gemm_t(static_cast<const __nv_bfloat16*>(a), static_cast<const __nv_bfloat16*>(w), out, T, K, N, s, &g_umma_used);
+    return gemm_t(static_cast<const __nv_bfloat16*>(a), static_cast<const __nv_bfloat16*>(w), bias, out, T, K, N, s, &g_umma_used);
+  return KLLM_E_INVALID;
+}
+
+int gemm_gated(int dtype, const void* a, const void* w, void* out, int T, int K, int ff, const GatedAct& act, cudaStream_t s) {
+  if (!a || !w || !out || T <= 0 || K <= 0 || ff <= 0) return KLLM_E_INVALID;
+  if (dtype == KLLM_SEQ_F32)
+    return gemm_gated_t(static_cast<const float*>(a), static_cast<const float*>(w), static_cast<float*>(out), T, K, ff, act, s,
+                        &g_umma_used);
+  if (dtype == KLLM_SEQ_BF16)
+    return gemm_gated_t(static_cast<const __nv_bfloat16*>(a), static_cast<const __nv_bfloat16*>(w),
+                        static_cast<__nv_bfloat16*>(out), T, K, ff, act, s, &g_umma_used);
   return KLLM_E_INVALID;
 }
 

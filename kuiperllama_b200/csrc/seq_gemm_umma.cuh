@@ -1,5 +1,7 @@
 // bf16 token-block product on the 5th-generation tensor cores (sm_100a):
-//     out[T, N] (fp32) = a[T, K] (bf16) . w[N, K]^T (bf16), fp32 accumulation in TMEM
+//     out[T, N] (fp32) = a[T, K] (bf16) . w[N, K]^T (bf16) (+ bias[N]), fp32 accumulation in TMEM
+// and its gated form: w holds N gate rows, then N up rows; both accumulate side by side in TMEM and
+//     out[T, N] (bf16) = gated_act(a . gate^T, a . up^T)
 //
 // One CTA computes 128 weight rows x BN tokens.  The weight rows are the M side of tcgen05.mma (so an accumulator lane
 // is an output feature and a column is a token), the tokens the N side.  Six warps:
@@ -94,16 +96,17 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&r)[32]) {
       : "r"(taddr) : "memory");
 }
 
-template <int BN>
+template <int BN, bool GATED>
 __global__ void __launch_bounds__(THREADS, 1)
 umma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_a,
-            float* __restrict__ out, int T, int N, int K) {
-  constexpr int B_BYTES = BN * BK * 2;
-  constexpr uint32_t TMEM_COLS = BN < 32 ? 32 : BN;
+            void* __restrict__ out_, const float* __restrict__ bias, int T, int N, int K, GatedAct act) {
+  constexpr int NA = GATED ? 2 : 1;  // weight tiles per stage
+  constexpr int W_BYTES = NA * A_BYTES, B_BYTES = BN * BK * 2;
+  constexpr uint32_t TMEM_COLS = NA * (BN < 32 ? 32 : BN);
   extern __shared__ uint8_t raw_smem[];
   uint8_t* base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(raw_smem) + 1023) & ~uintptr_t(1023));
   uint8_t* a_tiles = base;                       // weight tiles (MMA A)
-  uint8_t* b_tiles = base + STAGES * A_BYTES;    // token tiles (MMA B)
+  uint8_t* b_tiles = base + STAGES * W_BYTES;    // token tiles (MMA B)
   uint64_t* bars = reinterpret_cast<uint64_t*>(b_tiles + STAGES * B_BYTES);
   uint64_t* full = bars;
   uint64_t* empty = bars + STAGES;
@@ -140,8 +143,9 @@ umma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ C
         const int s = kb % STAGES;
         if (!mbar_wait(smem_u32(&empty[s]), ((kb / STAGES) & 1) ^ 1u, stop)) break;
         const uint32_t bar = smem_u32(&full[s]);
-        mbar_expect_tx(bar, A_BYTES + B_BYTES);
-        tma_load_2d(smem_u32(a_tiles + s * A_BYTES), &map_w, bar, kb * BK, n0);
+        mbar_expect_tx(bar, W_BYTES + B_BYTES);
+        tma_load_2d(smem_u32(a_tiles + s * W_BYTES), &map_w, bar, kb * BK, n0);
+        if (GATED) tma_load_2d(smem_u32(a_tiles + s * W_BYTES + A_BYTES), &map_w, bar, kb * BK, N + n0);
         tma_load_2d(smem_u32(b_tiles + s * B_BYTES), &map_a, bar, kb * BK, t0);
       }
     }
@@ -154,11 +158,14 @@ umma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ C
         ok = mbar_wait(smem_u32(&full[s]), (kb / STAGES) & 1, stop);
         if (!ok) break;
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
-        const uint32_t a_addr = smem_u32(a_tiles + s * A_BYTES);
+        const uint32_t a_addr = smem_u32(a_tiles + s * W_BYTES);
         const uint32_t b_addr = smem_u32(b_tiles + s * B_BYTES);
 #pragma unroll
-        for (int k = 0; k < BK / UK; ++k)  // 32 bytes of K per instruction, inside the swizzle row
-          mma_bf16(tmem_d, smem_desc(a_addr + k * UK * 2), smem_desc(b_addr + k * UK * 2), idesc, (kb > 0 || k > 0) ? 1u : 0u);
+        for (int z = 0; z < NA; ++z)
+#pragma unroll
+          for (int k = 0; k < BK / UK; ++k)  // 32 bytes of K per instruction, inside the swizzle row
+            mma_bf16(tmem_d + z * BN, smem_desc(a_addr + z * A_BYTES + k * UK * 2), smem_desc(b_addr + k * UK * 2), idesc,
+                     (kb > 0 || k > 0) ? 1u : 0u);
         mma_commit(smem_u32(&empty[s]));
       }
       if (ok) mma_commit(smem_u32(tmem_full));
@@ -168,25 +175,24 @@ umma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ C
     if (mbar_wait(smem_u32(tmem_full), 0u, stop)) {
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       const int row = n0 + quarter * 32 + lane;
+      const float add = !GATED && bias != nullptr && row < N ? bias[row] : 0.f;
 #pragma unroll 1
       for (int c = 0; c < BN; c += 32) {
-        uint32_t r[32];
+        uint32_t r[32], u[GATED ? 32 : 1];
         const uint32_t taddr = tmem_d + (static_cast<uint32_t>(quarter * 32) << 16) + static_cast<uint32_t>(c);
-        asm volatile(
-            "tcgen05.ld.sync.aligned.32x32b.x32.b32 "
-            "{%0, %1, %2, %3, %4, %5, %6, %7, %8, %9, %10, %11, %12, %13, %14, %15, "
-            "%16, %17, %18, %19, %20, %21, %22, %23, %24, %25, %26, %27, %28, %29, %30, %31}, [%32];"
-            : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]), "=r"(r[4]), "=r"(r[5]), "=r"(r[6]), "=r"(r[7]),
-              "=r"(r[8]), "=r"(r[9]), "=r"(r[10]), "=r"(r[11]), "=r"(r[12]), "=r"(r[13]), "=r"(r[14]), "=r"(r[15]),
-              "=r"(r[16]), "=r"(r[17]), "=r"(r[18]), "=r"(r[19]), "=r"(r[20]), "=r"(r[21]), "=r"(r[22]), "=r"(r[23]),
-              "=r"(r[24]), "=r"(r[25]), "=r"(r[26]), "=r"(r[27]), "=r"(r[28]), "=r"(r[29]), "=r"(r[30]), "=r"(r[31])
-            : "r"(taddr) : "memory");
+        tmem_ld32(taddr, r);
+        if constexpr (GATED) tmem_ld32(taddr + BN, u);
         asm volatile("tcgen05.wait::ld.sync.aligned;" ::: "memory");
         if (row < N) {
 #pragma unroll
           for (int j = 0; j < 32; ++j) {
             const int t = t0 + c + j;
-            if (t < T) out[static_cast<size_t>(t) * N + row] = __uint_as_float(r[j]);
+            if (t >= T) continue;
+            if constexpr (GATED)
+              static_cast<__nv_bfloat16*>(out_)[static_cast<size_t>(t) * N + row] =
+                  __float2bfloat16_rn(gated_act(act, __uint_as_float(r[j]), __uint_as_float(u[j])));
+            else
+              static_cast<float*>(out_)[static_cast<size_t>(t) * N + row] = __uint_as_float(r[j]) + add;
           }
         }
       }
@@ -373,21 +379,23 @@ inline int make_map(CUtensorMap* map, const void* ptr, int rows, int cols, int b
   return r == CUDA_SUCCESS ? 0 : KLLM_E_INVALID;
 }
 
-template <int BN>
-inline int launch_bn(const void* a, const void* w, float* out, int T, int K, int N, cudaStream_t stream) {
+template <int BN, bool GATED>
+inline int launch_bn(const void* a, const void* w, const float* bias, void* out, int T, int K, int N, const GatedAct& act,
+                     cudaStream_t stream) {
+  constexpr int NA = GATED ? 2 : 1;
   CUtensorMap map_w, map_a;
-  if (int rc = make_map(&map_w, w, N, K, BM)) return rc;
+  if (int rc = make_map(&map_w, w, NA * N, K, BM)) return rc;
   if (int rc = make_map(&map_a, a, T, K, BN)) return rc;
-  const size_t smem = 1024 + static_cast<size_t>(STAGES) * (A_BYTES + BN * BK * 2) + 256;
+  const size_t smem = 1024 + static_cast<size_t>(STAGES) * (NA * A_BYTES + BN * BK * 2) + 256;
   static bool configured = false;
   if (!configured) {
-    const cudaError_t e = cudaFuncSetAttribute(umma_kernel<BN>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    const cudaError_t e = cudaFuncSetAttribute(umma_kernel<BN, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
     configured = true;
   }
   const dim3 grid((N + BM - 1) / BM, (T + BN - 1) / BN);
-  umma_kernel<BN><<<grid, THREADS, smem, stream>>>(map_w, map_a, out, T, N, K);
+  umma_kernel<BN, GATED><<<grid, THREADS, smem, stream>>>(map_w, map_a, out, bias, T, N, K, act);
   count_launch();
   return static_cast<int>(cudaGetLastError());
 }
@@ -402,15 +410,27 @@ inline bool usable<__nv_bfloat16>(const __nv_bfloat16* a, const __nv_bfloat16* w
 }
 
 template <typename AT>
-inline int launch(const AT*, const AT*, float*, int, int, int, cudaStream_t) { return KLLM_E_UNSUPPORTED; }
+inline int launch(const AT*, const AT*, const float*, float*, int, int, int, cudaStream_t) { return KLLM_E_UNSUPPORTED; }
 template <>
-inline int launch<__nv_bfloat16>(const __nv_bfloat16* a, const __nv_bfloat16* w, float* out, int T, int K, int N,
-                                 cudaStream_t s) {
+inline int launch<__nv_bfloat16>(const __nv_bfloat16* a, const __nv_bfloat16* w, const float* bias, float* out, int T, int K,
+                                 int N, cudaStream_t s) {
+  const GatedAct none{KLLM_SEQ_ACT_SWIGLU, 0.f, 0.f};
   // few feature tiles: narrower token blocks give more CTAs
   const int feature_tiles = (N + BM - 1) / BM;
-  if (T <= 64 || feature_tiles * ((T + 127) / 128) < 100) return launch_bn<64>(a, w, out, T, K, N, s);
-  if (T <= 128 || feature_tiles * ((T + 255) / 256) < 148) return launch_bn<128>(a, w, out, T, K, N, s);
-  return launch_bn<256>(a, w, out, T, K, N, s);
+  if (T <= 64 || feature_tiles * ((T + 127) / 128) < 100) return launch_bn<64, false>(a, w, bias, out, T, K, N, none, s);
+  if (T <= 128 || feature_tiles * ((T + 255) / 256) < 148) return launch_bn<128, false>(a, w, bias, out, T, K, N, none, s);
+  return launch_bn<256, false>(a, w, bias, out, T, K, N, none, s);
+}
+
+// w: [2 * N, K], gate rows then up rows; two weight tiles share a token tile, so a CTA computes 128 features x BN tokens twice
+template <typename AT>
+inline int launch_gated(const AT*, const AT*, AT*, int, int, int, const GatedAct&, cudaStream_t) { return KLLM_E_UNSUPPORTED; }
+template <>
+inline int launch_gated<__nv_bfloat16>(const __nv_bfloat16* a, const __nv_bfloat16* w, __nv_bfloat16* out, int T, int K, int N,
+                                       const GatedAct& act, cudaStream_t s) {
+  const int feature_tiles = (N + BM - 1) / BM;
+  if (T <= 64 || feature_tiles * ((T + 127) / 128) < 100) return launch_bn<64, true>(a, w, nullptr, out, T, K, N, act, s);
+  return launch_bn<128, true>(a, w, nullptr, out, T, K, N, act, s);
 }
 
 inline bool grouped_usable(int K, int N) {

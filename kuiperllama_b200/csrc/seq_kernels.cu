@@ -469,12 +469,14 @@ __device__ __forceinline__ AT* page_row(AT* base, const PagedKV& kv, int seq, in
 // One warp per query / key head (per map of a head, when the heads hold several): the head's row goes through shared
 // memory -- head norm with weights (before the rotation), rotation of the first rope.dims coordinates, unit norm (after
 // it), temperature -- and leaves as a query row or as the key row of the token's page.  Angles, cos and sin are fp32.
+// One norm over all query rows (and one over all key rows) takes its two sums of squares over the CTA first.
 template <typename AT>
 __global__ void qk_prepare_kernel(AttnShape a, RopeArgs rope, const float* __restrict__ qkvg,
                                   const float* __restrict__ qnorm_w, const float* __restrict__ knorm_w, float eps,
                                   const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ tok_pos,
-                                  AT* __restrict__ q, float* __restrict__ gates, PagedKV kv) {
+                                  AT* __restrict__ q, float* __restrict__ gates, PagedKV kv, ValueBlend blend) {
   extern __shared__ float head_rows[];  // [warps][dim]
+  __shared__ float red[33];
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
   const int maps = v_share_of(a);
   const int qn = a.heads * a.dim, kn = a.kv_heads * a.dim, vn = a.kv_heads / maps * a.vdim, gn = gate_floats(a);
@@ -489,6 +491,16 @@ __global__ void qk_prepare_kernel(AttnShape a, RopeArgs rope, const float* __res
   const int rd = rope.dims, half = rd / 2;
   const float inv_dim = 1.0f / static_cast<float>(a.dim);
   float* hr = head_rows + warp * a.dim;
+  const bool whole = a.qk_norm == KLLM_SEQ_QKNORM_PROJECTION, weighted = whole || a.qk_norm == KLLM_SEQ_QKNORM_WEIGHTED;
+  float rq = 1.0f, rk = 1.0f;
+  if (whole) {
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < qn; i += blockDim.x) ss = fmaf(row[i], row[i], ss);
+    rq = 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(qn) + eps);
+    ss = 0.f;
+    for (int i = threadIdx.x; i < kn; i += blockDim.x) ss = fmaf(row[qn + i], row[qn + i], ss);
+    rk = 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(kn) + eps);
+  }
   for (int u = warp; u < a.heads + a.kv_heads; u += nw) {
     const bool is_q = u < a.heads;
     const float* src = row + (is_q ? u * a.dim : qn + (u - a.heads) * a.dim);
@@ -501,14 +513,14 @@ __global__ void qk_prepare_kernel(AttnShape a, RopeArgs rope, const float* __res
     } else {
       dst = krow + (u - a.heads) * a.dim;
     }
-    float rinv = 1.0f;
+    float rinv = is_q ? rq : rk;
     if (a.qk_norm == KLLM_SEQ_QKNORM_WEIGHTED) {
       float ss = 0.f;
       for (int d = lane; d < a.dim; d += 32) ss = fmaf(src[d], src[d], ss);
       rinv = 1.0f / sqrtf(warp_sum(ss) * inv_dim + eps);
     }
-    const float* nw_ = is_q ? qnorm_w : knorm_w;
-    for (int d = lane; d < a.dim; d += 32) hr[d] = a.qk_norm == KLLM_SEQ_QKNORM_WEIGHTED ? src[d] * rinv * nw_[d] : src[d];
+    const float* nw_ = (is_q ? qnorm_w : knorm_w) + (whole ? (is_q ? u : u - a.heads) * a.dim : 0);
+    for (int d = lane; d < a.dim; d += 32) hr[d] = weighted ? src[d] * rinv * nw_[d] : src[d];
     __syncwarp();
     for (int i = lane; i < half; i += 32) {
       const int d0 = rope.pairing == KLLM_SEQ_ROPE_PAIRS ? 2 * i : i, d1 = rope.pairing == KLLM_SEQ_ROPE_PAIRS ? 2 * i + 1 : i + half;
@@ -529,7 +541,12 @@ __global__ void qk_prepare_kernel(AttnShape a, RopeArgs rope, const float* __res
     for (int d = lane; d < a.dim; d += 32) dst[d] = from_f<AT>(hr[d] * post);
     __syncwarp();
   }
-  for (int i = threadIdx.x; i < vn; i += blockDim.x) vrow[i] = from_f<AT>(row[qn + kn + i]);
+  for (int i = threadIdx.x; i < vn; i += blockDim.x) {
+    float v = row[qn + kn + i];
+    if (blend.mode == KLLM_SEQ_VBLEND_SOURCE) blend.rows[static_cast<size_t>(t) * vn + i] = v;
+    if (blend.mode == KLLM_SEQ_VBLEND_MIX) v = (1.0f - blend.lambda) * v + blend.lambda * blend.rows[static_cast<size_t>(t) * vn + i];
+    vrow[i] = from_f<AT>(v);
+  }
   for (int i = threadIdx.x; i < gn; i += blockDim.x)
     gates[static_cast<size_t>(t) * gn + i] = 1.0f / (1.0f + expf(-row[qn + kn + vn + i]));
 }
@@ -1124,7 +1141,7 @@ int launch_resid_norm(const ResidNormArgs& a, cudaStream_t s) {
 
 int launch_qk_prepare(int dtype, const AttnShape& a, const RopeArgs& rope_, const float* qkvg, const float* qnorm_w,
                       const float* knorm_w, float eps, const int32_t* tok_seq, const int32_t* tok_pos, void* q, float* gates,
-                      const PagedKV& kv, int T, cudaStream_t s) {
+                      const PagedKV& kv, const ValueBlend& blend, int T, cudaStream_t s) {
   RopeArgs rope = rope_;
   if (rope.mag == 0.f) rope.mag = 1.0f;
   if (rope.dims < 0 || (rope.dims & 1) || rope.dims > a.dim || a.kv_heads % v_share_of(a) || a.heads % v_share_of(a) ||
@@ -1136,7 +1153,7 @@ int launch_qk_prepare(int dtype, const AttnShape& a, const RopeArgs& rope_, cons
   warps = std::max(1, std::min(warps, 48 * 1024 / (4 * a.dim)));
   const size_t smem = static_cast<size_t>(warps) * a.dim * sizeof(float);
   KLLM_SEQ_DISPATCH(dtype, (qk_prepare_kernel<AT><<<T, 32 * warps, smem, s>>>(a, rope, qkvg, qnorm_w, knorm_w, eps, tok_seq,
-                                                                             tok_pos, static_cast<AT*>(q), gates, kv)));
+                                                                             tok_pos, static_cast<AT*>(q), gates, kv, blend)));
   return done();
 }
 

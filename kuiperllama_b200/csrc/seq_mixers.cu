@@ -47,15 +47,19 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 __device__ __forceinline__ float sigmoidf(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float siluf(float z) { return z / (1.0f + expf(-z)); }
 
-// Rotary position: coordinate i < dims / 2 pairs with i + dims / 2; angle = pos * base^(-2 i / dims); coordinates past
-// `dims` pass unchanged.  v: the vector before rotation.
-__device__ __forceinline__ float rotated(const float* v, int i, int dims, float base, int pos) {
+// Rotary position: coordinate i < dims / 2 pairs with i + dims / 2 (or 2i with 2i + 1); angle of pair i = pos * freq[i], or
+// pos * base^(-2 i / dims) without a table; coordinates past `dims` pass unchanged.  v: the vector before rotation.
+__device__ __forceinline__ float rotated(const LatentShape& a, const float* v, int i, int pos) {
+  const int dims = a.rope_dims;
   if (i >= dims) return v[i];
   const int half = dims >> 1;
-  const int j = i < half ? i : i - half;
-  const float freq = exp2f(-2.0f * static_cast<float>(j) / static_cast<float>(dims) * log2f(base));
+  const bool pairs = a.rope_pairing == KLLM_SEQ_ROPE_PAIRS;
+  const int j = pairs ? i >> 1 : (i < half ? i : i - half);
+  const float freq =
+      a.rope_freq ? __ldg(a.rope_freq + j) : exp2f(-2.0f * static_cast<float>(j) / static_cast<float>(dims) * log2f(a.rope_base));
   float sn, cs;
   sincosf(static_cast<float>(pos) * freq, &sn, &cs);
+  if (pairs) return (i & 1) == 0 ? v[i] * cs - v[i + 1] * sn : v[i] * cs + v[i - 1] * sn;
   return i < half ? v[i] * cs - v[i + half] * sn : v[i] * cs + v[i - half] * sn;
 }
 
@@ -67,15 +71,17 @@ __global__ void latent_prepare_kernel(LatentShape a, const float* __restrict__ p
                                       PagedKV kv, AT* __restrict__ c_rows, float* __restrict__ kr_rows) {
   __shared__ float red[33];
   const int t = blockIdx.x;
-  const int stride = a.q_rank + a.kv_rank + a.rot_dim + a.heads;
+  const int stride = latent_proj_rows(a);
   const float* row = proj + static_cast<size_t>(t) * stride;
   const int seq = tok_seq[t], pos = tok_pos[t];
   float ss = 0.f;
-  for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) ss += row[i] * row[i];
-  const float rq = 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(a.q_rank) + eps);
-  for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x)
-    cq[static_cast<size_t>(t) * a.q_rank + i] = from_f<AT>(row[i] * rq * q_norm_w[i]);
-  const float* c = row + a.q_rank;
+  if (a.q_rank > 0) {
+    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x) ss += row[i] * row[i];
+    const float rq = 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(a.q_rank) + eps);
+    for (int i = threadIdx.x; i < a.q_rank; i += blockDim.x)
+      cq[static_cast<size_t>(t) * a.q_rank + i] = from_f<AT>(row[i] * rq * q_norm_w[i]);
+  }
+  const float* c = row + latent_query_rows(a);
   ss = 0.f;
   for (int i = threadIdx.x; i < a.kv_rank; i += blockDim.x) ss += c[i] * c[i];
   const float rc = 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(a.kv_rank) + eps);
@@ -88,12 +94,12 @@ __global__ void latent_prepare_kernel(LatentShape a, const float* __restrict__ p
   }
   const float* kr = c + a.kv_rank;
   for (int i = threadIdx.x; i < a.rot_dim; i += blockDim.x) {
-    const float v = rotated(kr, i, a.rope_dims, a.rope_base, pos);
+    const float v = rotated(a, kr, i, pos);
     dst[a.kv_rank + i] = from_f<AT>(v);
     if (kr_rows) kr_rows[static_cast<size_t>(t) * a.rot_dim + i] = v;
   }
   const float* g = kr + a.rot_dim;
-  for (int h = threadIdx.x; h < a.heads; h += blockDim.x) gates[static_cast<size_t>(t) * a.heads + h] = sigmoidf(g[h]);
+  for (int h = threadIdx.x; a.gate && h < a.heads; h += blockDim.x) gates[static_cast<size_t>(t) * a.heads + h] = sigmoidf(g[h]);
 }
 
 // ---- latent attention: queries into the latent space --------------------------------------------------------------------
@@ -101,14 +107,14 @@ __global__ void latent_prepare_kernel(LatentShape a, const float* __restrict__ p
 // rows d of the head's block of W_uk (coalesced over r) with the tokens' queries in shared memory.
 constexpr int kAbsTokens = 16;
 template <typename AT>
-__global__ void latent_absorb_kernel(LatentShape a, const float* __restrict__ q, const AT* __restrict__ w_uk,
+__global__ void latent_absorb_kernel(LatentShape a, const float* __restrict__ q, int q_row, const AT* __restrict__ w_uk,
                                      const int32_t* __restrict__ tok_pos, float* __restrict__ qa, int T) {
   extern __shared__ float qs[];  // [kAbsTokens][dim + rot_dim]
   const int h = blockIdx.y, t0 = blockIdx.x * kAbsTokens;
   const int n = min(kAbsTokens, T - t0);
   const int dq = a.dim + a.rot_dim, dl = a.kv_rank + a.rot_dim;
   for (int i = threadIdx.x; i < n * dq; i += blockDim.x)
-    qs[i] = q[(static_cast<size_t>(t0 + i / dq) * a.heads + h) * dq + i % dq];
+    qs[i] = q[static_cast<size_t>(t0 + i / dq) * q_row + h * dq + i % dq];
   __syncthreads();
   const AT* w = w_uk + static_cast<size_t>(h) * a.dim * a.kv_rank;
   // blockIdx.z: a slice of the latent coordinates, so that a step of few tokens still spreads over many SMs
@@ -130,38 +136,38 @@ __global__ void latent_absorb_kernel(LatentShape a, const float* __restrict__ q,
   for (int i = threadIdx.x; i < n * a.rot_dim; i += blockDim.x) {
     const int j = i / a.rot_dim, c = i % a.rot_dim;
     qa[(static_cast<size_t>(t0 + j) * a.heads + h) * dl + a.kv_rank + c] =
-        rotated(qs + j * dq + a.dim, c, a.rope_dims, a.rope_base, tok_pos[t0 + j]);
+        rotated(a, qs + j * dq + a.dim, c, tok_pos[t0 + j]);
   }
 }
 
 // ---- latent attention with per-head keys and values (prompt steps on the tensor cores) ---------------------------------------
 // q [T, heads, dim + rot_dim] fp32 -> the same in the compute type with the rotated part rotated
 template <typename AT>
-__global__ void latent_pack_q_kernel(LatentShape a, const float* __restrict__ q, const int32_t* __restrict__ tok_pos,
+__global__ void latent_pack_q_kernel(LatentShape a, const float* __restrict__ q, int q_row, const int32_t* __restrict__ tok_pos,
                                      AT* __restrict__ out) {
   const int t = blockIdx.x, dq = a.dim + a.rot_dim;
   const int pos = tok_pos[t];
-  const float* row = q + static_cast<size_t>(t) * a.heads * dq;
+  const float* row = q + static_cast<size_t>(t) * q_row;
   for (int i = threadIdx.x; i < a.heads * dq; i += blockDim.x) {
     const int h = i / dq, d = i % dq;
-    const float v = d < a.dim ? row[i] : rotated(row + h * dq + a.dim, d - a.dim, a.rope_dims, a.rope_base, pos);
+    const float v = d < a.dim ? row[i] : rotated(a, row + h * dq + a.dim, d - a.dim, pos);
     out[static_cast<size_t>(t) * a.heads * dq + i] = from_f<AT>(v);
   }
 }
 // kp [T, heads * dim] fp32 (W_uk c) and kr [T, rot_dim] (rotated, shared by the heads) -> k [T, heads, dim + rot_dim];
 // vp [T, heads * vdim] fp32 (W_uv c) -> v, both in the compute type
 template <typename AT>
-__global__ void latent_pack_kv_kernel(LatentShape a, const float* __restrict__ kp, const float* __restrict__ kr,
-                                      const float* __restrict__ vp, AT* __restrict__ k, AT* __restrict__ v) {
+__global__ void latent_pack_kv_kernel(LatentShape a, const float* __restrict__ kp, int kp_row, const float* __restrict__ kr,
+                                      const float* __restrict__ vp, int vp_row, AT* __restrict__ k, AT* __restrict__ v) {
   const int t = blockIdx.x, dq = a.dim + a.rot_dim;
   for (int i = threadIdx.x; i < a.heads * dq; i += blockDim.x) {
     const int h = i / dq, d = i % dq;
-    const float x = d < a.dim ? kp[(static_cast<size_t>(t) * a.heads + h) * a.dim + d]
+    const float x = d < a.dim ? kp[static_cast<size_t>(t) * kp_row + h * a.dim + d]
                               : kr[static_cast<size_t>(t) * a.rot_dim + d - a.dim];
     k[static_cast<size_t>(t) * a.heads * dq + i] = from_f<AT>(x);
   }
   for (int i = threadIdx.x; i < a.heads * a.vdim; i += blockDim.x)
-    v[static_cast<size_t>(t) * a.heads * a.vdim + i] = from_f<AT>(vp[static_cast<size_t>(t) * a.heads * a.vdim + i]);
+    v[static_cast<size_t>(t) * a.heads * a.vdim + i] = from_f<AT>(vp[static_cast<size_t>(t) * vp_row + i]);
 }
 
 // ---- latent attention: weighted sums of latents -> per-head values ---------------------------------------------------------
@@ -589,27 +595,27 @@ int launch_latent_prepare(int dtype, const LatentShape& a, const float* proj, co
   return done();
 }
 
-int launch_latent_pack_q(int dtype, const LatentShape& a, const float* q, const int32_t* tok_pos, void* out, int T,
+int launch_latent_pack_q(int dtype, const LatentShape& a, const float* q, int q_row, const int32_t* tok_pos, void* out, int T,
                          cudaStream_t s) {
-  KLLM_SEQ_DISPATCH(dtype, (latent_pack_q_kernel<AT><<<T, 256, 0, s>>>(a, q, tok_pos, static_cast<AT*>(out))));
+  KLLM_SEQ_DISPATCH(dtype, (latent_pack_q_kernel<AT><<<T, 256, 0, s>>>(a, q, q_row, tok_pos, static_cast<AT*>(out))));
   return done();
 }
 
-int launch_latent_pack_kv(int dtype, const LatentShape& a, const float* kp, const float* kr, const float* vp, void* k, void* v,
-                          int T, cudaStream_t s) {
-  KLLM_SEQ_DISPATCH(dtype, (latent_pack_kv_kernel<AT><<<T, 256, 0, s>>>(a, kp, kr, vp, static_cast<AT*>(k),
+int launch_latent_pack_kv(int dtype, const LatentShape& a, const float* kp, int kp_row, const float* kr, const float* vp,
+                          int vp_row, void* k, void* v, int T, cudaStream_t s) {
+  KLLM_SEQ_DISPATCH(dtype, (latent_pack_kv_kernel<AT><<<T, 256, 0, s>>>(a, kp, kp_row, kr, vp, vp_row, static_cast<AT*>(k),
                                                                        static_cast<AT*>(v))));
   return done();
 }
 
-int launch_latent_absorb(int dtype, const LatentShape& a, const float* q, const void* w_uk, const int32_t* tok_pos, float* qa,
-                         int T, cudaStream_t s) {
+int launch_latent_absorb(int dtype, const LatentShape& a, const float* q, int q_row, const void* w_uk, const int32_t* tok_pos,
+                         float* qa, int T, cudaStream_t s) {
   const size_t smem = static_cast<size_t>(kAbsTokens) * (a.dim + a.rot_dim) * sizeof(float);
   if (smem > 48 * 1024) return KLLM_E_UNSUPPORTED;
   // few tokens: 64 latent coordinates per CTA; many tokens: the whole latent (the queries are staged once per CTA)
   const int threads = T <= kAbsTokens ? 64 : (a.kv_rank <= 64 ? 64 : (a.kv_rank <= 128 ? 128 : 256));
   const dim3 grid((T + kAbsTokens - 1) / kAbsTokens, a.heads, (a.kv_rank + threads - 1) / threads);
-  KLLM_SEQ_DISPATCH(dtype, (latent_absorb_kernel<AT><<<grid, threads, smem, s>>>(a, q, static_cast<const AT*>(w_uk), tok_pos,
+  KLLM_SEQ_DISPATCH(dtype, (latent_absorb_kernel<AT><<<grid, threads, smem, s>>>(a, q, q_row, static_cast<const AT*>(w_uk), tok_pos,
                                                                                 qa, T)));
   return done();
 }

@@ -51,6 +51,10 @@ class Value {
     if (d != std::floor(d)) throw std::runtime_error("json: not an integer");
     return static_cast<long long>(d);
   }
+  bool as_bool() const {
+    if (kind != Kind::kBool) throw std::runtime_error("json: not true or false");
+    return boolean;
+  }
   const std::string& as_string() const {
     if (kind != Kind::kString) throw std::runtime_error("json: not a string");
     return string;

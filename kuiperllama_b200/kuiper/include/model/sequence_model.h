@@ -105,6 +105,7 @@ class SequenceModel : public base::NoCopyable {
   float logit_scale_ = 1.0f;
   float embed_scale_ = 1.0f;    // the embedding rows are multiplied by it
   float logit_softcap_ = 0.0f;  // logits <- cap * tanh(logits / cap); 0: none
+  int32_t streams_ = 0;         // residual streams joined by hyper-connections; 0: one plain residual
 
  private:
   SequenceOptions options_;

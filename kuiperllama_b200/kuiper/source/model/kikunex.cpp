@@ -30,6 +30,7 @@ base::Status KikunexModel::build_latent(const json::Value& c, const SafetensorsF
   a->q_rank = get_int(c, "q_rank"), a->kv_rank = get_int(c, "kv_rank");
   a->scale = static_cast<float>(c.at("scale").as_number());
   a->window = present(c, "mask") ? get_int(c.at("mask"), "size") : 0;
+  a->gate = KLLM_SEQ_GATE_HEAD, a->rope_pairing = KLLM_SEQ_ROPE_HALVES, a->rope_freq = nullptr;
   a->rope_dims = 0, a->rope_base = 1.f;
   if (present(c, "rot")) {
     a->rope_dims = get_int(c.at("rot"), "dims");

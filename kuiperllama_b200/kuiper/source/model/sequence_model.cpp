@@ -160,7 +160,7 @@ base::Status SequenceModel::init(const std::string& dir, const SequenceOptions& 
   d.run_vectors = run_vectors_, d.embed = embed_, d.final_norm = final_norm_, d.head = head_;
   d.max_tokens = options.max_tokens, d.max_seqs = options.max_seqs, d.page_tokens = options.page_tokens;
   d.embed_norm = embed_norm_, d.logit_scale = logit_scale_;
-  d.embed_scale = embed_scale_, d.logit_softcap = logit_softcap_;
+  d.embed_scale = embed_scale_, d.logit_softcap = logit_softcap_, d.streams = streams_;
   d.run_embed = run_embed_.size() == run_layer_.size() ? run_embed_.data() : nullptr;
   return engine_status(kllm_seq_create(&d, nullptr, &engine_), "kllm_seq_create");
 }

@@ -28,7 +28,7 @@ class Attention(ctypes.Structure):
                 ("in_bias", c_void_p), ("conv_taps", c_int32), ("conv_w", c_void_p), ("rope_dims", c_int32),
                 ("rope_base", c_float), ("rope_pairing", c_int32), ("values_are_keys", c_int32),
                 ("rope_freq", c_void_p), ("rope_mag", c_float), ("differential", c_int32), ("diff_lambda", c_float),
-                ("diff_out_scale", c_float)]
+                ("diff_out_scale", c_float), ("out_bias", c_void_p), ("v_blend", c_int32), ("v_lambda", c_float)]
 
 
 class Moe(ctypes.Structure):
@@ -44,7 +44,8 @@ class Latent(ctypes.Structure):
     _fields_ = [("heads", c_int32), ("dim", c_int32), ("rot_dim", c_int32), ("vdim", c_int32), ("q_rank", c_int32),
                 ("kv_rank", c_int32), ("scale", c_float), ("window", c_int32), ("rope_dims", c_int32),
                 ("rope_base", c_float), ("w_in", c_void_p), ("q_norm_w", c_void_p), ("kv_norm_w", c_void_p),
-                ("w_uq", c_void_p), ("w_uk", c_void_p), ("w_uv", c_void_p), ("sink", c_void_p), ("w_out", c_void_p)]
+                ("w_uq", c_void_p), ("w_uk", c_void_p), ("w_uv", c_void_p), ("sink", c_void_p), ("w_out", c_void_p),
+                ("gate", c_int32), ("rope_pairing", c_int32), ("rope_freq", c_void_p)]
 
 
 class Linear(ctypes.Structure):
@@ -76,12 +77,17 @@ class Ssd(ctypes.Structure):
                 ("dt_bias", c_void_p), ("a", c_void_p), ("d", c_void_p), ("out_norm_w", c_void_p), ("w_out", c_void_p)]
 
 
+class Hyper(ctypes.Structure):
+    # named fields of kllm_seq_hyper; `in` is a keyword
+    _fields_ = [("in_w", c_void_p), ("out", c_void_p), ("mix", c_void_p)]
+
+
 class Layer(ctypes.Structure):
     _fields_ = [("mixer_kind", c_int32), ("ff_kind", c_int32), ("pre_mixer", Norm), ("post_mixer", Norm),
                 ("pre_ff", Norm), ("post_ff", Norm), ("attn", Attention), ("moe", Moe), ("shift", c_void_p),
                 ("latent", Latent), ("linear", Linear), ("dense", Dense), ("ssm", Ssm), ("delta", Delta),
                 ("mixer2_kind", c_int32), ("mixer_scale", c_float), ("mixer2_scale", c_float), ("parallel_ff", c_int32),
-                ("ssd", Ssd), ("mixer_out_norm", Norm), ("mixer2_out_norm", Norm)]
+                ("ssd", Ssd), ("mixer_out_norm", Norm), ("mixer2_out_norm", Norm), ("hyper_mixer", Hyper), ("hyper_ff", Hyper)]
 
 
 class Desc(ctypes.Structure):
@@ -90,7 +96,7 @@ class Desc(ctypes.Structure):
                 ("run_add", POINTER(c_int32)), ("run_vectors", c_void_p), ("embed", c_void_p), ("final_norm", Norm),
                 ("head", c_void_p), ("max_tokens", c_int32), ("max_seqs", c_int32), ("page_tokens", c_int32),
                 ("embed_norm", Norm), ("run_embed", POINTER(c_int32)), ("logit_scale", c_float), ("embed_scale", c_float),
-                ("logit_softcap", c_float)]
+                ("logit_softcap", c_float), ("streams", c_int32)]
 
 
 class SeqError(RuntimeError):
@@ -523,7 +529,7 @@ class SeqEngine:
                 L.mixer_kind = 2
                 a = L.latent
                 a.heads, a.dim, a.rot_dim, a.vdim = shape.heads, shape.dim, shape.rot_dim, shape.vdim
-                a.q_rank, a.kv_rank, a.window = shape.q_rank, shape.kv_rank, shape.window
+                a.q_rank, a.kv_rank, a.window, a.gate = shape.q_rank, shape.kv_rank, shape.window, 1
                 a.scale, a.rope_dims, a.rope_base = (shape.dim + shape.rot_dim) ** -0.5, shape.rot_dim, 10000.0
                 a.w_in = rnd(shape.n_in("latent"), W, std=W ** -0.5).data_ptr()
                 a.q_norm_w = f32(shape.q_rank, std=0.05, mean=1.0).data_ptr()
