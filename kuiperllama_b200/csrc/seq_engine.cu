@@ -230,7 +230,8 @@ static int validate_mixer(const kllm_seq_layer& L, int kind) {
     if (a.differential && (a.sink || a.values_are_keys)) return KLLM_E_UNSUPPORTED;
     if (a.v_blend < 0 || a.v_blend > KLLM_SEQ_VBLEND_MIX) return KLLM_E_INVALID;
     if (a.differential && a.qk_norm == KLLM_SEQ_QKNORM_PROJECTION) return KLLM_E_UNSUPPORTED;
-    if (a.vdim > 256 || a.dim > 512) return KLLM_E_UNSUPPORTED;
+    if ((a.differential || a.values_are_keys) && (a.vdim > 256 || a.dim > 512)) return KLLM_E_UNSUPPORTED;
+    if (a.dim > 4096 || a.vdim > 4096) return KLLM_E_UNSUPPORTED;
     if (a.window < 0 || a.keep_first < 0 || a.softcap < 0.f || a.conv_taps < 0 || a.rope_dims < 0 || a.rope_dims > a.dim ||
         (a.rope_dims & 1) || (a.rope_dims > 0 && a.rope_base <= 0.f))
       return KLLM_E_INVALID;
@@ -245,8 +246,8 @@ static int validate_mixer(const kllm_seq_layer& L, int kind) {
         !a.w_in || (a.q_rank > 0 && (!a.q_norm_w || !a.w_uq)) || !a.kv_norm_w || !a.w_uk || !a.w_uv || !a.w_out)
       return KLLM_E_INVALID;
     if (a.gate != KLLM_SEQ_GATE_NONE && a.gate != KLLM_SEQ_GATE_HEAD) return KLLM_E_UNSUPPORTED;
-    // the latent is the value of the paged attention kernel, latent + rotated part its key
-    if (a.kv_rank > 256 || a.kv_rank + a.rot_dim > 512) return KLLM_E_UNSUPPORTED;
+    // the kernels around the latent stage a block of tokens' queries and latent sums in shared memory
+    if (a.kv_rank > 768 || a.dim + a.rot_dim > 768) return KLLM_E_UNSUPPORTED;
   } else if (kind == KLLM_SEQ_MIXER_LINEAR) {
     const kllm_seq_linear& a = L.linear;
     if (a.heads <= 0 || a.dim <= 0 || a.vdim <= 0 || !a.decay || !a.w_in || !a.out_norm_w || !a.w_out) return KLLM_E_INVALID;

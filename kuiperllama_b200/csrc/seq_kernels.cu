@@ -795,6 +795,67 @@ attention_kernel(AttnShape a, const void* __restrict__ q_, PagedKV kv, const int
   }
 }
 
+// Heads too wide for the tiles above (more than 4 * kAttnKeys value or kAttnMaxDim key coordinates, or tiles that exceed shared
+// memory): a CTA per (token, query head, split of the keys).  A warp scores a key with its lanes over the coordinates; the
+// output accumulates in shared memory, each thread owning its columns.  Same partial results as attention_kernel.
+template <typename AT>
+__global__ void __launch_bounds__(kAttnThreads)
+attention_wide_kernel(AttnShape a, const void* __restrict__ q_, PagedKV kv, const int32_t* __restrict__ tok_seq,
+                      const int32_t* __restrict__ tok_pos, int splits, float* __restrict__ ws) {
+  extern __shared__ float sm[];
+  float* qs = sm;            // [dim], scaled
+  float* acc = qs + a.dim;   // [vdim]
+  float* sc = acc + a.vdim;  // [keys]
+  const int t = blockIdx.x / a.heads, h = blockIdx.x % a.heads, split = blockIdx.y;
+  const int g = h / (a.heads / a.kv_heads), gv = g / v_share_of(a);
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const int pos = tok_pos[t];
+  for (int d = tid; d < a.dim; d += kAttnThreads) {
+    const size_t i = static_cast<size_t>(blockIdx.x) * a.dim + d;
+    qs[d] = (a.q_f32 ? static_cast<const float*>(q_)[i] : to_f(static_cast<const AT*>(q_)[i])) * a.scale;
+  }
+  for (int d = tid; d < a.vdim; d += kAttnThreads) acc[d] = 0.f;
+  // visible keys: [0, kept) and [lo, pos], cut into `splits` parts
+  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
+  const int kept = a.window > 0 ? min(lo, a.keep_first) : 0;
+  const int n_keys = kept + pos - lo + 1, per = (n_keys + splits - 1) / splits;
+  const int first = split * per, last = min(n_keys, first + per);
+  const int32_t* table = kv.table + static_cast<size_t>(tok_seq[t]) * kv.table_stride;
+  auto slot_of = [&](int i) {
+    const int kj = i < kept ? i : lo + i - kept;
+    return static_cast<size_t>(table[kj / kv.page]) * kv.page + kj % kv.page;
+  };
+  const AT* kbase = static_cast<const AT*>(kv.k) + static_cast<size_t>(g) * a.dim;
+  const AT* vbase = static_cast<const AT*>(kv.v) + static_cast<size_t>(gv) * a.vdim;
+  float m = -INFINITY, l = 0.f;
+  for (int k0 = first; k0 < last; k0 += kAttnKeys) {
+    const int n = min(kAttnKeys, last - k0);
+    __syncthreads();
+    for (int j = warp; j < n; j += kAttnThreads / 32) {
+      const AT* kr = kbase + slot_of(k0 + j) * kv.k_row;
+      float s = 0.f;
+      for (int d = lane; d < a.dim; d += 32) s = fmaf(qs[d], to_f(kr[d]), s);
+      s = warp_sum(s);
+      if (lane == 0) sc[j] = a.softcap > 0.f ? a.softcap * tanhf(s / a.softcap) : s;
+    }
+    __syncthreads();
+    float m_new = m;
+    for (int j = 0; j < n; ++j) m_new = fmaxf(m_new, sc[j]);
+    const float alpha = expf(m - m_new);
+    l *= alpha;
+    for (int j = 0; j < n; ++j) l += expf(sc[j] - m_new);
+    for (int d = tid; d < a.vdim; d += kAttnThreads) {
+      float o = acc[d] * alpha;
+      for (int j = 0; j < n; ++j) o = fmaf(expf(sc[j] - m_new), to_f(vbase[slot_of(k0 + j) * kv.v_row + d]), o);
+      acc[d] = o;
+    }
+    m = m_new;
+  }
+  float* p = ws + (static_cast<size_t>(blockIdx.x) * splits + split) * (a.vdim + 2);
+  if (tid == 0) p[0] = m, p[1] = l;
+  for (int d = tid; d < a.vdim; d += kAttnThreads) p[2 + d] = acc[d];
+}
+
 template <typename AT>
 __global__ void attention_merge_kernel(int heads, int vdim, int splits, const float* __restrict__ ws,
                                        const float* __restrict__ gates, int gate_kind, const float* __restrict__ sink,
@@ -1145,7 +1206,7 @@ int launch_qk_prepare(int dtype, const AttnShape& a, const RopeArgs& rope_, cons
   RopeArgs rope = rope_;
   if (rope.mag == 0.f) rope.mag = 1.0f;
   if (rope.dims < 0 || (rope.dims & 1) || rope.dims > a.dim || a.kv_heads % v_share_of(a) || a.heads % v_share_of(a) ||
-      a.dim > 512)
+      a.dim > 4096)
     return KLLM_E_INVALID;
   // a warp per head: few tokens get as many warps as there are query and key heads (at most 16: the kernel's registers
   // do not fit 1024 threads); a head's row lives in shared memory
@@ -1180,14 +1241,19 @@ size_t attention_workspace_bytes(const AttnShape& a, int T, int splits) {
   return static_cast<size_t>(T) * a.heads * splits * (a.vdim + 2) * sizeof(float);
 }
 
+static size_t attention_tile_bytes(const AttnShape& a) {
+  const int dq = (a.dim + 3) & ~3;
+  return (static_cast<size_t>(kAttnRows) * dq + static_cast<size_t>(kAttnKeys) * (dq + 1) +
+          static_cast<size_t>(kAttnKeys) * a.vdim + kAttnRows * kAttnKeys + 3 * kAttnRows) * sizeof(float);
+}
+constexpr size_t kAttnMaxTileBytes = 220 * 1024;
+constexpr int kAttnMaxDim = 512;
+
 template <typename AT, int C, bool SPARSE, int RS>
 static int launch_attention_cs(const AttnShape& a, const void* q, const PagedKV& kv, int n_entries,
                               const int32_t* ent_first, const int32_t* ent_count, const int32_t* ent_seq,
                               const int32_t* ent_pos0, int max_count, int splits, float* ws, cudaStream_t s) {
-  const int dq = (a.dim + 3) & ~3;
-  const size_t smem = (static_cast<size_t>(kAttnRows) * dq + static_cast<size_t>(kAttnKeys) * (dq + 1) +
-                       static_cast<size_t>(kAttnKeys) * a.vdim + kAttnRows * kAttnKeys + 3 * kAttnRows) * sizeof(float);
-  if (smem > 220 * 1024) return KLLM_E_UNSUPPORTED;
+  const size_t smem = attention_tile_bytes(a);
   static size_t configured = 0;
   if (smem > 48 * 1024 && smem > configured) {
     const cudaError_t e = cudaFuncSetAttribute(attention_kernel<AT, C, SPARSE, RS>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -1220,15 +1286,20 @@ int launch_attention(int dtype, const AttnShape& a, const void* q, const float* 
                      int n_entries, const int32_t* ent_first, const int32_t* ent_count, const int32_t* ent_seq,
                      const int32_t* ent_pos0, int max_count, int max_ctx, int splits, float* ws, void* out, int T,
                      const int32_t* tok_seq, const int32_t* tok_pos, cudaStream_t s) {
-  (void)max_ctx, (void)tok_seq, (void)tok_pos;
-  if (a.kv_heads <= 0 || a.heads % a.kv_heads != 0 || a.vdim > 4 * kAttnKeys || a.dim <= 0 || a.vdim <= 0)
-    return KLLM_E_UNSUPPORTED;
+  (void)max_ctx;
+  if (a.kv_heads <= 0 || a.heads % a.kv_heads != 0 || a.dim <= 0 || a.vdim <= 0) return KLLM_E_UNSUPPORTED;
   const int C = (a.vdim + kAttnKeys - 1) / kAttnKeys;
   int rc = 0;
   if (attention_mma_usable(dtype, a, max_count)) {
     rc = launch_attention_mma(a, q, gates, kv, n_entries, ent_first, ent_count, ent_seq, ent_pos0, max_count, splits, ws,
                               out, s);
     if (rc || (splits == 1 && !a.no_merge)) return rc;
+  } else if (a.vdim > 4 * kAttnKeys || a.dim > kAttnMaxDim || attention_tile_bytes(a) > kAttnMaxTileBytes) {
+    const size_t smem = (static_cast<size_t>(a.dim) + a.vdim + kAttnKeys) * sizeof(float);
+    if (smem > 48 * 1024 || kv.table == nullptr) return KLLM_E_UNSUPPORTED;
+    const dim3 grid(T * a.heads, splits);
+    KLLM_SEQ_DISPATCH(dtype, (attention_wide_kernel<AT><<<grid, kAttnThreads, smem, s>>>(a, q, kv, tok_seq, tok_pos, splits, ws)));
+    rc = done();
   } else {
 #define KLLM_ATTN_C(c)                                                                                              \
   KLLM_SEQ_DISPATCH(dtype, (rc = launch_attention_c<AT, c>(a, q, kv, n_entries, ent_first, ent_count, ent_seq, ent_pos0, \
