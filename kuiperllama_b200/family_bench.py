@@ -1,7 +1,8 @@
-"""`bench.py --family fobolorn | kikunex | vurazen | bukuvik`: prefill and decode throughput of a batched family (sequence-batch
+"""`bench.py --family fobolorn | kikunex | vurazen | bukuvik | bifazen`: prefill and decode throughput of a batched family (sequence-batch
 engine) at sizes that resemble a real model's layers, random weights, beside the closest existing model at equal width,
 heads, active feed-forward size and number of layer runs: Fobolorn beside the Llama family of the single-sequence decoder,
-Kikunex beside Fobolorn, Vurazen beside Kikunex, Bukuvik beside Vurazen.
+Kikunex beside Fobolorn, Vurazen beside Kikunex, Bukuvik beside Vurazen, Bifazen beside Kikunex (its latent attention) and
+Fobolorn (its attention).
 
 What is timed.  A step is the call a server makes: kllm_seq_step() with token ids in host memory and the greedy ids
 read back to host memory, blocking -- so every number here is end to end.  Between timed steps a buffer larger than
@@ -19,7 +20,7 @@ import statistics
 import time
 from pathlib import Path
 
-from .sequence import BF16, BukuvikShape, F32, FobolornShape, KikunexShape, SeqEngine, VurazenShape, load_seq_library
+from .sequence import BF16, BifazenShape, BukuvikShape, F32, FobolornShape, KikunexShape, SeqEngine, VurazenShape, load_seq_library
 
 ROOT = Path(__file__).resolve().parent.parent
 
@@ -72,6 +73,67 @@ BUKUVIK_SIZES = {
     "debug": BukuvikShape("bukuvik-debug", 256, 4096, _bp(512)[:3], 4, 2, 32, 64, 96, 16, 4, 2, 32, 32, 64, 2, 16,
                           8, 32, 16, 2, 2),
 }
+
+
+def _fp(kinds, ff):
+    return tuple(({"L": "latent", "A": "attention"}[k], ff) for k in kinds)
+
+
+def _bifazen(name, width, vocab, kinds, ff, *rest):
+    return BifazenShape(name, width, vocab, _fp(kinds, ff), 4, *rest)
+
+
+# the sizes of KIKUNEX_SIZES: same width, heads, head sizes, key/value rank and window in the latent layers, the heads of
+# SIZES over 4 key heads (window 512) in the others; six layers, none looped; gated feed-forwards of 2 x width; 4 streams
+_BIFAZEN_DIMS = {"s": (1024, 32000, 2048, 16, 64, 32, 64, 128, 512, 16, 4, 64, 64, 512),
+                 "m": (2048, 32000, 4096, 16, 128, 64, 128, 256, 512, 16, 4, 128, 128, 512),
+                 "debug": (256, 4096, 512, 4, 32, 16, 32, 64, 96, 4, 2, 32, 32, 96)}
+
+
+def bifazen_shape(size, kinds, tag):
+    w, v, ff, *rest = _BIFAZEN_DIMS[size]
+    return _bifazen(f"bifazen-{size}{tag}", w, v, kinds, ff, *rest)
+
+
+def kikunex_latent_shape(size):
+    """Kikunex with latent attention and a dense feed-forward in all of six layers."""
+    import dataclasses
+    base = KIKUNEX_SIZES[size]
+    return dataclasses.replace(base, name=base.name + "-latent", pattern=(("latent", "dense"),) * 6, loop=(0, 0, 1))
+
+
+def bifazen_costs(shape, prompt_len):
+    """FLOPs of a prompt step by phase class of the engine's profile (latents in their per-head form, whose expansion is
+    counted with the preparation, where the engine runs it)."""
+    W, T = shape.width, prompt_len
+
+    def pairs(window):
+        win = min(window, T)
+        return T * win - win * (win - 1) / 2
+    n_lat = sum(1 for m, _ in shape.pattern if m == "latent")
+    n_att = shape.layers - n_lat
+    return {"in_proj": 2 * T * W * sum(shape.n_in(m) for m, _ in shape.pattern),
+            "qk_prepare": 2 * T * sum(shape.expand_elems(m) for m, _ in shape.pattern),
+            "attention": n_lat * 2 * pairs(shape.window) * shape.heads * (shape.dim + shape.rot_dim + shape.vdim) +
+            n_att * 2 * pairs(shape.a_window) * shape.a_heads * (shape.a_dim + shape.a_vdim),
+            "out_proj": 2 * T * W * sum(shape.n_out(m) for m, _ in shape.pattern),
+            "experts": 2 * T * sum(3 * (f or 0) * W for _, f in shape.pattern),
+            "head": 2 * shape.vocab * W}
+
+
+def bifazen_decode_bytes(shape, B, ctx, es):
+    """Bytes a decode step must move, by phase class: weights once per step, the windows' latents, keys and values, the
+    streams (read and written once per sublayer)."""
+    W = shape.width
+    n_sub = sum(2 if f else 1 for _, f in shape.pattern)
+    return {"norm": n_sub * B * W * (2 * shape.streams + 1) * 4,
+            "in_proj": sum(shape.n_in(m) for m, _ in shape.pattern) * W * es,
+            "out_proj": sum(shape.n_out(m) for m, _ in shape.pattern) * W * es,
+            "qk_prepare": sum(shape.heads * shape.dim * shape.kv_rank for m, _ in shape.pattern if m == "latent") * es,
+            "experts": sum(3 * (f or 0) * W for _, f in shape.pattern) * es,
+            "attention": shape.state_bytes_per_step(B, ctx, es) +
+            sum(shape.heads * shape.vdim * shape.kv_rank for m, _ in shape.pattern if m == "latent") * es,
+            "head": shape.vocab * W * es}
 
 
 def bukuvik_costs(shape, prompt_len):
@@ -252,7 +314,8 @@ def bench_engine(torch, shape, dtype, prompt_len, ctx, batches, steps, warm, flu
     kiku = isinstance(shape, KikunexShape)
     vura = isinstance(shape, VurazenShape)
     buku = isinstance(shape, BukuvikShape)
-    phase_flops = (bukuvik_costs if buku else vurazen_costs if vura else kikunex_costs if kiku else
+    bifa = isinstance(shape, BifazenShape)
+    phase_flops = (bifazen_costs if bifa else bukuvik_costs if buku else vurazen_costs if vura else kikunex_costs if kiku else
                    fobolorn_costs)(shape, prompt_len)
     flops = sum(phase_flops.values())
     out["prefill"] = {"tokens": prompt_len, "tok_s": prompt_len / sec, "ms": sec * 1e3, "launches": launches,
@@ -283,9 +346,10 @@ def bench_engine(torch, shape, dtype, prompt_len, ctx, batches, steps, warm, flu
         # bytes a step must read: the active weights (distinct experts per token, an upper bound when tokens share
         # experts) and the cached keys / values
         W = shape.width
-        if vura or buku:
-            phase_bytes = (bukuvik_decode_bytes if buku else vurazen_decode_bytes)(shape, B, ctx, es)
-            bytes_step = shape.weight_elems_per_step(B) * es + phase_bytes["attention"]
+        if vura or buku or bifa:
+            phase_bytes = (bifazen_decode_bytes if bifa else bukuvik_decode_bytes if buku else vurazen_decode_bytes)(shape, B, ctx, es)
+            bytes_step = shape.weight_elems_per_step(B) * es + \
+                (shape.state_bytes_per_step(B, ctx, es) + phase_bytes["norm"] if bifa else phase_bytes["attention"])
             out["decode"][str(B)] = {
                 "batch": B, "context": ctx, "tok_s": B / sec, "ms_per_step": sec * 1e3, "launches": launches,
                 "bytes_per_step": bytes_step, "frac_of_hbm_peak": bytes_step / sec / 1e9 / hbm, "phase_ms": ph,
@@ -435,6 +499,8 @@ def run(args, emit):
         return run_vurazen(args, emit, torch, sizes, steps, warm, flush, hbm, tf, src)
     if args.family == "bukuvik":
         return run_bukuvik(args, emit, torch, sizes, steps, warm, flush, hbm, tf, src)
+    if args.family == "bifazen":
+        return run_bifazen(args, emit, torch, sizes, steps, warm, flush, hbm, tf, src)
     line = {"family": "fobolorn", "metric": "prefill_and_decode_tokens_per_s", "n_gpus": 1, "steps": steps, "warmup": warm,
             "data": "synthetic", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": src},
             "config": {"l2": "a 256 MiB buffer is written between timed steps", "timing": "wall clock around the blocking "
@@ -510,5 +576,27 @@ def run_bukuvik(args, emit, torch, sizes, steps, warm, flush, hbm, tf, src):
             entry["bukuvik"].append(bench_engine(torch, shape, dtype, prompt, ctx, [1, 8], steps, warm, flush, hbm, tf))
             entry["closest"].append(bench_engine(torch, close, dtype, prompt, ctx, [1, 8], steps, warm, flush, hbm, tf))
         entry["closest_model"] = close.name
+        line["sizes"][name] = entry
+    emit(line)
+
+
+def run_bifazen(args, emit, torch, sizes, steps, warm, flush, hbm, tf, src):
+    """Bifazen (its two kinds of layer mixed, and each kind alone) beside its closest existing models on the same engine at
+    equal width, heads and layer runs: Kikunex with latent attention and dense feed-forwards only, and Fobolorn for the
+    grouped-query attention."""
+    line = {"family": "bifazen", "metric": "prefill_and_decode_tokens_per_s", "n_gpus": 1, "steps": steps, "warmup": warm,
+            "data": "synthetic", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": src},
+            "config": {"l2": "a 256 MiB buffer is written between timed steps", "timing": "wall clock around the blocking "
+                       "step call (token ids from host memory, greedy ids back to host memory); phases by CUDA events"},
+            "sizes": {}}
+    for name in sizes:
+        ctx, prompt = (256, 512) if name == "debug" else (1024, 2048)
+        shapes = {"bifazen": bifazen_shape(name, "LALLAL", ""), "bifazen_latent": bifazen_shape(name, "LLLLLL", "-latent"),
+                  "kikunex_latent": kikunex_latent_shape(name), "bifazen_attention": bifazen_shape(name, "AAAAAA", "-attention"),
+                  "fobolorn": SIZES[name]}
+        entry = {"shape": dict(shapes["bifazen"].__dict__)}
+        for key, shape in shapes.items():
+            entry[key] = [bench_engine(torch, shape, dtype, prompt, ctx, [1, 8], steps, warm, flush, hbm, tf)
+                          for dtype in (BF16, F32)]
         line["sizes"][name] = entry
     emit(line)

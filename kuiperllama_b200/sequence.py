@@ -2,7 +2,7 @@
 device memory, the engine and every kernel are the product library's.  Like the rest of this package it has no
 fallback: without libkllm_seq.so (or libkllm_b200.so, which carries the same symbols) it raises.
 
-`FobolornShape` / `KikunexShape` / `VurazenShape` / `BukuvikShape` + `SeqEngine` build a random-weight model of a family directly in device memory
+`FobolornShape` / `KikunexShape` / `VurazenShape` / `BukuvikShape` / `BifazenShape` + `SeqEngine` build a random-weight model of a family directly in device memory
 (no model folder), for measurements at sizes that resemble a real model's layers.
 """
 from __future__ import annotations
@@ -429,8 +429,69 @@ class BukuvikShape:
         return total
 
 
+@dataclass
+class BifazenShape:
+    """A Bifazen model: `pattern` lists the layers ("latent" | "attention", feed-forward size or None)."""
+    name: str
+    width: int
+    vocab: int
+    pattern: tuple
+    streams: int
+    heads: int           # latent attention
+    dim: int
+    rot_dim: int
+    vdim: int
+    kv_rank: int
+    window: int
+    a_heads: int         # attention normed over whole projections
+    a_kv_heads: int
+    a_dim: int
+    a_vdim: int
+    a_window: int
+    eps: float = 1e-5
+
+    @property
+    def layers(self):
+        return len(self.pattern)
+
+    @property
+    def runs(self):
+        return len(self.pattern)
+
+    def run_order(self):
+        return [(i, -1, 0) for i in range(self.layers)]
+
+    def n_in(self, kind):
+        if kind == "latent":
+            return self.heads * (self.dim + self.rot_dim) + self.kv_rank + self.rot_dim
+        return (self.a_heads + self.a_kv_heads) * self.a_dim + self.a_kv_heads * self.a_vdim + self.a_heads
+
+    def n_out(self, kind):
+        return self.heads * self.vdim if kind == "latent" else self.a_heads * self.a_vdim
+
+    def expand_elems(self, kind):
+        return self.heads * (self.dim + self.vdim) * self.kv_rank if kind == "latent" else 0
+
+    def weight_elems_per_step(self, batch):
+        return self.vocab * self.width + sum((self.n_in(m) + self.n_out(m)) * self.width + self.expand_elems(m) +
+                                             3 * (f or 0) * self.width for m, f in self.pattern)
+
+    def flops_per_token(self):
+        return 2 * self.weight_elems_per_step(1)
+
+    def state_bytes_per_step(self, batch, ctx, es):
+        """Cache a decode step reads: the windows' latents, keys and values."""
+        total = 0
+        for m, _ in self.pattern:
+            if m == "latent":
+                total += batch * min(ctx, self.window) * (self.kv_rank + self.rot_dim) * es
+            else:
+                total += batch * min(ctx, self.a_window) * self.a_kv_heads * (self.a_dim + self.a_vdim) * es
+        return total
+
+
 class SeqEngine:
-    """A random-weight model (Fobolorn, Kikunex, Vurazen or Bukuvik, by the shape's class) in device memory behind the engine's C-ABI."""
+    """A random-weight model (Fobolorn, Kikunex, Vurazen, Bukuvik or Bifazen, by the shape's class) in device memory behind the engine's C-ABI."""
 
     def __init__(self, shape, dtype=BF16, max_tokens=4096, max_seqs=16, page=0, seed=1):
         import torch
@@ -445,6 +506,9 @@ class SeqEngine:
             return
         if isinstance(shape, BukuvikShape):
             self._init_bukuvik(shape, dtype, max_tokens, max_seqs, page, seed)
+            return
+        if isinstance(shape, BifazenShape):
+            self._init_bifazen(shape, dtype, max_tokens, max_seqs, page, seed)
             return
         td = torch.bfloat16 if dtype == BF16 else torch.float32
         g = torch.Generator(device="cuda").manual_seed(seed)
@@ -793,6 +857,89 @@ class SeqEngine:
         d.final_norm = out_norm()
         d.head = d.embed  # the classifier is the embedding table
         d.embed_scale = W ** 0.5
+        d.max_tokens, d.max_seqs, d.page_tokens = max_tokens, max_seqs, page
+        self._desc = (d, layers, run_layer, run_add, run_embed)
+        self.handle = c_void_p()
+        torch.cuda.synchronize()
+        _check(self.lib, self.lib.kllm_seq_create(ctypes.byref(d), None, ctypes.byref(self.handle)), "kllm_seq_create")
+
+    def _init_bifazen(self, shape, dtype, max_tokens, max_seqs, page, seed):
+        torch = self.torch
+        td = torch.bfloat16 if dtype == BF16 else torch.float32
+        g = torch.Generator(device="cuda").manual_seed(seed)
+        keep = self._keep = []
+        W, S = shape.width, shape.streams
+
+        def rnd(*dims, std, t=td, mean=0.0):
+            x = (torch.randn(*dims, device="cuda", generator=g) * std + mean).to(t).contiguous()
+            keep.append(x)
+            return x
+
+        def f32(*dims, std, mean=0.0):
+            return rnd(*dims, std=std, t=torch.float32, mean=mean)
+
+        def norm():
+            return Norm(f32(W, std=0.1, mean=1.0).data_ptr(), None, 1)
+
+        def hyper():
+            mix = 0.8 * torch.eye(S, device="cuda") + 0.2 / S + 0.05 * torch.randn(S, S, device="cuda", generator=g)
+            mix = mix.contiguous()
+            keep.append(mix)
+            return Hyper(f32(S, std=0.3 / S, mean=1.0 / S).data_ptr(), f32(S, std=0.3, mean=0.6).data_ptr(), mix.data_ptr())
+
+        layers = (Layer * shape.layers)()
+        source = False
+        for L, (mix, ff) in zip(layers, shape.pattern):
+            L.pre_mixer = norm()
+            L.mixer_scale = L.mixer2_scale = 1.0
+            if S > 0:
+                L.hyper_mixer, L.hyper_ff = hyper(), hyper()
+            if mix == "latent":
+                L.mixer_kind = 2
+                a = L.latent
+                a.heads, a.dim, a.rot_dim, a.vdim = shape.heads, shape.dim, shape.rot_dim, shape.vdim
+                a.q_rank, a.kv_rank, a.window, a.gate = 0, shape.kv_rank, shape.window, 0
+                a.scale, a.rope_dims, a.rope_base, a.rope_pairing = (shape.dim + shape.rot_dim) ** -0.5, shape.rot_dim, 1e5, 1
+                freq = torch.tensor([1e5 ** (-2.0 * i / shape.rot_dim) for i in range(shape.rot_dim // 2)], device="cuda")
+                keep.append(freq)
+                a.rope_freq = freq.data_ptr()
+                a.w_in = rnd(shape.n_in("latent"), W, std=W ** -0.5).data_ptr()
+                a.kv_norm_w = f32(shape.kv_rank, std=0.05, mean=1.0).data_ptr()
+                ukv = rnd(shape.heads * (shape.dim + shape.vdim), shape.kv_rank, std=shape.kv_rank ** -0.5)
+                a.w_uk = ukv.data_ptr()
+                a.w_uv = ukv.data_ptr() + shape.heads * shape.dim * shape.kv_rank * ukv.element_size()
+                a.w_out = rnd(W, shape.heads * shape.vdim, std=(shape.heads * shape.vdim) ** -0.5).data_ptr()
+            else:
+                L.mixer_kind = 1
+                a = L.attn
+                a.heads, a.kv_heads, a.dim, a.vdim = shape.a_heads, shape.a_kv_heads, shape.a_dim, shape.a_vdim
+                a.scale, a.window, a.qk_norm, a.gate = shape.a_dim ** -0.5, shape.a_window, 3, 1
+                a.w_in = rnd(shape.n_in("attention"), W, std=W ** -0.5).data_ptr()
+                a.in_bias = f32(shape.n_in("attention"), std=0.1).data_ptr()
+                a.out_bias = f32(W, std=0.1).data_ptr()
+                a.q_norm_w = f32(shape.a_heads * shape.a_dim, std=0.1, mean=1.0).data_ptr()
+                a.k_norm_w = f32(shape.a_kv_heads * shape.a_dim, std=0.1, mean=1.0).data_ptr()
+                a.w_out = rnd(W, shape.a_heads * shape.a_vdim, std=(shape.a_heads * shape.a_vdim) ** -0.5).data_ptr()
+                a.v_blend, a.v_lambda = (2 if source else 1), 0.4
+                source = True
+            L.ff_kind = 2 if ff else 0
+            if ff:
+                L.pre_ff = norm()
+                d = L.dense
+                d.ff, d.act = ff, 5
+                d.up = rnd(2 * ff, W, std=W ** -0.5).data_ptr()
+                d.down = rnd(W, ff, std=ff ** -0.5).data_ptr()
+        order = shape.run_order()
+        run_layer = (c_int32 * len(order))(*[i for i, _, _ in order])
+        run_add = (c_int32 * len(order))(*[p for _, p, _ in order])
+        run_embed = (c_int32 * len(order))(*[x for _, _, x in order])
+        d = Desc()
+        d.dtype, d.width, d.vocab, d.norm_eps, d.streams = dtype, W, shape.vocab, shape.eps, S
+        d.n_layers, d.layers = shape.layers, layers
+        d.n_runs, d.run_layer, d.run_add, d.run_embed = len(order), run_layer, run_add, run_embed
+        d.embed = rnd(shape.vocab, W, std=1.0).data_ptr()
+        d.final_norm = norm()
+        d.head = d.embed  # the classifier is the embedding table
         d.max_tokens, d.max_seqs, d.page_tokens = max_tokens, max_seqs, page
         self._desc = (d, layers, run_layer, run_add, run_embed)
         self.handle = c_void_p()
