@@ -18,6 +18,11 @@
 //
 // With one split the kernel divides by the sum, applies the output gate and writes the compute type; with several it
 // leaves (max, sum, unnormalised output) per split for attention_merge_kernel, like the fp32 kernel.
+// attention_rows_mma_kernel (second half of this file) serves steps of FEW rows per key head -- single-token steps, short
+// portions -- and fp32 queries (an attention through a latent: all query heads share one key row per token): one CTA takes
+// at most 16 (token, query head) rows, one split of the keys, and walks tiles of 32 keys.  The queries enter as two bf16
+// terms when they are fp32, the weights always do, so both products see their left operand to about 2^-17.
+//
 // tcgen05 is not used here: at head sizes of 64..128 a 64-row tile is small against TMEM's 128-lane accumulators, and
 // the softmax between the two products wants the scores in registers anyway.
 #include <cuda_bf16.h>
@@ -25,6 +30,7 @@
 
 #include <cmath>
 #include <cstdint>
+#include <cstdlib>
 
 #include "seq_engine.h"
 
@@ -356,7 +362,276 @@ int launch_mma(const AttnShape& a, const void* q, const float* gates, const Page
   return cuda_rc(cudaGetLastError());
 }
 
+// ---- few rows ---------------------------------------------------------------------------------------------------------------
+// Grid: x = 16-row tile, y = (entry, key/value head), z = split.  Four warps.  Scores: a warp takes 8 keys of the tile
+// against all 16 rows.  Softmax: a warp takes 4 rows, a lane per key.  Output: the 8-column blocks are dealt out to the
+// warps in turn (NBW per warp).  Values that are the head of the key row (SAME) are read from the key tile.
+constexpr int kFewRows = 16, kFewKeys = 32, kFewThreads = 128, kFewWarps = 4;
+
+struct FewLayout {  // shared memory, in bytes from its start
+  int ldk, ldv, dimp;
+  size_t k, v, q_hi, q_lo, s, p_hi, p_lo, stats, total;
+};
+__host__ __device__ inline FewLayout few_layout(const AttnShape& a, bool same, bool q_f32) {
+  FewLayout L;
+  L.dimp = (a.dim + 15) & ~15;
+  L.ldk = L.dimp + 8, L.ldv = same ? L.ldk : ((a.vdim + 15) & ~15) + 8;
+  size_t at = 0;
+  L.k = at, at += 2 * static_cast<size_t>(kFewKeys) * L.ldk * 2;
+  L.v = same ? L.k : at, at += same ? 0 : 2 * static_cast<size_t>(kFewKeys) * L.ldv * 2;
+  L.q_hi = at, at += static_cast<size_t>(kFewRows) * L.ldk * 2;
+  L.q_lo = at, at += q_f32 ? static_cast<size_t>(kFewRows) * L.ldk * 2 : 0;
+  L.s = at, at += kFewRows * (kFewKeys + 1) * 4;
+  at = (at + 15) & ~static_cast<size_t>(15);
+  L.p_hi = at, at += kFewRows * (kFewKeys + 8) * 2;
+  L.p_lo = at, at += kFewRows * (kFewKeys + 8) * 2;
+  L.stats = at, at += 3 * kFewRows * 4;
+  L.total = at;
+  return L;
+}
+
+template <int NBW, bool SAME, bool QF32>
+__global__ void __launch_bounds__(kFewThreads)
+attention_rows_mma_kernel(AttnShape a, const void* __restrict__ q_, PagedKV kv, const int32_t* __restrict__ ent_first,
+                          const int32_t* __restrict__ ent_count, const int32_t* __restrict__ ent_seq,
+                          const int32_t* __restrict__ ent_pos0, int splits, float* __restrict__ ws) {
+  const int e = blockIdx.y / a.kv_heads, g = blockIdx.y % a.kv_heads, split = blockIdx.z;
+  const int gv = g / v_share_of(a);
+  const int rep = a.heads / a.kv_heads, dim = a.dim, vdim = a.vdim;
+  const int count = ent_count[e], first = ent_first[e], pos0 = ent_pos0[e];
+  const int n_rows = count * rep, r0 = blockIdx.x * kFewRows;
+  if (r0 >= n_rows) return;
+  const int rows_here = min(kFewRows, n_rows - r0);
+  const int32_t* table = kv.table + static_cast<size_t>(ent_seq[e]) * kv.table_stride;
+  const int pmax = pos0 + (r0 + rows_here - 1) / rep;
+  const int n_tiles = pmax / kFewKeys + 1;
+  const int window = a.window, keep_first = window > 0 ? a.keep_first : 0;
+  const int tile_first = window > 0 ? max(0, pos0 + r0 / rep - window + 1) / kFewKeys : 0;
+  // this CTA's list of tiles: those with kept first positions ahead of the window, then the window's; cut into splits
+  const int keep_tiles = min(tile_first, (keep_first + kFewKeys - 1) / kFewKeys);
+  const int list_n = keep_tiles + n_tiles - tile_first;
+  const int per = (list_n + splits - 1) / splits;
+  const int tile_lo = split * per, tile_hi = min(list_n, tile_lo + per);
+  auto tile_of = [&](int li) { return li < keep_tiles ? li : tile_first + (li - keep_tiles); };
+
+  extern __shared__ __align__(16) unsigned char few_sm[];
+  const FewLayout L = few_layout(a, SAME, QF32);
+  const int ldk = L.ldk, ldv = L.ldv;
+  __nv_bfloat16* q_hi = reinterpret_cast<__nv_bfloat16*>(few_sm + L.q_hi);
+  __nv_bfloat16* q_lo = reinterpret_cast<__nv_bfloat16*>(few_sm + L.q_lo);
+  float* Ss = reinterpret_cast<float*>(few_sm + L.s);                          // [rows][keys + 1]
+  __nv_bfloat16* p_hi = reinterpret_cast<__nv_bfloat16*>(few_sm + L.p_hi);     // [rows][keys + 8]
+  __nv_bfloat16* p_lo = reinterpret_cast<__nv_bfloat16*>(few_sm + L.p_lo);
+  float* m_s = reinterpret_cast<float*>(few_sm + L.stats);
+  float* l_s = m_s + kFewRows;
+  float* al_s = l_s + kFewRows;
+  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
+  const uint32_t base = static_cast<uint32_t>(__cvta_generic_to_shared(few_sm));
+  const uint32_t k_addr = base + static_cast<uint32_t>(L.k), v_addr = base + static_cast<uint32_t>(L.v);
+
+  const __nv_bfloat16* kbase = static_cast<const __nv_bfloat16*>(kv.k) + static_cast<size_t>(g) * dim;
+  const __nv_bfloat16* vbase = static_cast<const __nv_bfloat16*>(kv.v) + static_cast<size_t>(gv) * vdim;
+  const int kc = L.dimp / 8, vc = SAME ? 0 : (ldv - 8) / 8;
+  auto load_tile = [&](int tile, int stage) {  // four threads per key: one page lookup per thread
+    const int j = tid >> 2, kj = tile * kFewKeys + j;
+    const bool valid = kj <= pmax;
+    const size_t slot = valid ? static_cast<size_t>(table[kj / kv.page]) * kv.page + kj % kv.page : 0;
+    const __nv_bfloat16 *kr = kbase + slot * kv.k_row, *vr = vbase + slot * kv.v_row;
+    const uint32_t kd = k_addr + ((stage * kFewKeys + j) * ldk) * 2, vd = v_addr + ((stage * kFewKeys + j) * ldv) * 2;
+    for (int c = tid & 3; c < kc; c += 4) {
+      const bool in = valid && c * 8 < dim;
+      cp_async16(kd + c * 16, in ? kr + c * 8 : kbase, in);
+    }
+    for (int c = tid & 3; c < vc; c += 4) {
+      const bool in = valid && c * 8 < vdim;
+      cp_async16(vd + c * 16, in ? vr + c * 8 : vbase, in);
+    }
+    cp_async_commit();
+  };
+  if (tile_lo < tile_hi) load_tile(tile_of(tile_lo), 0);
+
+  // the queries, two neighbouring coordinates at a time (dim is even); rows and coordinates that do not exist are zero
+  const int half = L.dimp / 2;
+  for (int i = tid; i < kFewRows * half; i += kFewThreads) {
+    const int r = i / half, d = (i % half) * 2;
+    float x = 0.f, y = 0.f;
+    if (r < rows_here && d < dim) {
+      const int rr = r0 + r;
+      const size_t qi = (static_cast<size_t>(first + rr / rep) * a.heads + g * rep + rr % rep) * dim + d;
+      if (QF32) {
+        const float2 v = *reinterpret_cast<const float2*>(static_cast<const float*>(q_) + qi);
+        x = v.x, y = v.y;
+      } else {
+        const __nv_bfloat162 v = *reinterpret_cast<const __nv_bfloat162*>(static_cast<const __nv_bfloat16*>(q_) + qi);
+        x = __low2float(v), y = __high2float(v);
+      }
+    }
+    uint32_t hi, lo;
+    split_pack(x, y, hi, lo);
+    *reinterpret_cast<uint32_t*>(q_hi + r * ldk + d) = hi;
+    if (QF32) *reinterpret_cast<uint32_t*>(q_lo + r * ldk + d) = lo;
+  }
+  if (tid < kFewRows) m_s[tid] = -INFINITY, l_s[tid] = 0.f;
+  float o[NBW][4];
+#pragma unroll
+  for (int i = 0; i < NBW; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  const int nb_all = (vdim + 7) / 8;
+  const int gq = lane >> 2, t4 = lane & 3;
+  // addresses of this lane's rows in the A fragments (16 x 16 tiles: rows lane % 16, columns + 8 for the upper lanes)
+  const uint32_t qh_addr = base + static_cast<uint32_t>(L.q_hi) + ((lane & 15) * ldk + (lane >> 4) * 8) * 2;
+  const uint32_t ql_addr = base + static_cast<uint32_t>(L.q_lo) + ((lane & 15) * ldk + (lane >> 4) * 8) * 2;
+  const uint32_t ph_addr = base + static_cast<uint32_t>(L.p_hi) + ((lane & 15) * (kFewKeys + 8) + (lane >> 4) * 8) * 2;
+  const uint32_t pl_addr = base + static_cast<uint32_t>(L.p_lo) + ((lane & 15) * (kFewKeys + 8) + (lane >> 4) * 8) * 2;
+
+  for (int li = tile_lo; li < tile_hi; ++li) {
+    const int tile = tile_of(li), stage = (li - tile_lo) & 1, k0 = tile * kFewKeys;
+    if (li + 1 < tile_hi) {
+      load_tile(tile_of(li + 1), stage ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    {  // scores of 8 keys: one ldmatrix.x2 brings the key fragments of a k-step (key row lane % 8, coordinates + 8 for lanes 8..15)
+      float s0[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
+      const uint32_t kt = k_addr + ((stage * kFewKeys + warp * 8 + (lane & 7)) * ldk + ((lane >> 3) & 1) * 8) * 2;
+#pragma unroll 4
+      for (int ks = 0; ks < L.dimp / 16; ++ks) {
+        uint32_t b0, b1, af[4];
+        asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(b0), "=r"(b1) : "r"(kt + ks * 32));
+        ldmatrix_x4(qh_addr + ks * 32, af[0], af[1], af[2], af[3]);
+        mma_bf16(s0, af, b0, b1);
+        if (QF32) {
+          ldmatrix_x4(ql_addr + ks * 32, af[0], af[1], af[2], af[3]);
+          mma_bf16(s1, af, b0, b1);
+        }
+      }
+#pragma unroll
+      for (int c = 0; c < 4; ++c) {
+        const int r = gq + (c >> 1) * 8, j = warp * 8 + t4 * 2 + (c & 1), kj = k0 + j;
+        const int pr = pos0 + (r0 + r) / rep;
+        float sv = (s0[c] + s1[c]) * a.scale;
+        if (a.softcap > 0.f) sv = a.softcap * tanhf(sv / a.softcap);
+        const bool visible = r < rows_here && kj <= pr && (window == 0 || pr - kj < window || kj < keep_first);
+        Ss[r * (kFewKeys + 1) + j] = visible ? sv : -INFINITY;
+      }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int i = 0; i < kFewRows / kFewWarps; ++i) {
+      const int r = warp * (kFewRows / kFewWarps) + i;
+      const float sv = Ss[r * (kFewKeys + 1) + lane];
+      float mx = sv;
+#pragma unroll
+      for (int off = 16; off > 0; off >>= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, off));
+      const float m_old = m_s[r], m_new = fmaxf(m_old, mx);
+      float p = 0.f, alpha = 1.0f;
+      if (m_new > -INFINITY) p = expf(sv - m_new), alpha = expf(m_old - m_new);
+      float sum = p;
+#pragma unroll
+      for (int off = 16; off > 0; off >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, off);
+      const __nv_bfloat16 h = __float2bfloat16_rn(p);
+      p_hi[r * (kFewKeys + 8) + lane] = h;
+      p_lo[r * (kFewKeys + 8) + lane] = __float2bfloat16_rn(p - __bfloat162float(h));
+      __syncwarp();  // every lane has read m_s[r]
+      if (lane == 0) m_s[r] = m_new, l_s[r] = l_s[r] * alpha + sum, al_s[r] = alpha;
+    }
+    __syncthreads();
+    {
+      const float aA = al_s[gq], aB = al_s[gq + 8];
+#pragma unroll
+      for (int i = 0; i < NBW; ++i) o[i][0] *= aA, o[i][1] *= aA, o[i][2] *= aB, o[i][3] *= aB;
+#pragma unroll
+      for (int kk = 0; kk < kFewKeys / 16; ++kk) {
+        uint32_t ph[4], pl[4];
+        ldmatrix_x4(ph_addr + kk * 32, ph[0], ph[1], ph[2], ph[3]);
+        ldmatrix_x4(pl_addr + kk * 32, pl[0], pl[1], pl[2], pl[3]);
+        const uint32_t vt = v_addr + ((stage * kFewKeys + kk * 16 + (lane & 15)) * ldv) * 2;
+#pragma unroll
+        for (int i = 0; i < NBW; ++i) {
+          const int nb = warp + i * kFewWarps;
+          if (nb < nb_all) {  // the same for the whole warp
+            uint32_t b0, b1;
+            asm volatile("ldmatrix.sync.aligned.m8n8.x2.trans.shared.b16 {%0,%1}, [%2];" : "=r"(b0), "=r"(b1) : "r"(vt + nb * 16));
+            mma_bf16(o[i], ph, b0, b1);
+            mma_bf16(o[i], pl, b0, b1);
+          }
+        }
+      }
+    }
+    __syncthreads();  // the stage is loaded again, the scores are written again
+  }
+  if (tile_lo >= tile_hi) __syncthreads();  // an empty split still writes its (empty) statistics
+  const int pstride = vdim + 2;
+#pragma unroll
+  for (int z = 0; z < 2; ++z) {
+    const int r = gq + z * 8;
+    if (r >= rows_here) continue;
+    const int rr = r0 + r;
+    float* p = ws + ((static_cast<size_t>(first + rr / rep) * a.heads + g * rep + rr % rep) * splits + split) * pstride;
+    if (warp == 0 && t4 == 0) p[0] = m_s[r], p[1] = l_s[r];
+#pragma unroll
+    for (int i = 0; i < NBW; ++i) {
+      const int col = (warp + i * kFewWarps) * 8 + t4 * 2;
+      if (col < vdim) *reinterpret_cast<float2*>(p + 2 + col) = make_float2(o[i][z * 2], o[i][z * 2 + 1]);
+    }
+  }
+}
+
+template <int NBW, bool SAME, bool QF32>
+int launch_few(const AttnShape& a, const void* q, const PagedKV& kv, int n_entries, const int32_t* ent_first,
+               const int32_t* ent_count, const int32_t* ent_seq, const int32_t* ent_pos0, int max_count, int splits, float* ws,
+               cudaStream_t s) {
+  const size_t smem = few_layout(a, SAME, QF32).total;
+  static size_t configured = 0;
+  if (smem > 48 * 1024 && smem > configured) {
+    const cudaError_t e = cudaFuncSetAttribute(attention_rows_mma_kernel<NBW, SAME, QF32>,
+                                               cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem));
+    if (e != cudaSuccess) return cuda_rc(e);
+    configured = smem;
+  }
+  const dim3 grid((max_count * (a.heads / a.kv_heads) + kFewRows - 1) / kFewRows, n_entries * a.kv_heads, splits);
+  if (grid.y > 65535u) return KLLM_E_UNSUPPORTED;
+  attention_rows_mma_kernel<NBW, SAME, QF32><<<grid, kFewThreads, smem, s>>>(a, q, kv, ent_first, ent_count, ent_seq, ent_pos0,
+                                                                            splits, ws);
+  count_launch();
+  return cuda_rc(cudaGetLastError());
+}
+
+inline bool values_in_keys(const AttnShape& a, const PagedKV& kv) {
+  return kv.v == kv.k && kv.v_row == kv.k_row && a.kv_heads == 1 && a.vdim <= a.dim;
+}
+
 }  // namespace
+
+bool attention_rows_mma_usable(int dtype, const AttnShape& a, const PagedKV& kv, int n_entries) {
+  static const bool off = [] { const char* e = getenv("KLLM_SEQ_ROWS_MMA"); return e != nullptr && e[0] == '0'; }();
+  if (off || dtype != KLLM_SEQ_BF16 || a.kv_heads <= 0 || a.heads % a.kv_heads || kv.table == nullptr) return false;
+  // 16-byte chunks of every key and value row
+  if (a.dim % 8 || a.vdim % 8 || kv.k_row % 8 || kv.v_row % 8 || a.vdim > 512) return false;
+  if (static_cast<long long>(n_entries) * a.kv_heads > 65535) return false;
+  return few_layout(a, values_in_keys(a, kv), a.q_f32 != 0).total <= 200 * 1024;
+}
+
+int launch_attention_rows_mma(const AttnShape& a, const void* q, const PagedKV& kv, int n_entries, const int32_t* ent_first,
+                              const int32_t* ent_count, const int32_t* ent_seq, const int32_t* ent_pos0, int max_count,
+                              int splits, float* ws, cudaStream_t s) {
+  const bool same = values_in_keys(a, kv);
+#define KLLM_FEW(N)                                                                                                              \
+  if (a.vdim <= N * kFewWarps * 8) {                                                                                              \
+    if (same)                                                                                                                     \
+      return a.q_f32 ? launch_few<N, true, true>(a, q, kv, n_entries, ent_first, ent_count, ent_seq, ent_pos0, max_count, splits, ws, s)   \
+                     : launch_few<N, true, false>(a, q, kv, n_entries, ent_first, ent_count, ent_seq, ent_pos0, max_count, splits, ws, s); \
+    return a.q_f32 ? launch_few<N, false, true>(a, q, kv, n_entries, ent_first, ent_count, ent_seq, ent_pos0, max_count, splits, ws, s)    \
+                   : launch_few<N, false, false>(a, q, kv, n_entries, ent_first, ent_count, ent_seq, ent_pos0, max_count, splits, ws, s);  \
+  }
+  KLLM_FEW(2)
+  KLLM_FEW(4)
+  KLLM_FEW(8)
+  KLLM_FEW(16)
+#undef KLLM_FEW
+  return KLLM_E_UNSUPPORTED;
+}
 
 bool attention_mma_usable(int dtype, const AttnShape& a, int max_count) {
   if (dtype != KLLM_SEQ_BF16 || a.kv_heads <= 0 || a.heads % a.kv_heads) return false;

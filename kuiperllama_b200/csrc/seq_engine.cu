@@ -816,13 +816,12 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
         RC(launch_latent_prepare(dtype, ls, proj, A.q_norm_w, A.kv_norm_w, d.norm_eps, d_seq, d_pos, e->q.p, gates, kv,
                                  e->lat_c.p, static_cast<float*>(e->lat_kr.p), T, st));
         RC(expand_queries());
-        RC(launch_latent_pack_q(dtype, ls, queries, q_row, d_pos, e->lat_q.p, T, st));
         float* kp = static_cast<float*>(e->lat_kp.p);
         RC(gemm(dtype, e->lat_c.p, A.w_uk, kp, T, A.kv_rank, stacked ? kn + vn : kn, st));
         if (!stacked) RC(gemm(dtype, e->lat_c.p, A.w_uv, static_cast<float*>(e->lat_vp.p), T, A.kv_rank, vn, st));
-        RC(launch_latent_pack_kv(dtype, ls, kp, stacked ? kn + vn : kn, static_cast<const float*>(e->lat_kr.p),
-                                 stacked ? kp + kn : static_cast<const float*>(e->lat_vp.p), stacked ? kn + vn : vn, e->lat_k.p,
-                                 e->lat_v.p, T, st));
+        RC(launch_latent_pack(dtype, ls, queries, q_row, kp, stacked ? kn + vn : kn, static_cast<const float*>(e->lat_kr.p),
+                              stacked ? kp + kn : static_cast<const float*>(e->lat_vp.p), stacked ? kn + vn : vn, d_pos,
+                              e->lat_q.p, e->lat_k.p, e->lat_v.p, T, st));
         e->mark(KLLM_SEQ_PHASE_QK_PREPARE);
         const PagedKV rows{e->lat_k.p, e->lat_v.p, nullptr, 0, 1, A.heads * dqk, A.heads * A.vdim};
         RC(launch_attention(dtype, eshape, e->lat_q.p, gates, rows, n_entries, d_first, d_count, d_eseq, d_pos0, max_count,

@@ -188,6 +188,13 @@ int launch_attention_mma(const AttnShape& a, const void* q, const float* gates, 
                          const int32_t* ent_first, const int32_t* ent_count, const int32_t* ent_seq,
                          const int32_t* ent_pos0, int max_count, int splits, float* ws, void* out, cudaStream_t s);
 
+// bf16 steps of few rows per key head, or with fp32 queries (head sizes that are multiples of 8): partial results of every
+// split in `ws`, like the split-key kernel.
+bool attention_rows_mma_usable(int dtype, const AttnShape& a, const PagedKV& kv, int n_entries);
+int launch_attention_rows_mma(const AttnShape& a, const void* q, const PagedKV& kv, int n_entries, const int32_t* ent_first,
+                              const int32_t* ent_count, const int32_t* ent_seq, const int32_t* ent_pos0, int max_count,
+                              int splits, float* ws, cudaStream_t s);
+
 // Token shift for steps with longer entries: out[t] = h[t] + (prev - h[t]) * mu in the compute type, prev = h[t - 1] inside
 // an entry, the sequence's state (zeros at position 0) for its first row; afterwards state[seq] = the entry's last h.
 int launch_token_shift(int dtype, const float* h, const float* mu, float* state, const int32_t* tok_seq,
@@ -215,13 +222,12 @@ int launch_latent_prepare(int dtype, const LatentShape& a, const float* proj, co
                           const PagedKV& kv, void* c_rows, float* kr_rows, int T, cudaStream_t s);
 // Prompt steps that start their sequences can expand the latents of the step into per-head keys and values and run the
 // tensor-core attention on them: c_rows [T, kv_rank] (compute type) and kr_rows [T, rot_dim] (fp32, rotated) are the
-// step's latents as rows (optional outputs of latent_prepare); pack_q rotates and converts the queries; pack_kv joins
-// W_uk c with the shared rotated part and converts W_uv c.
+// step's latents as rows (optional outputs of latent_prepare); latent_pack rotates and converts the queries, joins W_uk c with the
+// shared rotated part and converts W_uv c.
 // Row strides: q_row floats between two tokens' queries, kp_row / vp_row between two tokens' expanded keys / values.
-int launch_latent_pack_q(int dtype, const LatentShape& a, const float* q, int q_row, const int32_t* tok_pos, void* out, int T,
-                         cudaStream_t s);
-int launch_latent_pack_kv(int dtype, const LatentShape& a, const float* kp, int kp_row, const float* kr, const float* vp,
-                          int vp_row, void* k, void* v, int T, cudaStream_t s);
+int launch_latent_pack(int dtype, const LatentShape& a, const float* q, int q_row, const float* kp, int kp_row, const float* kr,
+                       const float* vp, int vp_row, const int32_t* tok_pos, void* q_out, void* k_out, void* v_out, int T,
+                       cudaStream_t s);
 // q [T, heads, dim + rot_dim] fp32 (rows q_row apart) -> qa [T, heads, kv_rank + rot_dim] fp32: W_uk(head)^T q_plain | rotated q_rot
 int launch_latent_absorb(int dtype, const LatentShape& a, const float* q, int q_row, const void* w_uk, const int32_t* tok_pos, float* qa,
                          int T, cudaStream_t s);

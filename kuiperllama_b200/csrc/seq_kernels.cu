@@ -16,6 +16,7 @@
 #include <cstdint>
 
 #include "seq_engine.h"
+#include "seq_merge.cuh"
 
 namespace kllm {
 namespace seq {
@@ -158,6 +159,20 @@ __global__ void embed_kernel(const AT* __restrict__ table, const int32_t* __rest
   __shared__ float red[33];
   const int t = blockIdx.x;
   const AT* row = table + static_cast<size_t>(tokens[t]) * width;
+  if (norm.w == nullptr && width % VecOf<AT>::N == 0 && (reinterpret_cast<uintptr_t>(table) & 15) == 0) {
+    constexpr int V = VecOf<AT>::N;
+    for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
+      float f[V];
+      VecOf<AT>::load(row + i, f);
+#pragma unroll
+      for (int j = 0; j < V; j += 4) {
+        const float4 v = make_float4(f[j] * scale, f[j + 1] * scale, f[j + 2] * scale, f[j + 3] * scale);
+        *reinterpret_cast<float4*>(x + static_cast<size_t>(t) * width + i + j) = v;
+        if (copy) *reinterpret_cast<float4*>(copy + static_cast<size_t>(t) * width + i + j) = v;
+      }
+    }
+    return;
+  }
   if (norm.w == nullptr) {
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
       const float v = to_f(row[i]) * scale;
@@ -551,6 +566,93 @@ __global__ void qk_prepare_kernel(AttnShape a, RopeArgs rope, const float* __res
     gates[static_cast<size_t>(t) * gn + i] = 1.0f / (1.0f + expf(-row[qn + kn + vn + i]));
 }
 
+// The same for heads without rotation, temperature or maps, normed over the whole projection or not at all: nothing is done
+// per head then, so the row is walked straight through, V columns at a time -- sums of squares, then query rows out, key and
+// value rows into the page, gates.
+template <typename AT, int V>
+__device__ __forceinline__ void put_cols(AT* dst, const float* v);
+template <> __device__ __forceinline__ void put_cols<float, 4>(float* dst, const float* v) {
+  *reinterpret_cast<float4*>(dst) = make_float4(v[0], v[1], v[2], v[3]);
+}
+template <> __device__ __forceinline__ void put_cols<__nv_bfloat16, 4>(__nv_bfloat16* dst, const float* v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
+  *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+template <> __device__ __forceinline__ void put_cols<float, 1>(float* dst, const float* v) { *dst = v[0]; }
+template <> __device__ __forceinline__ void put_cols<__nv_bfloat16, 1>(__nv_bfloat16* dst, const float* v) { *dst = __float2bfloat16_rn(v[0]); }
+template <int V> __device__ __forceinline__ void get_cols(const float* src, float* v);
+template <> __device__ __forceinline__ void get_cols<4>(const float* src, float* v) {
+  const float4 t = *reinterpret_cast<const float4*>(src);
+  v[0] = t.x, v[1] = t.y, v[2] = t.z, v[3] = t.w;
+}
+template <> __device__ __forceinline__ void get_cols<1>(const float* src, float* v) { v[0] = *src; }
+
+template <typename AT, int V>
+__global__ void qk_rows_kernel(AttnShape a, const float* __restrict__ qkvg, const float* __restrict__ qnorm_w,
+                               const float* __restrict__ knorm_w, float eps, const int32_t* __restrict__ tok_seq,
+                               const int32_t* __restrict__ tok_pos, AT* __restrict__ q, float* __restrict__ gates, PagedKV kv,
+                               ValueBlend blend) {
+  __shared__ float red[2][32];
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  const int qn = a.heads * a.dim, kn = a.kv_heads * a.dim, vn = a.kv_heads * a.vdim, gn = gate_floats(a);
+  const float* row = qkvg + static_cast<size_t>(t) * (qn + kn + vn + gn);
+  const int seq = tok_seq[t], pos = tok_pos[t];
+  AT* krow = page_row(static_cast<AT*>(kv.k), kv, seq, pos, a.kv_heads, a.dim);
+  AT* vrow = page_row(static_cast<AT*>(kv.v), kv, seq, pos, a.kv_heads, a.vdim);
+  AT* qrow = q + static_cast<size_t>(t) * qn;
+  const int step = blockDim.x * V;
+  const bool whole = a.qk_norm == KLLM_SEQ_QKNORM_PROJECTION;
+  float rq = 1.0f, rk = 1.0f;
+  if (whole) {
+    float sq = 0.f, sk = 0.f;
+    for (int i = threadIdx.x * V; i < qn + kn; i += step) {
+      float v[V];
+      get_cols<V>(row + i, v);
+      float ss = 0.f;
+#pragma unroll
+      for (int c = 0; c < V; ++c) ss = fmaf(v[c], v[c], ss);
+      if (i < qn) sq += ss;
+      else sk += ss;
+    }
+    sq = warp_sum(sq), sk = warp_sum(sk);
+    if (lane == 0) red[0][warp] = sq, red[1][warp] = sk;
+    __syncthreads();
+    sq = 0.f, sk = 0.f;
+    for (int i = 0; i < nw; ++i) sq += red[0][i], sk += red[1][i];
+    rq = 1.0f / sqrtf(sq / static_cast<float>(qn) + eps);
+    rk = 1.0f / sqrtf(sk / static_cast<float>(kn) + eps);
+  }
+  for (int i = threadIdx.x * V; i < qn + kn; i += step) {
+    float v[V];
+    get_cols<V>(row + i, v);
+    const bool is_q = i < qn;
+    const int j = is_q ? i : i - qn;
+    if (whole) {
+      float w[V];
+      get_cols<V>((is_q ? qnorm_w : knorm_w) + j, w);
+      const float r = is_q ? rq : rk;
+#pragma unroll
+      for (int c = 0; c < V; ++c) v[c] = v[c] * r * w[c];
+    }
+    put_cols<AT, V>((is_q ? qrow : krow) + j, v);
+  }
+  for (int i = threadIdx.x * V; i < vn; i += step) {
+    float v[V];
+    get_cols<V>(row + qn + kn + i, v);
+    float* kept = blend.rows + static_cast<size_t>(t) * vn + i;
+    if (blend.mode == KLLM_SEQ_VBLEND_SOURCE) put_cols<float, V>(kept, v);
+    if (blend.mode == KLLM_SEQ_VBLEND_MIX) {
+      float f[V];
+      get_cols<V>(kept, f);
+#pragma unroll
+      for (int c = 0; c < V; ++c) v[c] = (1.0f - blend.lambda) * v[c] + blend.lambda * f[c];
+    }
+    put_cols<AT, V>(vrow + i, v);
+  }
+  for (int i = threadIdx.x; i < gn; i += blockDim.x)
+    gates[static_cast<size_t>(t) * gn + i] = 1.0f / (1.0f + expf(-row[qn + kn + vn + i]));
+}
+
 // ---- attention ------------------------------------------------------------------------------------------------------
 // One CTA: one entry of the step, one key/value head g, kAttnRows consecutive rows (row r of the entry = token r / rep,
 // query head g * rep + r % rep, rep = heads / kv_heads), one split of the keys.  Tiles of kAttnKeys keys go through
@@ -856,31 +958,28 @@ attention_wide_kernel(AttnShape a, const void* __restrict__ q_, PagedKV kv, cons
   for (int d = tid; d < a.vdim; d += kAttnThreads) p[2 + d] = acc[d];
 }
 
+// One CTA per (token, head): the splits' weights (warp 0), the weighted sum of their outputs, the output gate, the conversion.
 template <typename AT>
 __global__ void attention_merge_kernel(int heads, int vdim, int splits, const float* __restrict__ ws,
                                        const float* __restrict__ gates, int gate_kind, const float* __restrict__ sink,
                                        int out_f32, void* __restrict__ out_) {
+  extern __shared__ float weight[];  // [splits]
   const size_t th = blockIdx.x;  // t * heads + h
   const int pstride = vdim + 2;
   const float* p = ws + th * splits * pstride;
-  float M = sink ? sink[th % heads] : -INFINITY;
-  for (int s = 0; s < splits; ++s) M = fmaxf(M, p[s * pstride]);
-  float L = sink ? expf(sink[th % heads] - M) : 0.f;
-  for (int s = 0; s < splits; ++s) {
-    const float m = p[s * pstride];
-    if (m > -INFINITY) L += p[s * pstride + 1] * expf(m - M);
-  }
   const bool per_element = gates != nullptr && gate_kind == KLLM_SEQ_GATE_ELEMENT;
+  MergeColumn col;
+  int d = threadIdx.x;
+  if (d < vdim) col.load(p, splits, pstride, d);
   const float head_gate = gates && !per_element ? gates[th] : 1.0f;
-  for (int d = threadIdx.x; d < vdim; d += blockDim.x) {
-    float o = 0.f;
-    for (int s = 0; s < splits; ++s) {
-      const float m = p[s * pstride];
-      if (m > -INFINITY) o += p[s * pstride + 2 + d] * expf(m - M);
-    }
-    const float gate = per_element ? gates[th * vdim + d] : head_gate;
-    if (out_f32) static_cast<float*>(out_)[th * vdim + d] = o / L * gate;
-    else static_cast<AT*>(out_)[th * vdim + d] = from_f<AT>(o / L * gate);
+  if (threadIdx.x < 32) split_weights(p, splits, pstride, sink != nullptr, sink ? sink[th % heads] : 0.f, weight);
+  __syncthreads();
+  while (d < vdim) {
+    const float o = col.join(p, splits, pstride, d, weight) * (per_element ? gates[th * vdim + d] : head_gate);
+    if (out_f32) static_cast<float*>(out_)[th * vdim + d] = o;
+    else static_cast<AT*>(out_)[th * vdim + d] = from_f<AT>(o);
+    d += blockDim.x;
+    if (d < vdim) col.load(p, splits, pstride, d);
   }
 }
 
@@ -1080,9 +1179,19 @@ __global__ void argmax_rows_kernel(const float* __restrict__ logits, int32_t* __
   const float* row = logits + static_cast<size_t>(blockIdx.x) * vocab;
   float best = -INFINITY;
   int idx = 0x7fffffff;
-  for (int i = threadIdx.x; i < vocab; i += blockDim.x) {
-    const float v = row[i];
-    if (v > best || (v == best && i < idx)) best = v, idx = i;
+  constexpr int U = 8;  // loads in flight per thread
+  for (int i0 = threadIdx.x; i0 < vocab; i0 += U * blockDim.x) {
+    float v[U];
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + u * blockDim.x;
+      v[u] = i < vocab ? row[i] : -INFINITY;
+    }
+#pragma unroll
+    for (int u = 0; u < U; ++u) {
+      const int i = i0 + u * blockDim.x;
+      if (i < vocab && (v[u] > best || (v[u] == best && i < idx))) best = v[u], idx = i;
+    }
   }
 #pragma unroll
   for (int o = 16; o > 0; o >>= 1) {
@@ -1208,6 +1317,19 @@ int launch_qk_prepare(int dtype, const AttnShape& a, const RopeArgs& rope_, cons
   if (rope.dims < 0 || (rope.dims & 1) || rope.dims > a.dim || a.kv_heads % v_share_of(a) || a.heads % v_share_of(a) ||
       a.dim > 4096)
     return KLLM_E_INVALID;
+  if (rope.dims == 0 && a.temp_every == 0 && v_share_of(a) == 1 &&
+      (a.qk_norm == KLLM_SEQ_QKNORM_PROJECTION || a.qk_norm == KLLM_SEQ_QKNORM_NONE)) {
+    const int qn = a.heads * a.dim, kn = a.kv_heads * a.dim, vn = a.kv_heads * a.vdim;
+    const bool vec = qn % 4 == 0 && kn % 4 == 0 && vn % 4 == 0 && gate_floats(a) % 4 == 0;
+    const int threads = T <= 16 ? 512 : 256;
+    if (vec)
+      KLLM_SEQ_DISPATCH(dtype, (qk_rows_kernel<AT, 4><<<T, threads, 0, s>>>(a, qkvg, qnorm_w, knorm_w, eps, tok_seq, tok_pos,
+                                                                            static_cast<AT*>(q), gates, kv, blend)));
+    else
+      KLLM_SEQ_DISPATCH(dtype, (qk_rows_kernel<AT, 1><<<T, threads, 0, s>>>(a, qkvg, qnorm_w, knorm_w, eps, tok_seq, tok_pos,
+                                                                            static_cast<AT*>(q), gates, kv, blend)));
+    return done();
+  }
   // a warp per head: few tokens get as many warps as there are query and key heads (at most 16: the kernel's registers
   // do not fit 1024 threads); a head's row lives in shared memory
   int warps = T <= 64 ? std::min(16, std::max(4, a.heads + a.kv_heads)) : 4;
@@ -1294,6 +1416,8 @@ int launch_attention(int dtype, const AttnShape& a, const void* q, const float* 
     rc = launch_attention_mma(a, q, gates, kv, n_entries, ent_first, ent_count, ent_seq, ent_pos0, max_count, splits, ws,
                               out, s);
     if (rc || (splits == 1 && !a.no_merge)) return rc;
+  } else if (attention_rows_mma_usable(dtype, a, kv, n_entries)) {
+    rc = launch_attention_rows_mma(a, q, kv, n_entries, ent_first, ent_count, ent_seq, ent_pos0, max_count, splits, ws, s);
   } else if (a.vdim > 4 * kAttnKeys || a.dim > kAttnMaxDim || attention_tile_bytes(a) > kAttnMaxTileBytes) {
     const size_t smem = (static_cast<size_t>(a.dim) + a.vdim + kAttnKeys) * sizeof(float);
     if (smem > 48 * 1024 || kv.table == nullptr) return KLLM_E_UNSUPPORTED;
@@ -1313,7 +1437,7 @@ int launch_attention(int dtype, const AttnShape& a, const void* q, const float* 
 #undef KLLM_ATTN_C
   }
   if (rc || a.no_merge) return rc;
-  KLLM_SEQ_DISPATCH(dtype, (attention_merge_kernel<AT><<<T * a.heads, 64, 0, s>>>(a.heads, a.vdim, splits, ws,
+  KLLM_SEQ_DISPATCH(dtype, (attention_merge_kernel<AT><<<T * a.heads, a.vdim <= 64 ? 64 : 128, splits * sizeof(float), s>>>(a.heads, a.vdim, splits, ws,
                                                                                  a.gate ? gates : nullptr, a.gate, a.sink,
                                                                                  a.out_f32, out)));
   return done();

@@ -16,6 +16,7 @@
 #include <cstdint>
 
 #include "seq_engine.h"
+#include "seq_merge.cuh"
 
 namespace kllm {
 namespace seq {
@@ -47,6 +48,64 @@ __device__ __forceinline__ float block_sum(float v, float* red) {
 __device__ __forceinline__ float sigmoidf(float z) { return 1.0f / (1.0f + expf(-z)); }
 __device__ __forceinline__ float siluf(float z) { return z / (1.0f + expf(-z)); }
 
+// V consecutive values of the compute type (16 bytes, or one value), widened to fp32
+template <typename AT> struct Wide;
+template <> struct Wide<float> {
+  static constexpr int N = 4;
+  template <int V> __device__ static __forceinline__ void load(const float* __restrict__ p, float* f) {
+    if constexpr (V == 4) {
+      const float4 v = __ldg(reinterpret_cast<const float4*>(p));
+      f[0] = v.x, f[1] = v.y, f[2] = v.z, f[3] = v.w;
+    } else {
+      f[0] = __ldg(p);
+    }
+  }
+};
+template <> struct Wide<__nv_bfloat16> {
+  static constexpr int N = 8;
+  template <int V> __device__ static __forceinline__ void load(const __nv_bfloat16* __restrict__ p, float* f) {
+    if constexpr (V == 8) {
+      const uint4 v = __ldg(reinterpret_cast<const uint4*>(p));
+      const uint32_t u[4] = {v.x, v.y, v.z, v.w};
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        f[2 * i] = __uint_as_float(u[i] << 16);
+        f[2 * i + 1] = __uint_as_float(u[i] & 0xffff0000u);
+      }
+    } else {
+      f[0] = to_f(p[0]);
+    }
+  }
+};
+
+// V consecutive fp32 values (16 bytes, or one)
+template <int V> __device__ __forceinline__ void get_floats(const float* p, float* f) {
+  if constexpr (V == 4) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    f[0] = v.x, f[1] = v.y, f[2] = v.z, f[3] = v.w;
+  } else {
+    f[0] = *p;
+  }
+}
+template <int V> __device__ __forceinline__ void put_values(float* p, const float* f) {
+  if constexpr (V == 4) *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]);
+  else *p = f[0];
+}
+template <int V> __device__ __forceinline__ void put_values(__nv_bfloat16* p, const float* f) {
+  if constexpr (V == 4) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+    *reinterpret_cast<uint2*>(p) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+  } else {
+    *p = __float2bfloat16_rn(f[0]);
+  }
+}
+
+// frequency of rotated pair j
+__device__ __forceinline__ float rope_frequency(const LatentShape& a, int j) {
+  if (a.rope_freq) return __ldg(a.rope_freq + j);
+  return exp2f(-2.0f * static_cast<float>(j) / static_cast<float>(a.rope_dims) * log2f(a.rope_base));
+}
+
 // Rotary position: coordinate i < dims / 2 pairs with i + dims / 2 (or 2i with 2i + 1); angle of pair i = pos * freq[i], or
 // pos * base^(-2 i / dims) without a table; coordinates past `dims` pass unchanged.  v: the vector before rotation.
 __device__ __forceinline__ float rotated(const LatentShape& a, const float* v, int i, int pos) {
@@ -55,10 +114,8 @@ __device__ __forceinline__ float rotated(const LatentShape& a, const float* v, i
   const int half = dims >> 1;
   const bool pairs = a.rope_pairing == KLLM_SEQ_ROPE_PAIRS;
   const int j = pairs ? i >> 1 : (i < half ? i : i - half);
-  const float freq =
-      a.rope_freq ? __ldg(a.rope_freq + j) : exp2f(-2.0f * static_cast<float>(j) / static_cast<float>(dims) * log2f(a.rope_base));
   float sn, cs;
-  sincosf(static_cast<float>(pos) * freq, &sn, &cs);
+  sincosf(static_cast<float>(pos) * rope_frequency(a, j), &sn, &cs);
   if (pairs) return (i & 1) == 0 ? v[i] * cs - v[i + 1] * sn : v[i] * cs + v[i - 1] * sn;
   return i < half ? v[i] * cs - v[i + half] * sn : v[i] * cs + v[i - half] * sn;
 }
@@ -140,34 +197,137 @@ __global__ void latent_absorb_kernel(LatentShape a, const float* __restrict__ q,
   }
 }
 
-// ---- latent attention with per-head keys and values (prompt steps on the tensor cores) ---------------------------------------
-// q [T, heads, dim + rot_dim] fp32 -> the same in the compute type with the rotated part rotated
-template <typename AT>
-__global__ void latent_pack_q_kernel(LatentShape a, const float* __restrict__ q, int q_row, const int32_t* __restrict__ tok_pos,
-                                     AT* __restrict__ out) {
-  const int t = blockIdx.x, dq = a.dim + a.rot_dim;
-  const int pos = tok_pos[t];
-  const float* row = q + static_cast<size_t>(t) * q_row;
-  for (int i = threadIdx.x; i < a.heads * dq; i += blockDim.x) {
-    const int h = i / dq, d = i % dq;
-    const float v = d < a.dim ? row[i] : rotated(a, row + h * dq + a.dim, d - a.dim, pos);
-    out[static_cast<size_t>(t) * a.heads * dq + i] = from_f<AT>(v);
+// The same for steps of at most NT <= 8 tokens: a CTA takes 64 latent coordinates of one head.  A lane owns 16 bytes of a row of
+// W_uk, groups of lanes and warps own different rows, and their sums meet at the end; the first rows are fetched before the
+// queries have arrived in shared memory.
+constexpr int kFewCols = 64, kFewWarps = 8, kFewAhead = 4;
+template <typename AT, int NT>
+__global__ void __launch_bounds__(kFewWarps * 32)
+latent_absorb_few_kernel(LatentShape a, const float* __restrict__ q, int q_row, const AT* __restrict__ w_uk,
+                         const int32_t* __restrict__ tok_pos, float* __restrict__ qa, int T) {
+  constexpr int V = Wide<AT>::N, LPR = kFewCols / V, RPW = 32 / LPR;  // values per lane, lanes per row, rows per warp
+  constexpr int kStep = kFewWarps * RPW;
+  extern __shared__ float qs[];                 // [NT][dim + rot_dim]
+  __shared__ float red[kFewWarps][NT][kFewCols];
+  const int h = blockIdx.x, c0 = blockIdx.y * kFewCols;
+  const int dq = a.dim + a.rot_dim, dl = a.kv_rank + a.rot_dim;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int col = c0 + (lane % LPR) * V, d0 = warp * RPW + lane / LPR;
+  const bool in = col < a.kv_rank;  // kv_rank is a multiple of V
+  const AT* w = w_uk + static_cast<size_t>(h) * a.dim * a.kv_rank + col;
+  float wf[kFewAhead][V];
+#pragma unroll
+  for (int k = 0; k < kFewAhead; ++k)
+    if (in && d0 + k * kStep < a.dim) Wide<AT>::template load<V>(w + static_cast<size_t>(d0 + k * kStep) * a.kv_rank, wf[k]);
+  for (int i = threadIdx.x; i < T * dq; i += blockDim.x) qs[i] = q[static_cast<size_t>(i / dq) * q_row + h * dq + i % dq];
+  __syncthreads();
+  float acc[NT][V];
+#pragma unroll
+  for (int t = 0; t < NT; ++t)
+#pragma unroll
+    for (int c = 0; c < V; ++c) acc[t][c] = 0.f;
+  if (in) {
+    for (int base = 0; base < a.dim; base += kFewAhead * kStep) {
+#pragma unroll
+      for (int k = 0; k < kFewAhead; ++k) {
+        const int d = base + d0 + k * kStep;
+        if (base > 0 && d < a.dim) Wide<AT>::template load<V>(w + static_cast<size_t>(d) * a.kv_rank, wf[k]);
+      }
+#pragma unroll
+      for (int k = 0; k < kFewAhead; ++k) {
+        const int d = base + d0 + k * kStep;
+        if (d >= a.dim) continue;
+#pragma unroll
+        for (int t = 0; t < NT; ++t) {
+          if (t >= T) break;
+          const float qv = qs[t * dq + d];
+#pragma unroll
+          for (int c = 0; c < V; ++c) acc[t][c] = fmaf(qv, wf[k][c], acc[t][c]);
+        }
+      }
+    }
+  }
+#pragma unroll
+  for (int t = 0; t < NT; ++t)
+#pragma unroll
+    for (int c = 0; c < V; ++c) {
+      float v = acc[t][c];
+#pragma unroll
+      for (int o = LPR; o < 32; o <<= 1) v += __shfl_xor_sync(kAll, v, o);
+      if (lane < LPR) red[warp][t][lane * V + c] = v;
+    }
+  __syncthreads();
+  for (int i = threadIdx.x; i < T * kFewCols; i += blockDim.x) {
+    const int t = i / kFewCols, c = i % kFewCols;
+    if (c0 + c >= a.kv_rank) continue;
+    float v = 0.f;
+#pragma unroll
+    for (int k = 0; k < kFewWarps; ++k) v += red[k][t][c];
+    qa[(static_cast<size_t>(t) * a.heads + h) * dl + c0 + c] = v;
+  }
+  if (blockIdx.y != 0) return;
+  for (int i = threadIdx.x; i < T * a.rot_dim; i += blockDim.x) {
+    const int t = i / a.rot_dim, c = i % a.rot_dim;
+    qa[(static_cast<size_t>(t) * a.heads + h) * dl + a.kv_rank + c] = rotated(a, qs + t * dq + a.dim, c, tok_pos[t]);
   }
 }
-// kp [T, heads * dim] fp32 (W_uk c) and kr [T, rot_dim] (rotated, shared by the heads) -> k [T, heads, dim + rot_dim];
-// vp [T, heads * vdim] fp32 (W_uv c) -> v, both in the compute type
-template <typename AT>
-__global__ void latent_pack_kv_kernel(LatentShape a, const float* __restrict__ kp, int kp_row, const float* __restrict__ kr,
-                                      const float* __restrict__ vp, int vp_row, AT* __restrict__ k, AT* __restrict__ v) {
-  const int t = blockIdx.x, dq = a.dim + a.rot_dim;
-  for (int i = threadIdx.x; i < a.heads * dq; i += blockDim.x) {
-    const int h = i / dq, d = i % dq;
-    const float x = d < a.dim ? kp[static_cast<size_t>(t) * kp_row + h * a.dim + d]
-                              : kr[static_cast<size_t>(t) * a.rot_dim + d - a.dim];
-    k[static_cast<size_t>(t) * a.heads * dq + i] = from_f<AT>(x);
+
+// ---- latent attention with per-head keys and values (prompt steps on the tensor cores) ---------------------------------------
+// One CTA per token, a warp per head in turn.  q [heads, dim + rot_dim] fp32 -> the same in the compute type with the rotated part
+// rotated; kp [heads * dim] (W_uk c) and kr [rot_dim] (rotated, shared by the heads) -> k [heads, dim + rot_dim];
+// vp [heads * vdim] (W_uv c) -> v.  The token's cosines and sines are computed once.  V columns at a time: V == 4 needs sizes
+// and row strides that are multiples of 4.
+template <typename AT, int V>
+__global__ void latent_pack_kernel(LatentShape a, const float* __restrict__ q, int q_row, const float* __restrict__ kp,
+                                   int kp_row, const float* __restrict__ kr, const float* __restrict__ vp, int vp_row,
+                                   const int32_t* __restrict__ tok_pos, AT* __restrict__ q_out, AT* __restrict__ k_out,
+                                   AT* __restrict__ v_out) {
+  extern __shared__ float cs[];  // [rope_dims / 2] cosines, then sines
+  const int t = blockIdx.x, dq = a.dim + a.rot_dim, half = a.rope_dims >> 1;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    const float ang = static_cast<float>(tok_pos[t]) * rope_frequency(a, i);
+    sincosf(ang, cs + half + i, cs + i);
   }
-  for (int i = threadIdx.x; i < a.heads * a.vdim; i += blockDim.x)
-    v[static_cast<size_t>(t) * a.heads * a.vdim + i] = from_f<AT>(vp[static_cast<size_t>(t) * vp_row + i]);
+  __syncthreads();
+  const float* kr_t = kr + static_cast<size_t>(t) * a.rot_dim;
+  for (int h = warp; h < a.heads; h += nw) {
+    const float* qh = q + static_cast<size_t>(t) * q_row + h * dq;
+    const float* kh = kp + static_cast<size_t>(t) * kp_row + h * a.dim;
+    AT* qo = q_out + (static_cast<size_t>(t) * a.heads + h) * dq;
+    AT* ko = k_out + (static_cast<size_t>(t) * a.heads + h) * dq;
+    for (int d = lane * V; d < dq; d += 32 * V) {
+      float x[V], y[V];
+      get_floats<V>(qh + d, x);
+      get_floats<V>(d < a.dim ? kh + d : kr_t + d - a.dim, y);
+      if (d >= a.dim) {
+#pragma unroll
+        for (int c = 0; c < V; ++c) {
+          const int i = d - a.dim + c;
+          if (i < a.rope_dims) {
+            const float* r = qh + a.dim;
+            if (a.rope_pairing == KLLM_SEQ_ROPE_PAIRS) {
+              const float co = cs[i >> 1], si = cs[half + (i >> 1)];
+              x[c] = (i & 1) == 0 ? r[i] * co - r[i + 1] * si : r[i] * co + r[i - 1] * si;
+            } else {
+              const int p = i < half ? i : i - half;
+              const float co = cs[p], si = cs[half + p];
+              x[c] = i < half ? r[i] * co - r[i + half] * si : r[i] * co + r[i - half] * si;
+            }
+          }
+        }
+      }
+      put_values<V>(qo + d, x);
+      put_values<V>(ko + d, y);
+    }
+    const float* vh = vp + static_cast<size_t>(t) * vp_row + h * a.vdim;
+    AT* vo = v_out + (static_cast<size_t>(t) * a.heads + h) * a.vdim;
+    for (int d = lane * V; d < a.vdim; d += 32 * V) {
+      float x[V];
+      get_floats<V>(vh + d, x);
+      put_values<V>(vo + d, x);
+    }
+  }
 }
 
 // ---- latent attention: weighted sums of latents -> per-head values ---------------------------------------------------------
@@ -205,39 +365,55 @@ __global__ void latent_expand_kernel(LatentShape a, const float* __restrict__ ol
 // The same for steps of single tokens, fused with the merge of the key splits: a CTA per (token, head) joins the splits'
 // (max, sum, unnormalised latent sums), adds the sink to the denominator, applies the gate, and multiplies by the head's
 // block of W_uv -- the merged latent sum never leaves shared memory.
-template <typename AT>
-__global__ void latent_merge_expand_kernel(LatentShape a, int splits, const float* __restrict__ ws,
-                                           const float* __restrict__ gates, const float* __restrict__ sink,
-                                           const AT* __restrict__ w_uv, AT* __restrict__ out) {
-  extern __shared__ float ls[];  // [kv_rank]
+// The grid's y takes slices of kExpandRows value rows of a head; every slice joins the latent sums again (they are few), and
+// the first 16 bytes per lane of a warp's rows of W_uv are fetched before the sums are ready.
+constexpr int kExpandWarps = 8, kExpandRowsPerWarp = 4, kExpandRows = kExpandWarps * kExpandRowsPerWarp;
+template <typename AT, bool VEC>
+__global__ void __launch_bounds__(kExpandWarps * 32)
+latent_merge_expand_kernel(LatentShape a, int splits, const float* __restrict__ ws, const float* __restrict__ gates,
+                           const float* __restrict__ sink, const AT* __restrict__ w_uv, AT* __restrict__ out) {
+  extern __shared__ __align__(16) float ls[];  // [kv_rank], then [splits] weights
+  float* weight = ls + a.kv_rank;
+  constexpr int V = VEC ? Wide<AT>::N : 1;
   const size_t th = blockIdx.x;  // t * heads + h
   const int h = static_cast<int>(th % a.heads);
   const int pstride = a.kv_rank + 2;
   const float* p = ws + th * splits * pstride;
-  float M = sink ? sink[h] : -INFINITY;
-  for (int s = 0; s < splits; ++s) M = fmaxf(M, p[s * pstride]);
-  float L = sink ? expf(sink[h] - M) : 0.f;
-  for (int s = 0; s < splits; ++s) {
-    const float m = p[s * pstride];
-    if (m > -INFINITY) L += p[s * pstride + 1] * expf(m - M);
-  }
-  const float g = (gates ? gates[th] : 1.0f) / L;
-  for (int d = threadIdx.x; d < a.kv_rank; d += blockDim.x) {
-    float o = 0.f;
-    for (int s = 0; s < splits; ++s) {
-      const float m = p[s * pstride];
-      if (m > -INFINITY) o += p[s * pstride + 2 + d] * expf(m - M);
-    }
-    ls[d] = o * g;
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const int f0 = blockIdx.y * kExpandRows + warp * kExpandRowsPerWarp;
+  const AT* w = w_uv + (static_cast<size_t>(h) * a.vdim + f0) * a.kv_rank;
+  float wf[kExpandRowsPerWarp][V];
+#pragma unroll
+  for (int k = 0; k < kExpandRowsPerWarp; ++k)
+    if (f0 + k < a.vdim && lane * V < a.kv_rank) Wide<AT>::template load<V>(w + static_cast<size_t>(k) * a.kv_rank + lane * V, wf[k]);
+  MergeColumn col;
+  int d = threadIdx.x;
+  if (d < a.kv_rank) col.load(p, splits, pstride, d);
+  const float g = gates ? gates[th] : 1.0f;
+  if (warp == 0) split_weights(p, splits, pstride, sink != nullptr, sink ? sink[h] : 0.f, weight);
+  __syncthreads();
+  while (d < a.kv_rank) {
+    ls[d] = col.join(p, splits, pstride, d, weight) * g;
+    d += blockDim.x;
+    if (d < a.kv_rank) col.load(p, splits, pstride, d);
   }
   __syncthreads();
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  for (int f = warp; f < a.vdim; f += nw) {
-    const AT* w = w_uv + (static_cast<size_t>(h) * a.vdim + f) * a.kv_rank;
-    float acc = 0.f;
-    for (int r = lane; r < a.kv_rank; r += 32) acc = fmaf(ls[r], to_f(w[r]), acc);
-    acc = warp_sum(acc);
-    if (lane == 0) out[th * a.vdim + f] = from_f<AT>(acc);
+  float acc[kExpandRowsPerWarp];
+#pragma unroll
+  for (int k = 0; k < kExpandRowsPerWarp; ++k) acc[k] = 0.f;
+  for (int r = lane * V; r < a.kv_rank; r += 32 * V) {
+#pragma unroll
+    for (int k = 0; k < kExpandRowsPerWarp; ++k) {
+      if (f0 + k >= a.vdim) continue;
+      if (r >= 32 * V) Wide<AT>::template load<V>(w + static_cast<size_t>(k) * a.kv_rank + r, wf[k]);
+#pragma unroll
+      for (int c = 0; c < V; ++c) acc[k] = fmaf(ls[r + c], wf[k][c], acc[k]);
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < kExpandRowsPerWarp; ++k) {
+    const float v = warp_sum(acc[k]);
+    if (lane == 0 && f0 + k < a.vdim) out[th * a.vdim + f0 + k] = from_f<AT>(v);
   }
 }
 
@@ -595,16 +771,20 @@ int launch_latent_prepare(int dtype, const LatentShape& a, const float* proj, co
   return done();
 }
 
-int launch_latent_pack_q(int dtype, const LatentShape& a, const float* q, int q_row, const int32_t* tok_pos, void* out, int T,
-                         cudaStream_t s) {
-  KLLM_SEQ_DISPATCH(dtype, (latent_pack_q_kernel<AT><<<T, 256, 0, s>>>(a, q, q_row, tok_pos, static_cast<AT*>(out))));
-  return done();
-}
-
-int launch_latent_pack_kv(int dtype, const LatentShape& a, const float* kp, int kp_row, const float* kr, const float* vp,
-                          int vp_row, void* k, void* v, int T, cudaStream_t s) {
-  KLLM_SEQ_DISPATCH(dtype, (latent_pack_kv_kernel<AT><<<T, 256, 0, s>>>(a, kp, kp_row, kr, vp, vp_row, static_cast<AT*>(k),
-                                                                       static_cast<AT*>(v))));
+int launch_latent_pack(int dtype, const LatentShape& a, const float* q, int q_row, const float* kp, int kp_row, const float* kr,
+                       const float* vp, int vp_row, const int32_t* tok_pos, void* q_out, void* k_out, void* v_out, int T,
+                       cudaStream_t s) {
+  const bool vec = ((a.dim | a.rot_dim | a.vdim | q_row | kp_row | vp_row) & 3) == 0 && (reinterpret_cast<uintptr_t>(vp) & 15) == 0;
+  const size_t smem = static_cast<size_t>(a.rope_dims) * sizeof(float);
+  if (smem > 48 * 1024) return KLLM_E_UNSUPPORTED;
+  if (vec)
+    KLLM_SEQ_DISPATCH(dtype, (latent_pack_kernel<AT, 4><<<T, 256, smem, s>>>(
+                                 a, q, q_row, kp, kp_row, kr, vp, vp_row, tok_pos, static_cast<AT*>(q_out),
+                                 static_cast<AT*>(k_out), static_cast<AT*>(v_out))));
+  else
+    KLLM_SEQ_DISPATCH(dtype, (latent_pack_kernel<AT, 1><<<T, 256, smem, s>>>(
+                                 a, q, q_row, kp, kp_row, kr, vp, vp_row, tok_pos, static_cast<AT*>(q_out),
+                                 static_cast<AT*>(k_out), static_cast<AT*>(v_out))));
   return done();
 }
 
@@ -612,6 +792,20 @@ int launch_latent_absorb(int dtype, const LatentShape& a, const float* q, int q_
                          float* qa, int T, cudaStream_t s) {
   const size_t smem = static_cast<size_t>(kAbsTokens) * (a.dim + a.rot_dim) * sizeof(float);
   if (smem > 48 * 1024) return KLLM_E_UNSUPPORTED;
+  if (T <= 8 && a.kv_rank % 8 == 0 && (reinterpret_cast<uintptr_t>(w_uk) & 15) == 0) {
+    const dim3 grid(a.heads, (a.kv_rank + kFewCols - 1) / kFewCols);
+    const size_t few = static_cast<size_t>(T) * (a.dim + a.rot_dim) * sizeof(float);
+#define KLLM_ABSORB(NT)                                                                                                   \
+  KLLM_SEQ_DISPATCH(dtype, (latent_absorb_few_kernel<AT, NT><<<grid, kFewWarps * 32, few, s>>>(a, q, q_row,               \
+                                                                                               static_cast<const AT*>(w_uk), \
+                                                                                               tok_pos, qa, T)))
+    if (T == 1) KLLM_ABSORB(1);
+    else if (T == 2) KLLM_ABSORB(2);
+    else if (T <= 4) KLLM_ABSORB(4);
+    else KLLM_ABSORB(8);
+#undef KLLM_ABSORB
+    return done();
+  }
   // few tokens: 64 latent coordinates per CTA; many tokens: the whole latent (the queries are staged once per CTA)
   const int threads = T <= kAbsTokens ? 64 : (a.kv_rank <= 64 ? 64 : (a.kv_rank <= 128 ? 128 : 256));
   const dim3 grid((T + kAbsTokens - 1) / kAbsTokens, a.heads, (a.kv_rank + threads - 1) / threads);
@@ -622,9 +816,15 @@ int launch_latent_absorb(int dtype, const LatentShape& a, const float* q, int q_
 
 int launch_latent_merge_expand(int dtype, const LatentShape& a, int splits, const float* ws, const float* gates,
                                const float* sink, const void* w_uv, void* out, int T, cudaStream_t s) {
-  const size_t smem = static_cast<size_t>(a.kv_rank) * sizeof(float);
-  KLLM_SEQ_DISPATCH(dtype, (latent_merge_expand_kernel<AT><<<T * a.heads, 256, smem, s>>>(
-                               a, splits, ws, gates, sink, static_cast<const AT*>(w_uv), static_cast<AT*>(out))));
+  const size_t smem = (static_cast<size_t>(a.kv_rank) + splits) * sizeof(float);
+  const dim3 grid(T * a.heads, (a.vdim + kExpandRows - 1) / kExpandRows);
+  const bool vec = a.kv_rank % 8 == 0 && (reinterpret_cast<uintptr_t>(w_uv) & 15) == 0;
+  if (vec)
+    KLLM_SEQ_DISPATCH(dtype, (latent_merge_expand_kernel<AT, true><<<grid, kExpandWarps * 32, smem, s>>>(
+                                 a, splits, ws, gates, sink, static_cast<const AT*>(w_uv), static_cast<AT*>(out))));
+  else
+    KLLM_SEQ_DISPATCH(dtype, (latent_merge_expand_kernel<AT, false><<<grid, kExpandWarps * 32, smem, s>>>(
+                                 a, splits, ws, gates, sink, static_cast<const AT*>(w_uv), static_cast<AT*>(out))));
   return done();
 }
 

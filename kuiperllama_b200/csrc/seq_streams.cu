@@ -167,7 +167,9 @@ int launch_s(const StreamArgs& a, cudaStream_t s) {
   if (smem > 48 * 1024) return KLLM_E_UNSUPPORTED;
   const bool vec = a.width % 4 == 0;
   const int per = vec ? (a.width + 3) / 4 : a.width;
-  const int threads = std::max(64, std::min(512, (per + 31) / 32 * 32));
+  // few rows: as many loads in flight as a row has; many rows: several CTAs per SM, so that one's reduction hides behind the
+  // others' loads
+  const int threads = std::max(64, std::min(a.T <= 16 ? 512 : 256, (per + 31) / 32 * 32));
   if (vec) streams_kernel<AT, S, 4, EXACT><<<a.T, threads, smem, s>>>(a);
   else streams_kernel<AT, S, 1, EXACT><<<a.T, threads, smem, s>>>(a);
   count_launch();
