@@ -77,16 +77,24 @@ rows_kernel(const AT* __restrict__ a, const AT* __restrict__ w, const float* __r
 #pragma unroll
   for (int r = 0; r < R; ++r) acc[r] = 0.f;
   if (VEC) {
-    for (int k = lane * V; k < K; k += 32 * V) {
-      float wf[V];
-      Vec16<AT>::load_stream(wr + k, wf);
+    constexpr int U = 4;  // 16-byte weight loads in flight per lane
+    for (int k0 = lane * V; k0 < K; k0 += U * 32 * V) {
+      float wf[U][V];
 #pragma unroll
-      for (int r = 0; r < R; ++r) {
-        if (r < T) {
-          float af[V];
-          Vec16<AT>::load(a + static_cast<size_t>(r) * K + k, af);
+      for (int u = 0; u < U; ++u)
+        if (k0 + u * 32 * V < K) Vec16<AT>::load_stream(wr + k0 + u * 32 * V, wf[u]);
 #pragma unroll
-          for (int i = 0; i < V; ++i) acc[r] = fmaf(af[i], wf[i], acc[r]);
+      for (int u = 0; u < U; ++u) {
+        const int k = k0 + u * 32 * V;
+        if (k >= K) break;
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+          if (r < T) {
+            float af[V];
+            Vec16<AT>::load(a + static_cast<size_t>(r) * K + k, af);
+#pragma unroll
+            for (int i = 0; i < V; ++i) acc[r] = fmaf(af[i], wf[u][i], acc[r]);
+          }
         }
       }
     }
@@ -121,17 +129,27 @@ rows_gated_kernel(const AT* __restrict__ a, const AT* __restrict__ w, AT* __rest
 #pragma unroll
   for (int r = 0; r < R; ++r) g[r] = u[r] = 0.f;
   if (VEC) {
-    for (int k = lane * V; k < K; k += 32 * V) {
-      float gf[V], uf[V];
-      Vec16<AT>::load_stream(wg + k, gf);
-      Vec16<AT>::load_stream(wu + k, uf);
+    constexpr int U = 2;  // of each row
+    for (int k0 = lane * V; k0 < K; k0 += U * 32 * V) {
+      float gf[U][V], uf[U][V];
 #pragma unroll
-      for (int r = 0; r < R; ++r) {
-        if (r < T) {
-          float af[V];
-          Vec16<AT>::load(a + static_cast<size_t>(r) * K + k, af);
+      for (int z = 0; z < U; ++z)
+        if (k0 + z * 32 * V < K) {
+          Vec16<AT>::load_stream(wg + k0 + z * 32 * V, gf[z]);
+          Vec16<AT>::load_stream(wu + k0 + z * 32 * V, uf[z]);
+        }
 #pragma unroll
-          for (int i = 0; i < V; ++i) g[r] = fmaf(af[i], gf[i], g[r]), u[r] = fmaf(af[i], uf[i], u[r]);
+      for (int z = 0; z < U; ++z) {
+        const int k = k0 + z * 32 * V;
+        if (k >= K) break;
+#pragma unroll
+        for (int r = 0; r < R; ++r) {
+          if (r < T) {
+            float af[V];
+            Vec16<AT>::load(a + static_cast<size_t>(r) * K + k, af);
+#pragma unroll
+            for (int i = 0; i < V; ++i) g[r] = fmaf(af[i], gf[z][i], g[r]), u[r] = fmaf(af[i], uf[z][i], u[r]);
+          }
         }
       }
     }

@@ -30,7 +30,8 @@ namespace umma {
 constexpr int BM = 128;    // weight rows per CTA = MMA M
 constexpr int BK = 64;     // bf16 elements per K block = 128 bytes = one swizzle row
 constexpr int UK = 16;     // K of one tcgen05.mma.kind::f16
-constexpr int STAGES = 4;
+constexpr int STAGES = 4;   // of the grouped form
+constexpr int kSms = 148;
 constexpr int A_BYTES = BM * BK * 2;
 constexpr int THREADS = 192;
 constexpr uint32_t kWaitLimit = 1u << 24;  // try_wait rounds before a wait gives up (each suspends up to ~1 us)
@@ -96,7 +97,9 @@ __device__ __forceinline__ void tmem_ld32(uint32_t taddr, uint32_t (&r)[32]) {
       : "r"(taddr) : "memory");
 }
 
-template <int BN, bool GATED>
+// ST: stages of the ring.  A ring of at most ~110 KB leaves room for a second CTA on the SM, whose products run under the
+// first one's epilogue.
+template <int BN, bool GATED, int ST>
 __global__ void __launch_bounds__(THREADS, 1)
 umma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ CUtensorMap map_a,
             void* __restrict__ out_, const float* __restrict__ bias, int T, int N, int K, GatedAct act) {
@@ -106,12 +109,12 @@ umma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ C
   extern __shared__ uint8_t raw_smem[];
   uint8_t* base = reinterpret_cast<uint8_t*>((reinterpret_cast<uintptr_t>(raw_smem) + 1023) & ~uintptr_t(1023));
   uint8_t* a_tiles = base;                       // weight tiles (MMA A)
-  uint8_t* b_tiles = base + STAGES * W_BYTES;    // token tiles (MMA B)
-  uint64_t* bars = reinterpret_cast<uint64_t*>(b_tiles + STAGES * B_BYTES);
+  uint8_t* b_tiles = base + ST * W_BYTES;    // token tiles (MMA B)
+  uint64_t* bars = reinterpret_cast<uint64_t*>(b_tiles + ST * B_BYTES);
   uint64_t* full = bars;
-  uint64_t* empty = bars + STAGES;
-  uint64_t* tmem_full = bars + 2 * STAGES;
-  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 2 * STAGES + 1);
+  uint64_t* empty = bars + ST;
+  uint64_t* tmem_full = bars + 2 * ST;
+  uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + 2 * ST + 1);
   volatile int* stop = reinterpret_cast<volatile int*>(tmem_slot + 1);
 
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -119,7 +122,7 @@ umma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ C
   const int kblocks = (K + BK - 1) / BK;
 
   if (threadIdx.x == 0) {
-    for (int s = 0; s < STAGES; ++s) {
+    for (int s = 0; s < ST; ++s) {
       mbar_init(smem_u32(&full[s]), 1);
       mbar_init(smem_u32(&empty[s]), 1);
     }
@@ -140,8 +143,8 @@ umma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ C
   if (warp == 0) {
     if (lane == 0) {
       for (int kb = 0; kb < kblocks; ++kb) {
-        const int s = kb % STAGES;
-        if (!mbar_wait(smem_u32(&empty[s]), ((kb / STAGES) & 1) ^ 1u, stop)) break;
+        const int s = kb % ST;
+        if (!mbar_wait(smem_u32(&empty[s]), ((kb / ST) & 1) ^ 1u, stop)) break;
         const uint32_t bar = smem_u32(&full[s]);
         mbar_expect_tx(bar, W_BYTES + B_BYTES);
         tma_load_2d(smem_u32(a_tiles + s * W_BYTES), &map_w, bar, kb * BK, n0);
@@ -154,8 +157,8 @@ umma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ C
       const uint32_t idesc = instr_desc(BN);
       bool ok = true;
       for (int kb = 0; kb < kblocks && ok; ++kb) {
-        const int s = kb % STAGES;
-        ok = mbar_wait(smem_u32(&full[s]), (kb / STAGES) & 1, stop);
+        const int s = kb % ST;
+        ok = mbar_wait(smem_u32(&full[s]), (kb / ST) & 1, stop);
         if (!ok) break;
         asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
         const uint32_t a_addr = smem_u32(a_tiles + s * W_BYTES);
@@ -379,23 +382,23 @@ inline int make_map(CUtensorMap* map, const void* ptr, int rows, int cols, int b
   return r == CUDA_SUCCESS ? 0 : KLLM_E_INVALID;
 }
 
-template <int BN, bool GATED>
+template <int BN, bool GATED, int ST>
 inline int launch_bn(const void* a, const void* w, const float* bias, void* out, int T, int K, int N, const GatedAct& act,
                      cudaStream_t stream) {
   constexpr int NA = GATED ? 2 : 1;
   CUtensorMap map_w, map_a;
   if (int rc = make_map(&map_w, w, NA * N, K, BM)) return rc;
   if (int rc = make_map(&map_a, a, T, K, BN)) return rc;
-  const size_t smem = 1024 + static_cast<size_t>(STAGES) * (NA * A_BYTES + BN * BK * 2) + 256;
+  const size_t smem = 1024 + static_cast<size_t>(ST) * (NA * A_BYTES + BN * BK * 2) + 256;
   static bool configured = false;
   if (!configured) {
-    const cudaError_t e = cudaFuncSetAttribute(umma_kernel<BN, GATED>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    const cudaError_t e = cudaFuncSetAttribute(umma_kernel<BN, GATED, ST>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                                static_cast<int>(smem));
     if (e != cudaSuccess) return static_cast<int>(e);
     configured = true;
   }
   const dim3 grid((N + BM - 1) / BM, (T + BN - 1) / BN);
-  umma_kernel<BN, GATED><<<grid, THREADS, smem, stream>>>(map_w, map_a, out, bias, T, N, K, act);
+  umma_kernel<BN, GATED, ST><<<grid, THREADS, smem, stream>>>(map_w, map_a, out, bias, T, N, K, act);
   count_launch();
   return static_cast<int>(cudaGetLastError());
 }
@@ -415,11 +418,10 @@ template <>
 inline int launch<__nv_bfloat16>(const __nv_bfloat16* a, const __nv_bfloat16* w, const float* bias, float* out, int T, int K,
                                  int N, cudaStream_t s) {
   const GatedAct none{KLLM_SEQ_ACT_SWIGLU, 0.f, 0.f};
-  // few feature tiles: narrower token blocks give more CTAs
+  // less than one tile of 128 tokens per SM: narrower token blocks give more CTAs; else two CTAs share an SM
   const int feature_tiles = (N + BM - 1) / BM;
-  if (T <= 64 || feature_tiles * ((T + 127) / 128) < 100) return launch_bn<64, false>(a, w, bias, out, T, K, N, none, s);
-  if (T <= 128 || feature_tiles * ((T + 255) / 256) < 148) return launch_bn<128, false>(a, w, bias, out, T, K, N, none, s);
-  return launch_bn<256, false>(a, w, bias, out, T, K, N, none, s);
+  if (T <= 64 || feature_tiles * ((T + 127) / 128) < kSms) return launch_bn<64, false, 4>(a, w, bias, out, T, K, N, none, s);
+  return launch_bn<128, false, 3>(a, w, bias, out, T, K, N, none, s);
 }
 
 // w: [2 * N, K], gate rows then up rows; two weight tiles share a token tile, so a CTA computes 128 features x BN tokens twice
@@ -429,8 +431,8 @@ template <>
 inline int launch_gated<__nv_bfloat16>(const __nv_bfloat16* a, const __nv_bfloat16* w, __nv_bfloat16* out, int T, int K, int N,
                                        const GatedAct& act, cudaStream_t s) {
   const int feature_tiles = (N + BM - 1) / BM;
-  if (T <= 64 || feature_tiles * ((T + 127) / 128) < 100) return launch_bn<64, true>(a, w, nullptr, out, T, K, N, act, s);
-  return launch_bn<128, true>(a, w, nullptr, out, T, K, N, act, s);
+  if (T <= 64 || feature_tiles * ((T + 127) / 128) < kSms) return launch_bn<64, true, 4>(a, w, nullptr, out, T, K, N, act, s);
+  return launch_bn<128, true, 2>(a, w, nullptr, out, T, K, N, act, s);
 }
 
 inline bool grouped_usable(int K, int N) {
