@@ -40,6 +40,8 @@
 //                  an attention may also rotate its queries and keys (frequencies from a table), norm them after the
 //                  rotation, gate every output element, and run as a DIFFERENTIAL attention: two maps per head over the
 //                  same values, joined by diff_merge
+//                  or be normed over the whole query / key projections, and blend their values with those an earlier layer of
+//                  the step kept; a latent attention may project its queries directly
 //                  a layer may run two mixers of different kinds on the same rows; their outputs join x with a weight each,
 //                  each after an RMS norm of its own when the layer names one
 //     gemm         output projection
@@ -47,11 +49,13 @@
 //                  is still in shared memory
 //                  (a layer whose feed-forward reads the mixer's input skips this: the first norm kernel routes its row, the
 //                  feed-forward runs on the same rows after the mixers, and ONE sum joins x at the end of the run)
-//     feed-forward dense: gemm, activation, gemm
+//     feed-forward dense: gemm, activation, gemm -- or, gated, one product whose epilogue joins gate and up rows, gemm
 //                  experts, few tokens: pair kernels (weights streamed once per chosen expert; a shared expert rides
 //                  along as one more pair per token); many tokens: pairs sorted by expert, two grouped products (SiLU-gate
 //                  or squared-ReLU epilogue in the first); shared expert: gemm gate|up, silu_mul, gemm down
 //     resid_norm   x += N_post_ff(ff output)   [+ what comes ahead of the next run's mixer, fused]
+// A model with residual STREAMS has one kernel (launch_streams) in place of resid_norm: it mixes the streams with the output of
+// the sublayer that ends, reads the weighted sum for the one that starts, and norms it.
 // then the final norm on the wanted rows only, the classifier product, the logit scale, argmax, and one device->host copy.
 #include <cuda_runtime.h>
 
