@@ -116,6 +116,8 @@ typedef struct kllm_seq_attention {
    * blend.  The latest source ahead of a MIX layer in the run order must have the same kv_heads * vdim. */
   int32_t v_blend;
   float v_lambda;
+  int32_t chunk;         /* > 0: position i sees j only inside its own chunk, floor(i / chunk) == floor(j / chunk), chunks counted
+                            from position 0 of the sequence (kept first positions stay visible); with a window both hold */
 } kllm_seq_attention;
 
 /* Attention through a latent.  Queries: cq = RMSnorm(W_dq h), q = W_uq cq -- or q = W_q h itself (q_rank == 0) --, per head
@@ -145,14 +147,32 @@ typedef struct kllm_seq_latent {
   const float* rope_freq; /* [rope_dims / 2] fp32: angle of pair i = position * rope_freq[i], or NULL: rope_base^(-2 i / rope_dims) */
 } kllm_seq_latent;
 
-/* Linear attention: q, k, v = silu(W h); per head S <- decay * S + k v^T, o = S^T q; the heads together are RMS-normed,
- * multiplied by sigmoid(W_g h) and projected.  S [dim, vdim] per head is fp32 state of the sequence. */
+/* what is done to the projected q, k and v of a linear attention (kllm_seq_linear.qkv_act) */
+#define KLLM_SEQ_QKV_SILU 0
+#define KLLM_SEQ_QKV_PLAIN 1
+/* its output norm (kllm_seq_linear.out_norm) and the activation of its gate rows (kllm_seq_linear.gate_act) */
+#define KLLM_SEQ_OUTNORM_ROW 0  /* ONE RMS norm over all heads, weights out_norm_w */
+#define KLLM_SEQ_OUTNORM_HEAD 1 /* every head is divided by its own root mean square, no weights */
+#define KLLM_SEQ_GATEACT_SIGMOID 0
+#define KLLM_SEQ_GATEACT_SILU 1
+
+/* Linear attention: q, k, v = silu(W h) or W h; per head S <- decay * S + k v^T, o = S^T q; the output is RMS-normed (all heads
+ * together or each on its own), multiplied by sigmoid(W_g h) or silu(W_g h) and projected.  S [dim, vdim] per head is fp32
+ * state of the sequence.  A retention is the form without activation: q and k rotated, k scaled, heads normed one by one. */
 typedef struct kllm_seq_linear {
   int32_t heads, dim, vdim;
   const float* decay;      /* [heads], device */
   const void* w_in;        /* [2 * heads * dim + 2 * heads * vdim, width]: q | k | v | gate rows */
-  const float* out_norm_w; /* [heads * vdim] */
+  const float* out_norm_w; /* [heads * vdim]; not read with KLLM_SEQ_OUTNORM_HEAD */
   const void* w_out;       /* [width, heads * vdim] */
+  int32_t qkv_act;         /* KLLM_SEQ_QKV_* */
+  int32_t rope_dims;       /* rotary positions on the first rope_dims coordinates of every q and k head (PLAIN only); 0: none */
+  float rope_base;
+  int32_t rope_pairing;    /* KLLM_SEQ_ROPE_* */
+  const float* rope_freq;  /* [rope_dims / 2] fp32: angle of pair i = position * rope_freq[i], or NULL: rope_base^(-2 i / rope_dims) */
+  float k_scale;           /* k is multiplied by it after the rotation (PLAIN only); 0 means 1 */
+  int32_t out_norm;        /* KLLM_SEQ_OUTNORM_* */
+  int32_t gate_act;        /* KLLM_SEQ_GATEACT_* */
 } kllm_seq_linear;
 
 /* Selective scan.  W_in h = [u | z] (inner each); u <- silu(conv(u) + conv_b); W_x u = [low: dt_rank | B: state | C: state];
@@ -207,10 +227,12 @@ typedef struct kllm_seq_ssd {
 } kllm_seq_ssd;
 
 typedef struct kllm_seq_dense {
-  int32_t ff, act;    /* inner size; KLLM_SEQ_ACT_* (XIELU, RELU2, or RELU_GATE / GELU_GATE: then `up` holds ff gate rows followed by ff up rows) */
-  float act_a, act_b; /* the two coefficients of KLLM_SEQ_ACT_XIELU */
+  int32_t ff, act;    /* inner size; KLLM_SEQ_ACT_* (XIELU, RELU2, or RELU_GATE / GELU_GATE / CLAMP_SWIGLU: then `up` holds ff gate rows followed by ff up rows) */
+  float act_a, act_b; /* the two coefficients of KLLM_SEQ_ACT_XIELU; KLLM_SEQ_ACT_CLAMP_SWIGLU: the limit and the sigmoid's slope */
   const void* up;     /* [ff, width] */
   const void* down;   /* [width, ff] */
+  const float* up_bias;   /* [rows of up] fp32 added to the inner products before the activation, or NULL */
+  const float* down_bias; /* [width] fp32, or NULL */
 } kllm_seq_dense;
 
 typedef struct kllm_seq_moe {
@@ -300,6 +322,12 @@ typedef struct kllm_seq_desc {
   int32_t streams;           /* residual streams joined by hyper-connections (kllm_seq_hyper); 0: one plain residual.  Streams
                                 take no post-norms, token shift, second mixer, feed-forward beside the mixer, routed experts
                                 or additions before a run */
+  /* Bigram embedding: row (previous token * bigram_mul_prev + token * bigram_mul_cur) mod bigram_buckets of `bigram` joins the
+   * (scaled) embedding row; a sequence's first token takes the row behind them, number bigram_buckets.  The previous token is
+   * state of the sequence. */
+  const void* bigram;        /* [bigram_buckets + 1, width] compute type, or NULL */
+  int32_t bigram_buckets;
+  int64_t bigram_mul_prev, bigram_mul_cur; /* >= 0 */
 } kllm_seq_desc;
 
 typedef struct kllm_seq_engine kllm_seq_engine;

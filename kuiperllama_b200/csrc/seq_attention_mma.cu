@@ -114,12 +114,11 @@ attention_mma_kernel(AttnShape a, const __nv_bfloat16* __restrict__ q, PagedKV k
   const int rows_here = min(kRows, n_rows - r0);
   const int pmax = pos0 + (r0 + rows_here - 1) / rep;  // last position any row of the tile sees
   const int n_tiles = pmax / kKeys + 1;
-  // with a window the first row of the tile sees nothing before its position - window + 1
-  const int window = a.window;
-  const int tile_first = window > 0 ? max(0, pos0 + r0 / rep - window + 1) / kKeys : 0;
+  // with a window or chunks no row of the tile sees anything before what its first row sees
+  const int tile_first = first_seen(a, pos0 + r0 / rep) / kKeys;
   // tiles before the window that hold kept first positions come ahead of the window's tiles: this CTA's list of tiles
   // is [0, keep_tiles) then [tile_first, n_tiles), cut into `splits` parts
-  const int keep_first = window > 0 ? a.keep_first : 0;
+  const int keep_first = a.keep_first;
   const int keep_tiles = min(tile_first, (keep_first + kKeys - 1) / kKeys);
   const int list_n = keep_tiles + n_tiles - tile_first;
   const int per = (list_n + splits - 1) / splits;
@@ -142,6 +141,11 @@ attention_mma_kernel(AttnShape a, const __nv_bfloat16* __restrict__ q, PagedKV k
   const int warp_last = __reduce_max_sync(0xffffffffu, max(posA, posB));  // last position any row of the warp sees
   // first position of the warp's rows (rows that do not exist count as -1: their tiles are always masked)
   const int warp_first = __reduce_min_sync(0xffffffffu, min(posA, posB));
+  // the first key each of the two rows sees, and the least and greatest of these among the warp's rows
+  constexpr int kNone = 0x7fffffff;
+  const int loA = exA ? first_seen(a, posA) : kNone, loB = exB ? first_seen(a, posB) : kNone;
+  const int warp_lo = __reduce_min_sync(0xffffffffu, min(loA, loB));
+  const int warp_lo_last = __reduce_max_sync(0xffffffffu, max(exA ? loA : 0, exB ? loB : 0));
   const float scale2_plain = a.scale * 1.4426950408889634f;  // scores are kept in units of log2: exp(x) = 2^(x log2 e)
 
   uint32_t qf[KS][4];
@@ -203,8 +207,8 @@ attention_mma_kernel(AttnShape a, const __nv_bfloat16* __restrict__ q, PagedKV k
     }
     __syncthreads();
     const int k0 = tile * kKeys;
-    // otherwise no row of this warp sees a key of the tile (all later, or all before every row's window)
-    if (k0 <= warp_last && (window == 0 || k0 + kKeys - 1 > warp_first - window || k0 < keep_first)) {
+    // otherwise no row of this warp sees a key of the tile (all later, or all before what every row sees)
+    if (k0 <= warp_last && (k0 + kKeys > warp_lo || k0 < keep_first)) {
       float s[kKeys / 8][4];
 #pragma unroll
       for (int j = 0; j < kKeys / 8; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
@@ -231,7 +235,7 @@ attention_mma_kernel(AttnShape a, const __nv_bfloat16* __restrict__ q, PagedKV k
       }
       const float scale2 = softcap > 0.f ? 1.4426950408889634f : scale2_plain;
       float mxA = -INFINITY, mxB = -INFINITY;
-      if (k0 + kKeys - 1 <= warp_first && (window == 0 || warp_last - k0 < window)) {  // every row of the warp sees the whole tile
+      if (k0 + kKeys - 1 <= warp_first && k0 >= warp_lo_last) {  // every row of the warp sees the whole tile
 #pragma unroll
         for (int j = 0; j < kKeys / 8; ++j) {
           s[j][0] *= scale2, s[j][1] *= scale2, s[j][2] *= scale2, s[j][3] *= scale2;
@@ -242,11 +246,10 @@ attention_mma_kernel(AttnShape a, const __nv_bfloat16* __restrict__ q, PagedKV k
 #pragma unroll
         for (int j = 0; j < kKeys / 8; ++j) {
           const int kj = k0 + j * 8 + t4 * 2;
-          const int loA = window > 0 ? posA - window : -1, loB = window > 0 ? posB - window : -1;  // the last key not seen
-          s[j][0] = kj <= posA && (kj > loA || kj < keep_first) ? s[j][0] * scale2 : -INFINITY;
-          s[j][1] = kj + 1 <= posA && (kj + 1 > loA || kj + 1 < keep_first) ? s[j][1] * scale2 : -INFINITY;
-          s[j][2] = kj <= posB && (kj > loB || kj < keep_first) ? s[j][2] * scale2 : -INFINITY;
-          s[j][3] = kj + 1 <= posB && (kj + 1 > loB || kj + 1 < keep_first) ? s[j][3] * scale2 : -INFINITY;
+          s[j][0] = kj <= posA && (kj >= loA || kj < keep_first) ? s[j][0] * scale2 : -INFINITY;
+          s[j][1] = kj + 1 <= posA && (kj + 1 >= loA || kj + 1 < keep_first) ? s[j][1] * scale2 : -INFINITY;
+          s[j][2] = kj <= posB && (kj >= loB || kj < keep_first) ? s[j][2] * scale2 : -INFINITY;
+          s[j][3] = kj + 1 <= posB && (kj + 1 >= loB || kj + 1 < keep_first) ? s[j][3] * scale2 : -INFINITY;
           mxA = fmaxf(mxA, fmaxf(s[j][0], s[j][1]));
           mxB = fmaxf(mxB, fmaxf(s[j][2], s[j][3]));
         }
@@ -405,9 +408,9 @@ attention_rows_mma_kernel(AttnShape a, const void* __restrict__ q_, PagedKV kv, 
   const int32_t* table = kv.table + static_cast<size_t>(ent_seq[e]) * kv.table_stride;
   const int pmax = pos0 + (r0 + rows_here - 1) / rep;
   const int n_tiles = pmax / kFewKeys + 1;
-  const int window = a.window, keep_first = window > 0 ? a.keep_first : 0;
-  const int tile_first = window > 0 ? max(0, pos0 + r0 / rep - window + 1) / kFewKeys : 0;
-  // this CTA's list of tiles: those with kept first positions ahead of the window, then the window's; cut into splits
+  const int keep_first = a.keep_first;
+  const int tile_first = first_seen(a, pos0 + r0 / rep) / kFewKeys;
+  // this CTA's list of tiles: those with kept first positions ahead of what the rows see, then the others; cut into splits
   const int keep_tiles = min(tile_first, (keep_first + kFewKeys - 1) / kFewKeys);
   const int list_n = keep_tiles + n_tiles - tile_first;
   const int per = (list_n + splits - 1) / splits;
@@ -477,6 +480,10 @@ attention_rows_mma_kernel(AttnShape a, const void* __restrict__ q_, PagedKV kv, 
   for (int i = 0; i < NBW; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
   const int nb_all = (vdim + 7) / 8;
   const int gq = lane >> 2, t4 = lane & 3;
+  // positions of this lane's two rows, and the first key each of them sees
+  int row_pos[2], row_lo[2];
+#pragma unroll
+  for (int z = 0; z < 2; ++z) row_pos[z] = pos0 + (r0 + gq + z * 8) / rep, row_lo[z] = first_seen(a, row_pos[z]);
   // addresses of this lane's rows in the A fragments (16 x 16 tiles: rows lane % 16, columns + 8 for the upper lanes)
   const uint32_t qh_addr = base + static_cast<uint32_t>(L.q_hi) + ((lane & 15) * ldk + (lane >> 4) * 8) * 2;
   const uint32_t ql_addr = base + static_cast<uint32_t>(L.q_lo) + ((lane & 15) * ldk + (lane >> 4) * 8) * 2;
@@ -509,10 +516,9 @@ attention_rows_mma_kernel(AttnShape a, const void* __restrict__ q_, PagedKV kv, 
 #pragma unroll
       for (int c = 0; c < 4; ++c) {
         const int r = gq + (c >> 1) * 8, j = warp * 8 + t4 * 2 + (c & 1), kj = k0 + j;
-        const int pr = pos0 + (r0 + r) / rep;
         float sv = (s0[c] + s1[c]) * a.scale;
         if (a.softcap > 0.f) sv = a.softcap * tanhf(sv / a.softcap);
-        const bool visible = r < rows_here && kj <= pr && (window == 0 || pr - kj < window || kj < keep_first);
+        const bool visible = r < rows_here && kj <= row_pos[c >> 1] && (kj >= row_lo[c >> 1] || kj < keep_first);
         Ss[r * (kFewKeys + 1) + j] = visible ? sv : -INFINITY;
       }
     }

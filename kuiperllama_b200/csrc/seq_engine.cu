@@ -136,6 +136,7 @@ struct kllm_seq_engine {
     bool live = false;
     int len = 0;
     int pages = 0;
+    int32_t last = -1;  // the token before the next one (bigram embedding); -1: none yet
   };
   std::vector<Slot> slots;
   // per-step staging
@@ -206,7 +207,7 @@ static AttnShape attn_shape(const kllm_seq_attention& A) {
   AttnShape s{};
   s.heads = A.heads * maps, s.kv_heads = A.kv_heads * maps, s.dim = A.dim, s.vdim = A.vdim, s.scale = A.scale;
   s.temp_coef = A.temp_coef, s.temp_every = A.temp_every, s.qk_norm = A.qk_norm, s.gate = A.gate, s.window = A.window;
-  s.sink = A.sink, s.keep_first = A.keep_first, s.softcap = A.softcap, s.v_share = maps;
+  s.sink = A.sink, s.keep_first = A.keep_first, s.softcap = A.softcap, s.v_share = maps, s.chunk = A.chunk;
   s.no_merge = A.differential ? 1 : 0;  // the maps' key splits are joined by diff_merge
   return s;
 }
@@ -219,7 +220,9 @@ static LatentShape latent_shape(const kllm_seq_latent& A) {
   return LatentShape{A.heads, A.dim, A.rot_dim, A.vdim, A.q_rank, A.kv_rank, A.rope_dims, A.rope_base, A.gate, A.rope_pairing, A.rope_freq};
 }
 // an inner layer of gate rows and up rows joined by the activation
-static bool dense_gated(const kllm_seq_dense& f) { return f.act == KLLM_SEQ_ACT_RELU_GATE || f.act == KLLM_SEQ_ACT_GELU_GATE; }
+static bool dense_gated(const kllm_seq_dense& f) {
+  return f.act == KLLM_SEQ_ACT_RELU_GATE || f.act == KLLM_SEQ_ACT_GELU_GATE || f.act == KLLM_SEQ_ACT_CLAMP_SWIGLU;
+}
 static bool has_cache(int kind) { return kind == KLLM_SEQ_MIXER_ATTENTION || kind == KLLM_SEQ_MIXER_LATENT; }
 
 static int validate_mixer(const kllm_seq_layer& L, int kind) {
@@ -236,7 +239,7 @@ static int validate_mixer(const kllm_seq_layer& L, int kind) {
     if (a.differential && a.qk_norm == KLLM_SEQ_QKNORM_PROJECTION) return KLLM_E_UNSUPPORTED;
     if ((a.differential || a.values_are_keys) && (a.vdim > 256 || a.dim > 512)) return KLLM_E_UNSUPPORTED;
     if (a.dim > 4096 || a.vdim > 4096) return KLLM_E_UNSUPPORTED;
-    if (a.window < 0 || a.keep_first < 0 || a.softcap < 0.f || a.conv_taps < 0 || a.rope_dims < 0 || a.rope_dims > a.dim ||
+    if (a.window < 0 || a.chunk < 0 || a.keep_first < 0 || a.softcap < 0.f || a.conv_taps < 0 || a.rope_dims < 0 || a.rope_dims > a.dim ||
         (a.rope_dims & 1) || (a.rope_dims > 0 && a.rope_base <= 0.f))
       return KLLM_E_INVALID;
     if (a.values_are_keys && a.vdim != a.dim) return KLLM_E_INVALID;
@@ -254,7 +257,15 @@ static int validate_mixer(const kllm_seq_layer& L, int kind) {
     if (a.kv_rank > 768 || a.dim + a.rot_dim > 768) return KLLM_E_UNSUPPORTED;
   } else if (kind == KLLM_SEQ_MIXER_LINEAR) {
     const kllm_seq_linear& a = L.linear;
-    if (a.heads <= 0 || a.dim <= 0 || a.vdim <= 0 || !a.decay || !a.w_in || !a.out_norm_w || !a.w_out) return KLLM_E_INVALID;
+    if (a.heads <= 0 || a.dim <= 0 || a.vdim <= 0 || !a.decay || !a.w_in || !a.w_out ||
+        (!a.out_norm_w && a.out_norm == KLLM_SEQ_OUTNORM_ROW))
+      return KLLM_E_INVALID;
+    if (a.qkv_act < 0 || a.qkv_act > KLLM_SEQ_QKV_PLAIN || a.out_norm < 0 || a.out_norm > KLLM_SEQ_OUTNORM_HEAD || a.gate_act < 0 ||
+        a.gate_act > KLLM_SEQ_GATEACT_SILU || a.rope_dims < 0 || a.rope_dims > a.dim || (a.rope_dims & 1) ||
+        (a.rope_dims > 0 && !a.rope_freq && a.rope_base <= 0.f))
+      return KLLM_E_INVALID;
+    // the activation's form has no rotation
+    if (a.qkv_act == KLLM_SEQ_QKV_SILU && (a.rope_dims > 0 || (a.k_scale != 0.f && a.k_scale != 1.0f))) return KLLM_E_UNSUPPORTED;
     if (a.dim > 256) return KLLM_E_UNSUPPORTED;
   } else if (kind == KLLM_SEQ_MIXER_SSM) {
     const kllm_seq_ssm& a = L.ssm;
@@ -287,6 +298,7 @@ static int validate(const kllm_seq_desc* d) {
       !d->embed || !d->head || !d->final_norm.w || d->max_tokens <= 0 || d->max_seqs <= 0)
     return KLLM_E_INVALID;
   if (d->dtype != KLLM_SEQ_F32 && d->dtype != KLLM_SEQ_BF16) return KLLM_E_INVALID;
+  if (d->bigram && (d->bigram_buckets <= 0 || d->bigram_mul_prev < 0 || d->bigram_mul_cur < 0)) return KLLM_E_INVALID;
   for (int r = 0; r < d->n_runs; ++r) {
     if (d->run_layer[r] < 0 || d->run_layer[r] >= d->n_layers) return KLLM_E_INVALID;
     if (d->run_add && d->run_add[r] >= 0 && !d->run_vectors) return KLLM_E_INVALID;
@@ -590,9 +602,9 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
   for (int i = 0; i < n_want; ++i)
     if (want_host[i] < 0 || want_host[i] >= T) return KLLM_E_INVALID;
 
-  // layout of the index block (int32): tokens[T] tok_seq[T] tok_pos[T] ent_first[E] ent_count[E] ent_seq[E] ent_pos0[E]
+  // layout of the index block (int32): tokens[T] tok_seq[T] tok_pos[T] prev_token[T] ent_first[E] ent_count[E] ent_seq[E] ent_pos0[E]
   // want[n_want]
-  const size_t n_idx = 3 * static_cast<size_t>(T) + 4 * static_cast<size_t>(n_entries) + static_cast<size_t>(n_want);
+  const size_t n_idx = 4 * static_cast<size_t>(T) + 4 * static_cast<size_t>(n_entries) + static_cast<size_t>(n_want);
   if (n_idx > e->pinned_cap) {
     if (e->pinned) cudaFreeHost(e->pinned);
     e->pinned = nullptr;
@@ -602,15 +614,19 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
   }
   RC(e->idx.reserve(n_idx * sizeof(int32_t)));
   int32_t* hp = e->pinned;
-  int32_t *h_tok = hp, *h_seq = hp + T, *h_pos = hp + 2 * T, *h_first = hp + 3 * T, *h_count = h_first + n_entries,
+  int32_t *h_tok = hp, *h_seq = hp + T, *h_pos = hp + 2 * T, *h_prev = hp + 3 * T, *h_first = hp + 4 * T, *h_count = h_first + n_entries,
           *h_eseq = h_count + n_entries, *h_pos0 = h_eseq + n_entries, *h_want = h_pos0 + n_entries;
   std::memcpy(h_tok, tokens_host, static_cast<size_t>(T) * sizeof(int32_t));
   int at = 0;
   for (int i = 0; i < n_entries; ++i) {
     kllm_seq_engine::Slot& s = e->slots[seqs[i]];
     h_first[i] = at, h_count[i] = counts[i], h_eseq[i] = seqs[i], h_pos0[i] = s.len;
-    for (int j = 0; j < counts[i]; ++j) h_seq[at + j] = seqs[i], h_pos[at + j] = s.len + j;
+    for (int j = 0; j < counts[i]; ++j) {
+      h_seq[at + j] = seqs[i], h_pos[at + j] = s.len + j;
+      h_prev[at + j] = j > 0 ? tokens_host[at + j - 1] : s.last;
+    }
     at += counts[i];
+    s.last = tokens_host[at - 1];
     const int new_len = s.len + counts[i];
     const int pages = (new_len + e->page - 1) / e->page;
     int32_t* row = e->table_host.data() + static_cast<size_t>(seqs[i]) * e->table_stride;
@@ -627,7 +643,7 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
   // the table rows above are pageable host memory: the copies are staged by the driver before the call returns
   CU(cudaMemcpyAsync(e->idx.p, hp, n_idx * sizeof(int32_t), cudaMemcpyHostToDevice, st));
   const int32_t* d_tok = static_cast<const int32_t*>(e->idx.p);
-  const int32_t *d_seq = d_tok + T, *d_pos = d_tok + 2 * T, *d_first = d_tok + 3 * T, *d_count = d_first + n_entries,
+  const int32_t *d_seq = d_tok + T, *d_pos = d_tok + 2 * T, *d_prev = d_tok + 3 * T, *d_first = d_tok + 4 * T, *d_count = d_first + n_entries,
                 *d_eseq = d_count + n_entries, *d_pos0 = d_eseq + n_entries, *d_want = d_pos0 + n_entries;
 
   // ---- workspaces ----------------------------------------------------------------------------------------------
@@ -641,13 +657,17 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
       while (splits < want) splits *= 2;  // a power of two: few distinct launch shapes as a context grows
     }
   }
-  // a layer with a window never has more key tiles in reach than the window spans: a function of `splits` and the
+  // a layer with a window or chunks never has more key tiles in reach than these span: a function of `splits` and the
   // layer's constants only, so that captured decode steps stay keyed by `splits`
-  auto window_splits = [&](int window) {
-    if (window <= 0) return splits;
+  auto reach_splits = [&](int reach) {
+    if (reach <= 0) return splits;
     int cap = 1;
-    while (cap < window / kAttnKeys + 2) cap *= 2;
+    while (cap < reach / kAttnKeys + 2) cap *= 2;
     return std::min(splits, cap);
+  };
+  auto attn_splits = [&](const kllm_seq_attention& a) {
+    if (a.keep_first > 0) return splits;
+    return reach_splits(a.window > 0 && a.chunk > 0 ? std::min(a.window, a.chunk) : std::max(a.window, a.chunk));
   };
   const size_t Ts = static_cast<size_t>(T);
   RC(e->x.reserve(Ts * W * 4));
@@ -726,7 +746,8 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
   e->mark(-1);
   auto run_device = [&]() -> int {
   RC(launch_embed(dtype, d.embed, d_tok, x, e->any_run_embed ? static_cast<float*>(e->x0.p) : nullptr, nw(d.embed_norm),
-                  d.norm_eps, d.embed_scale, T, W, st));
+                  d.norm_eps, d.embed_scale, BigramArgs{d.bigram, d_prev, d.bigram_mul_prev, d.bigram_mul_cur, d.bigram_buckets}, T, W,
+                  st));
   e->mark(KLLM_SEQ_PHASE_NORM);
   // What comes ahead of run r's mixer rides on one norm kernel (`a` may already carry the end of the run before):
   // the embedding output and the run's vector are added, the pre-norm is taken, and the token shift is applied -- inside
@@ -777,10 +798,10 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
       }
       e->mark(KLLM_SEQ_PHASE_QK_PREPARE);
       RC(launch_attention(dtype, shape, e->q.p, static_cast<const float*>(e->gates.p), kv, n_entries, d_first, d_count,
-                          d_eseq, d_pos0, max_count, max_ctx, window_splits(A.keep_first > 0 ? 0 : A.window),
+                          d_eseq, d_pos0, max_count, max_ctx, attn_splits(A),
                           static_cast<float*>(e->ws.p), e->att.p, T, d_seq, d_pos, st));
       if (A.differential)
-        RC(launch_diff_merge(dtype, shape, window_splits(A.keep_first > 0 ? 0 : A.window), static_cast<const float*>(e->ws.p),
+        RC(launch_diff_merge(dtype, shape, attn_splits(A), static_cast<const float*>(e->ws.p),
                              static_cast<const float*>(e->gates.p), A.diff_lambda, A.diff_out_scale, d.norm_eps, e->att.p, T,
                              st));
       e->mark(KLLM_SEQ_PHASE_ATTENTION);
@@ -843,7 +864,7 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
       // steps of single tokens merge the key splits and apply W_uv in one kernel
       const bool fused_merge = single && T <= 32;
       const AttnShape shape{A.heads, 1, krow, A.kv_rank, A.scale, 0.f, 0, 0, A.gate, A.window, A.sink, 1, 1, fused_merge ? 1 : 0};
-      const int lsplits = window_splits(A.window);
+      const int lsplits = reach_splits(A.window);
       RC(launch_attention(dtype, shape, e->qa.p, gates, kv, n_entries, d_first, d_count, d_eseq, d_pos0, max_count, max_ctx,
                           lsplits, static_cast<float*>(e->ws.p), e->ol.p, T, d_seq, d_pos, st));
       if (fused_merge)
@@ -857,12 +878,16 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
       }
     } else if (kind == KLLM_SEQ_MIXER_LINEAR) {
       const kllm_seq_linear& A = L.linear;
-      RC(gemm(dtype, e->h.p, A.w_in, proj, T, W, 2 * A.heads * (A.dim + A.vdim), st));
+      const int row = 2 * A.heads * (A.dim + A.vdim);
+      RC(gemm(dtype, e->h.p, A.w_in, proj, T, W, row, st));
       e->mark(KLLM_SEQ_PHASE_IN_PROJ);
-      RC(launch_linear_attention(A.heads, A.dim, A.vdim, A.decay, proj, e->linear_state[r], n_entries, d_first, d_count,
-                                 d_eseq, d_pos0, max_count, static_cast<float*>(e->ws.p), static_cast<float*>(e->ol.p), st));
-      RC(launch_linear_out(dtype, A.heads, A.dim, A.vdim, static_cast<const float*>(e->ol.p), proj, A.out_norm_w, d.norm_eps,
-                           e->att.p, T, st));
+      if (linear_attention_rotates(A, max_count)) {
+        RC(launch_linear_rotate(A, proj, row, d_pos, T, st));
+        e->mark(KLLM_SEQ_PHASE_QK_PREPARE);
+      }
+      RC(launch_linear_attention(A, proj, row, e->linear_state[r], n_entries, d_first, d_count, d_eseq, d_pos0, max_count,
+                                 static_cast<float*>(e->ws.p), static_cast<float*>(e->ol.p), st));
+      RC(launch_linear_out(dtype, A, static_cast<const float*>(e->ol.p), proj, row, d.norm_eps, e->att.p, T, st));
       e->mark(KLLM_SEQ_PHASE_ATTENTION);
       RC(gemm(dtype, e->att.p, A.w_out, yout, T, A.heads * A.vdim, W, st));
       e->mark(KLLM_SEQ_PHASE_OUT_PROJ);
@@ -921,12 +946,12 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
     if (L.ff_kind == KLLM_SEQ_FF_DENSE) {
       const kllm_seq_dense& F = L.dense;
       if (dense_gated(F)) {
-        RC(gemm_gated(dtype, e->h.p, F.up, e->att.p, T, W, F.ff, GatedAct{F.act, 0.f, 0.f}, st));
+        RC(gemm_gated(dtype, e->h.p, F.up, e->att.p, T, W, F.ff, GatedAct{F.act, F.act_a, F.act_b}, st, F.up_bias));
       } else {
-        RC(gemm(dtype, e->h.p, F.up, proj, T, W, F.ff, st));
+        RC(gemm(dtype, e->h.p, F.up, proj, T, W, F.ff, st, F.up_bias));
         RC(launch_activation(dtype, F.act, F.act_a, F.act_b, proj, e->att.p, Ts * F.ff, st));
       }
-      RC(gemm(dtype, e->att.p, F.down, yout, T, F.ff, W, st));
+      RC(gemm(dtype, e->att.p, F.down, yout, T, F.ff, W, st, F.down_bias));
       e->mark(KLLM_SEQ_PHASE_EXPERTS);
       return 0;
     }

@@ -59,7 +59,17 @@ struct AttnShape {
   // Attention maps that share values: v_share consecutive key heads read the values of ONE value head (key head g reads
   // value head g / v_share; the value rows hold kv_heads / v_share heads).  `heads` and `kv_heads` count the maps.  0: 1.
   int v_share;
+  int chunk;        // > 0: position i sees j only inside its own chunk of this many positions
 };
+// The first position that position p sees (kept first positions aside); it never falls as p grows.
+inline __host__ __device__ int first_seen(const AttnShape& a, int p) {
+  int lo = a.window > 0 && p >= a.window ? p - a.window + 1 : 0;
+  if (a.chunk > 0) {
+    const int c = p - p % a.chunk;
+    lo = c > lo ? c : lo;
+  }
+  return lo;
+}
 inline __host__ __device__ int v_share_of(const AttnShape& a) { return a.v_share > 1 ? a.v_share : 1; }
 // floats of one token's output gates: none, one per head, or one per output element (heads count maps; gates do not)
 inline __host__ __device__ int gate_floats(const AttnShape& a) {
@@ -93,9 +103,16 @@ __host__ __device__ inline float gated_act(const GatedAct& a, float g, float u) 
 }
 
 // ---- seq_kernels.cu -----------------------------------------------------------------------------------------------
-// x[t] = norm(table[tokens[t]] * scale) (norm.w == null: the scaled row itself); `copy` (optional) receives the same rows
+// x[t] = norm(table[tokens[t]] * scale + bigram row) (norm.w == null: the sum itself); `copy` (optional) receives the same rows.
+// Bigram rows (optional): see kllm_seq_desc; prev[t] is the token before tokens[t] in its sequence, -1 for a first token.
+struct BigramArgs {
+  const void* table;    // [buckets + 1][width] or null
+  const int32_t* prev;
+  int64_t mul_prev, mul_cur;
+  int buckets;
+};
 int launch_embed(int dtype, const void* table, const int32_t* tokens, float* x, float* copy, const NormW& norm, float eps,
-                 float scale, int T, int width, cudaStream_t s);
+                 float scale, const BigramArgs& bigram, int T, int width, cudaStream_t s);
 
 // x += N(c1 y1 + s2[t] * y2 + c3 y3 + c4 y4; post) (optional; y2, y3, y4 optional; post.w == null: the sum itself);  x += add_rows[t];
 // x += add (a [width] vector, optional);  out = N(x; pre) in the compute type (optional) -- in this order.  `rows` (optional) gathers: row i reads x[rows[i]], and x is then
@@ -238,17 +255,21 @@ int launch_latent_merge_expand(int dtype, const LatentShape& a, int splits, cons
 // ol [T, heads, kv_rank] fp32 (weighted sums of latents) -> out [T, heads * vdim] compute type: W_uv(head) ol
 int launch_latent_expand(int dtype, const LatentShape& a, const float* ol, const void* w_uv, void* out, int T, cudaStream_t s);
 
-// proj [T, 2 * heads * dim + 2 * heads * vdim] fp32: q | k | v | gate rows before their activations.  Runs the recurrence
-// of every entry from its sequence's state ([slots][heads][dim][vdim] fp32; zeros at position 0), writes o [T, heads * vdim]
-// fp32 and the new state.
+// proj [T, row] fp32 (rows `row` floats apart): q | k | v | gate rows (2 * heads * (dim + vdim) floats) before their activations.
+// launch_linear_rotate turns q and k in place (the PLAIN form: rotation, then k *= k_scale); steps with long entries need it
+// ahead of launch_linear_attention (linear_attention_rotates()), which turns the rows of short ones itself.
+bool linear_attention_rotates(const kllm_seq_linear& m, int max_count);
+int launch_linear_rotate(const kllm_seq_linear& m, float* proj, int row, const int32_t* tok_pos, int T, cudaStream_t s);
+// Runs the recurrence of every entry from its sequence's state ([slots][heads][dim][vdim] fp32; zeros at position 0), writes
+// o [T, heads * vdim] fp32 and the new state.
 // Steps with long entries work chunk-parallel through `scratch` (linear_attention_scratch_bytes(); 0: not needed).
 size_t linear_attention_scratch_bytes(int heads, int dim, int vdim, int T, int n_entries, int max_count);
-int launch_linear_attention(int heads, int dim, int vdim, const float* decay, const float* proj, float* state, int n_entries,
+int launch_linear_attention(const kllm_seq_linear& m, const float* proj, int row, float* state, int n_entries,
                             const int32_t* ent_first, const int32_t* ent_count, const int32_t* ent_seq,
                             const int32_t* ent_pos0, int max_count, float* scratch, float* o, cudaStream_t s);
-// out[t] = RMSnorm(o[t]; w) * sigmoid(gate rows of proj[t]) in the compute type
-int launch_linear_out(int dtype, int heads, int dim, int vdim, const float* o, const float* proj, const float* norm_w, float eps,
-                      void* out, int T, cudaStream_t s);
+// out[t] = norm(o[t]) * act(gate rows of proj[t]) in the compute type
+int launch_linear_out(int dtype, const kllm_seq_linear& m, const float* o, const float* proj, int row, float eps, void* out, int T,
+                      cudaStream_t s);
 // out = act(z) element by element (z fp32 [n], out compute type): KLLM_SEQ_ACT_XIELU with (a, b), or KLLM_SEQ_ACT_RELU2
 int launch_activation(int dtype, int act, float a, float b, const float* z, void* out, size_t n, cudaStream_t s);
 // v *= scale (0: 1), then v <- cap * tanh(v / cap) (cap 0: none)
@@ -390,8 +411,9 @@ int launch_ssd_out(int dtype, const kllm_seq_ssd& m, const float* y, const float
 // ---- seq_gemm.cu --------------------------------------------------------------------------------------------------
 // out[T, N] (fp32) = a[T, K] . w[N, K]^T (+ bias[N]), a and w in the compute type, fp32 accumulation.
 int gemm(int dtype, const void* a, const void* w, float* out, int T, int K, int N, cudaStream_t s, const float* bias = nullptr);
-// out[T, ff] (compute type) = gated_act(a . wg^T, a . wu^T), w = [ff gate rows, then ff up rows][K]
-int gemm_gated(int dtype, const void* a, const void* w, void* out, int T, int K, int ff, const GatedAct& act, cudaStream_t s);
+// out[T, ff] (compute type) = gated_act(a . wg^T + bias[f], a . wu^T + bias[ff + f]), w = [ff gate rows, then ff up rows][K]
+int gemm_gated(int dtype, const void* a, const void* w, void* out, int T, int K, int ff, const GatedAct& act, cudaStream_t s,
+               const float* bias = nullptr);
 // != 0 when a bounded wait inside a tensor-core product ran out since the last call (checked after a step's sync)
 int gemm_take_error();
 // Grouped form for the routed experts: block b (of `block` rows) multiplies rows a[row_of(b, i)] with the weights of

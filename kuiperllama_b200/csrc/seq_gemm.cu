@@ -118,7 +118,8 @@ rows_kernel(const AT* __restrict__ a, const AT* __restrict__ w, const float* __r
 // The gated form: a warp owns feature f and streams its gate row and its up row together.
 template <typename AT, int R, bool VEC>
 __global__ void __launch_bounds__(256)
-rows_gated_kernel(const AT* __restrict__ a, const AT* __restrict__ w, AT* __restrict__ out, int T, int K, int N, GatedAct act) {
+rows_gated_kernel(const AT* __restrict__ a, const AT* __restrict__ w, const float* __restrict__ bias, AT* __restrict__ out, int T,
+                  int K, int N, GatedAct act) {
   constexpr int V = Vec16<AT>::N;
   const int lane = threadIdx.x & 31;
   const int n = blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
@@ -164,6 +165,7 @@ rows_gated_kernel(const AT* __restrict__ a, const AT* __restrict__ w, AT* __rest
         }
     }
   }
+  const float bg = bias ? bias[n] : 0.f, bu = bias ? bias[N + n] : 0.f;
 #pragma unroll
   for (int r = 0; r < R; ++r) {
 #pragma unroll
@@ -171,7 +173,7 @@ rows_gated_kernel(const AT* __restrict__ a, const AT* __restrict__ w, AT* __rest
       g[r] += __shfl_xor_sync(0xffffffffu, g[r], o);
       u[r] += __shfl_xor_sync(0xffffffffu, u[r], o);
     }
-    if (lane == 0 && r < T) st_t(out + static_cast<size_t>(r) * N + n, gated_act(act, g[r], u[r]));
+    if (lane == 0 && r < T) st_t(out + static_cast<size_t>(r) * N + n, gated_act(act, g[r] + bg, u[r] + bu));
   }
 }
 
@@ -259,7 +261,7 @@ tiled_kernel(const AT* __restrict__ a, const AT* __restrict__ w, void* __restric
       const int n = n0 + tx * 4 + j;
       if (n >= N) continue;
       if (EPI == 1) {
-        const float g = acc[0][i][j], u = acc[EPI == 1 ? 1 : 0][i][j];
+        const float g = acc[0][i][j] + (bias ? bias[n] : 0.f), u = acc[EPI == 1 ? 1 : 0][i][j] + (bias ? bias[N + n] : 0.f);
         st_t(static_cast<AT*>(out_) + static_cast<size_t>(dst) * N + n, gated_act(act, g, u));
       } else if (EPI == 2) {
         const float u = fmaxf(acc[0][i][j], 0.f);
@@ -303,7 +305,8 @@ int gemm_t(const AT* a, const AT* w, const float* bias, float* out, int T, int K
 }
 
 template <typename AT>
-int gemm_gated_t(const AT* a, const AT* w, AT* out, int T, int K, int N, const GatedAct& act, cudaStream_t s, bool* umma_used) {
+int gemm_gated_t(const AT* a, const AT* w, const float* bias, AT* out, int T, int K, int N, const GatedAct& act, cudaStream_t s,
+                 bool* umma_used) {
   constexpr int V = Vec16<AT>::N;
   if (T <= 8) {
     const bool vec = (K % V) == 0 && (reinterpret_cast<uintptr_t>(a) & 15) == 0 && (reinterpret_cast<uintptr_t>(w) & 15) == 0;
@@ -312,8 +315,8 @@ int gemm_gated_t(const AT* a, const AT* w, AT* out, int T, int K, int N, const G
     const dim3 grid((N + warps - 1) / warps);
 #define KLLM_ROWS(R)                                                                                \
   do {                                                                                              \
-    if (vec) rows_gated_kernel<AT, R, true><<<grid, warps * 32, 0, s>>>(a, w, out, T, K, N, act);    \
-    else rows_gated_kernel<AT, R, false><<<grid, warps * 32, 0, s>>>(a, w, out, T, K, N, act);       \
+    if (vec) rows_gated_kernel<AT, R, true><<<grid, warps * 32, 0, s>>>(a, w, bias, out, T, K, N, act);    \
+    else rows_gated_kernel<AT, R, false><<<grid, warps * 32, 0, s>>>(a, w, bias, out, T, K, N, act);       \
   } while (0)
     if (T <= 1) KLLM_ROWS(1);
     else if (T <= 2) KLLM_ROWS(2);
@@ -325,10 +328,10 @@ int gemm_gated_t(const AT* a, const AT* w, AT* out, int T, int K, int N, const G
   }
   if (umma::usable<AT>(a, w, T, K, N)) {
     *umma_used = true;
-    return umma::launch_gated(a, w, out, T, K, N, act, s);
+    return umma::launch_gated(a, w, bias, out, T, K, N, act, s);
   }
   const dim3 grid((N + TN - 1) / TN, (T + TM - 1) / TM);
-  tiled_kernel<AT, false, 1><<<grid, 256, 0, s>>>(a, w, out, T, K, N, nullptr, nullptr, 1, act);
+  tiled_kernel<AT, false, 1><<<grid, 256, 0, s>>>(a, w, out, T, K, N, nullptr, nullptr, 1, act, bias);
   count_launch();
   return cuda_rc(cudaGetLastError());
 }
@@ -362,13 +365,14 @@ int gemm(int dtype, const void* a, const void* w, float* out, int T, int K, int 
   return KLLM_E_INVALID;
 }
 
-int gemm_gated(int dtype, const void* a, const void* w, void* out, int T, int K, int ff, const GatedAct& act, cudaStream_t s) {
+int gemm_gated(int dtype, const void* a, const void* w, void* out, int T, int K, int ff, const GatedAct& act, cudaStream_t s,
+               const float* bias) {
   if (!a || !w || !out || T <= 0 || K <= 0 || ff <= 0) return KLLM_E_INVALID;
   if (dtype == KLLM_SEQ_F32)
-    return gemm_gated_t(static_cast<const float*>(a), static_cast<const float*>(w), static_cast<float*>(out), T, K, ff, act, s,
+    return gemm_gated_t(static_cast<const float*>(a), static_cast<const float*>(w), bias, static_cast<float*>(out), T, K, ff, act, s,
                         &g_umma_used);
   if (dtype == KLLM_SEQ_BF16)
-    return gemm_gated_t(static_cast<const __nv_bfloat16*>(a), static_cast<const __nv_bfloat16*>(w),
+    return gemm_gated_t(static_cast<const __nv_bfloat16*>(a), static_cast<const __nv_bfloat16*>(w), bias,
                         static_cast<__nv_bfloat16*>(out), T, K, ff, act, s, &g_umma_used);
   return KLLM_E_INVALID;
 }

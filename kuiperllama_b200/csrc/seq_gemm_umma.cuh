@@ -1,7 +1,7 @@
 // bf16 token-block product on the 5th-generation tensor cores (sm_100a):
 //     out[T, N] (fp32) = a[T, K] (bf16) . w[N, K]^T (bf16) (+ bias[N]), fp32 accumulation in TMEM
 // and its gated form: w holds N gate rows, then N up rows; both accumulate side by side in TMEM and
-//     out[T, N] (bf16) = gated_act(a . gate^T, a . up^T)
+//     out[T, N] (bf16) = gated_act(a . gate^T (+ bias[n]), a . up^T (+ bias[N + n]))
 //
 // One CTA computes 128 weight rows x BN tokens.  The weight rows are the M side of tcgen05.mma (so an accumulator lane
 // is an output feature and a column is a token), the tokens the N side.  Six warps:
@@ -178,7 +178,8 @@ umma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ C
     if (mbar_wait(smem_u32(tmem_full), 0u, stop)) {
       asm volatile("tcgen05.fence::after_thread_sync;" ::: "memory");
       const int row = n0 + quarter * 32 + lane;
-      const float add = !GATED && bias != nullptr && row < N ? bias[row] : 0.f;
+      const float add = bias != nullptr && row < N ? bias[row] : 0.f;  // gated: the gate row's
+      const float add_up = GATED && bias != nullptr && row < N ? bias[N + row] : 0.f;
 #pragma unroll 1
       for (int c = 0; c < BN; c += 32) {
         uint32_t r[32], u[GATED ? 32 : 1];
@@ -193,7 +194,7 @@ umma_kernel(const __grid_constant__ CUtensorMap map_w, const __grid_constant__ C
             if (t >= T) continue;
             if constexpr (GATED)
               static_cast<__nv_bfloat16*>(out_)[static_cast<size_t>(t) * N + row] =
-                  __float2bfloat16_rn(gated_act(act, __uint_as_float(r[j]), __uint_as_float(u[j])));
+                  __float2bfloat16_rn(gated_act(act, __uint_as_float(r[j]) + add, __uint_as_float(u[j]) + add_up));
             else
               static_cast<float*>(out_)[static_cast<size_t>(t) * N + row] = __uint_as_float(r[j]) + add;
           }
@@ -426,13 +427,13 @@ inline int launch<__nv_bfloat16>(const __nv_bfloat16* a, const __nv_bfloat16* w,
 
 // w: [2 * N, K], gate rows then up rows; two weight tiles share a token tile, so a CTA computes 128 features x BN tokens twice
 template <typename AT>
-inline int launch_gated(const AT*, const AT*, AT*, int, int, int, const GatedAct&, cudaStream_t) { return KLLM_E_UNSUPPORTED; }
+inline int launch_gated(const AT*, const AT*, const float*, AT*, int, int, int, const GatedAct&, cudaStream_t) { return KLLM_E_UNSUPPORTED; }
 template <>
-inline int launch_gated<__nv_bfloat16>(const __nv_bfloat16* a, const __nv_bfloat16* w, __nv_bfloat16* out, int T, int K, int N,
-                                       const GatedAct& act, cudaStream_t s) {
+inline int launch_gated<__nv_bfloat16>(const __nv_bfloat16* a, const __nv_bfloat16* w, const float* bias, __nv_bfloat16* out, int T,
+                                       int K, int N, const GatedAct& act, cudaStream_t s) {
   const int feature_tiles = (N + BM - 1) / BM;
-  if (T <= 64 || feature_tiles * ((T + 127) / 128) < kSms) return launch_bn<64, true, 4>(a, w, nullptr, out, T, K, N, act, s);
-  return launch_bn<128, true, 2>(a, w, nullptr, out, T, K, N, act, s);
+  if (T <= 64 || feature_tiles * ((T + 127) / 128) < kSms) return launch_bn<64, true, 4>(a, w, bias, out, T, K, N, act, s);
+  return launch_bn<128, true, 2>(a, w, bias, out, T, K, N, act, s);
 }
 
 inline bool grouped_usable(int K, int N) {

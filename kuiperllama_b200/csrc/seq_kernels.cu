@@ -154,19 +154,29 @@ __device__ __forceinline__ void row_stats(const float* buf, int W, int kind, flo
 
 template <typename AT>
 __global__ void embed_kernel(const AT* __restrict__ table, const int32_t* __restrict__ tokens, float* __restrict__ x,
-                             float* __restrict__ copy, NormW norm, float eps, float scale, int width) {
+                             float* __restrict__ copy, NormW norm, float eps, float scale, BigramArgs bi, int width) {
   extern __shared__ float buf[];
   __shared__ float red[33];
   const int t = blockIdx.x;
   const AT* row = table + static_cast<size_t>(tokens[t]) * width;
-  if (norm.w == nullptr && width % VecOf<AT>::N == 0 && (reinterpret_cast<uintptr_t>(table) & 15) == 0) {
+  const AT* pair = nullptr;  // the bigram's row
+  if (bi.table != nullptr) {
+    const int64_t prev = bi.prev[t];
+    const int64_t b = prev < 0 ? bi.buckets : (prev * bi.mul_prev + tokens[t] * bi.mul_cur) % bi.buckets;
+    pair = static_cast<const AT*>(bi.table) + static_cast<size_t>(b) * width;
+  }
+  if (norm.w == nullptr && width % VecOf<AT>::N == 0 &&
+      ((reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(bi.table)) & 15) == 0) {
     constexpr int V = VecOf<AT>::N;
     for (int i = threadIdx.x * V; i < width; i += blockDim.x * V) {
-      float f[V];
+      float f[V], g[V];
       VecOf<AT>::load(row + i, f);
+      if (pair) VecOf<AT>::load(pair + i, g);
+#pragma unroll
+      for (int j = 0; j < V; ++j) f[j] = f[j] * scale + (pair ? g[j] : 0.f);
 #pragma unroll
       for (int j = 0; j < V; j += 4) {
-        const float4 v = make_float4(f[j] * scale, f[j + 1] * scale, f[j + 2] * scale, f[j + 3] * scale);
+        const float4 v = make_float4(f[j], f[j + 1], f[j + 2], f[j + 3]);
         *reinterpret_cast<float4*>(x + static_cast<size_t>(t) * width + i + j) = v;
         if (copy) *reinterpret_cast<float4*>(copy + static_cast<size_t>(t) * width + i + j) = v;
       }
@@ -175,13 +185,14 @@ __global__ void embed_kernel(const AT* __restrict__ table, const int32_t* __rest
   }
   if (norm.w == nullptr) {
     for (int i = threadIdx.x; i < width; i += blockDim.x) {
-      const float v = to_f(row[i]) * scale;
+      const float v = to_f(row[i]) * scale + (pair ? to_f(pair[i]) : 0.f);
       x[static_cast<size_t>(t) * width + i] = v;
       if (copy) copy[static_cast<size_t>(t) * width + i] = v;
     }
     return;
   }
-  for (int i = threadIdx.x; i < width; i += blockDim.x) buf[i] = to_f(row[i]) * scale;
+  for (int i = threadIdx.x; i < width; i += blockDim.x)
+    buf[i] = to_f(row[i]) * scale + (pair ? to_f(pair[i]) : 0.f);
   __syncthreads();
   float mean, rstd;
   row_stats(buf, width, norm.kind, eps, red, mean, rstd);
@@ -679,11 +690,11 @@ attention_kernel(AttnShape a, const void* __restrict__ q_, PagedKV kv, const int
   const int rows_here = min(kAttnRows, n_rows - r0);
   const int pmax = pos0 + (r0 + rows_here - 1) / rep;  // last position any row of the tile sees
   const int n_tiles = pmax / kAttnKeys + 1;
-  // with a window the first row of the tile sees nothing before its position - window + 1
-  const int tile_first = a.window > 0 ? max(0, pos0 + r0 / rep - a.window + 1) / kAttnKeys : 0;
+  // with a window or chunks no row of the tile sees anything before what its first row sees
+  const int tile_first = first_seen(a, pos0 + r0 / rep) / kAttnKeys;
   // tiles before the window that hold kept first positions come ahead of the window's tiles: the list of this CTA's
   // tiles is [0, keep_tiles) then [tile_first, n_tiles), cut into `splits` parts
-  const int keep_tiles = a.window > 0 ? min(tile_first, (a.keep_first + kAttnKeys - 1) / kAttnKeys) : 0;
+  const int keep_tiles = min(tile_first, (a.keep_first + kAttnKeys - 1) / kAttnKeys);
   const int list_n = keep_tiles + n_tiles - tile_first;
   const int per = (list_n + splits - 1) / splits;
   const int tile_lo = split * per, tile_hi = min(list_n, tile_lo + per);
@@ -819,7 +830,7 @@ attention_kernel(AttnShape a, const void* __restrict__ q_, PagedKV kv, const int
         if (SPARSE && i >= my_rows) break;  // the softmax below reads only rows that exist
         const int r = rg * rpt + i;
         const int pr = pos0 + (r0 + r) / rep;
-        const bool visible = r < rows_here && kj <= pr && (a.window == 0 || pr - kj < a.window || kj < a.keep_first);
+        const bool visible = r < rows_here && kj <= pr && (kj >= first_seen(a, pr) || kj < a.keep_first);
         float sv = sc[i];
         if (a.softcap > 0.f) sv = a.softcap * tanhf(sv / a.softcap);
         Ss[r * kAttnKeys + key] = visible ? sv : -INFINITY;
@@ -918,8 +929,8 @@ attention_wide_kernel(AttnShape a, const void* __restrict__ q_, PagedKV kv, cons
   }
   for (int d = tid; d < a.vdim; d += kAttnThreads) acc[d] = 0.f;
   // visible keys: [0, kept) and [lo, pos], cut into `splits` parts
-  const int lo = a.window > 0 ? max(0, pos - a.window + 1) : 0;
-  const int kept = a.window > 0 ? min(lo, a.keep_first) : 0;
+  const int lo = first_seen(a, pos);
+  const int kept = min(lo, a.keep_first);
   const int n_keys = kept + pos - lo + 1, per = (n_keys + splits - 1) / splits;
   const int first = split * per, last = min(n_keys, first + per);
   const int32_t* table = kv.table + static_cast<size_t>(tok_seq[t]) * kv.table_stride;
@@ -1278,12 +1289,12 @@ inline int done() {
 }  // namespace
 
 int launch_embed(int dtype, const void* table, const int32_t* tokens, float* x, float* copy, const NormW& norm, float eps,
-                 float scale, int T, int width, cudaStream_t s) {
+                 float scale, const BigramArgs& bigram, int T, int width, cudaStream_t s) {
   if (scale == 0.f) scale = 1.0f;
   const size_t smem = static_cast<size_t>(width) * sizeof(float);
   if (smem > 48 * 1024) return KLLM_E_UNSUPPORTED;
   KLLM_SEQ_DISPATCH(dtype, (embed_kernel<AT><<<T, 128, smem, s>>>(static_cast<const AT*>(table), tokens, x, copy, norm, eps,
-                                                                 scale, width)));
+                                                                 scale, bigram, width)));
   return done();
 }
 

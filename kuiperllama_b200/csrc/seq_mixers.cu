@@ -423,7 +423,55 @@ latent_merge_expand_kernel(LatentShape a, int splits, const float* __restrict__ 
 // tokens with the state S before it:
 //     o_i = l^(i+1) S^T q_i + sum_(j <= i) l^(i-j) (q_i . k_j) v_j
 //     S  <- l^n S + sum_j l^(n-1-j) k_j v_j^T
-// Only non-negative powers of l appear.  Everything is fp32; silu is applied to q, k, v as they are loaded.
+// Only non-negative powers of l appear.  Everything is fp32; SILU is applied to q, k, v as they are loaded.  The form without
+// the activation rotates q and k and scales k: steps of short entries do it on the rows in shared memory (`rot`), steps of long
+// ones in place in the projection, before the chunk kernels read them (linear_rotate_kernel).
+template <bool SILU> __device__ __forceinline__ float lin_act(float v) { return SILU ? siluf(v) : v; }
+struct LinearRot {
+  RopeArgs rope;   // dims == 0: none
+  float k_scale;
+};
+__device__ __forceinline__ void rope_turn(const RopeArgs& r, int i, int pos, float& co, float& si) {
+  const float f = r.freq ? r.freq[i] : powf(r.base, -2.0f * static_cast<float>(i) / static_cast<float>(r.dims));
+  const float a = static_cast<float>(pos) * f;
+  co = cosf(a), si = sinf(a);
+}
+
+// One CTA per token: the angles of its position once, then every q and k head, V pairs at a time.
+template <int V>
+__global__ void linear_rotate_kernel(int heads, int dim, LinearRot rot, float* __restrict__ proj, int stride,
+                                     const int32_t* __restrict__ tok_pos) {
+  extern __shared__ __align__(16) float turn[];  // [half] cos, [half] sin
+  const int t = blockIdx.x, half = rot.rope.dims / 2;
+  float* co = turn;
+  float* si = turn + half;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) rope_turn(rot.rope, i, tok_pos[t], co[i], si[i]);
+  __syncthreads();
+  float* row = proj + static_cast<size_t>(t) * stride;
+  const bool pairs = rot.rope.pairing == KLLM_SEQ_ROPE_PAIRS;
+  const int per = half / V;
+  for (int i = threadIdx.x; i < 2 * heads * per; i += blockDim.x) {
+    const int u = i / per, p0 = (i % per) * V;
+    const float ks = u < heads ? 1.0f : rot.k_scale;
+    float* h = row + u * dim;
+    if constexpr (V == 4) {  // halves only
+      float4 a = *reinterpret_cast<float4*>(h + p0), b = *reinterpret_cast<float4*>(h + half + p0);
+      const float4 c = *reinterpret_cast<const float4*>(co + p0), z = *reinterpret_cast<const float4*>(si + p0);
+      *reinterpret_cast<float4*>(h + p0) = make_float4((a.x * c.x - b.x * z.x) * ks, (a.y * c.y - b.y * z.y) * ks,
+                                                       (a.z * c.z - b.z * z.z) * ks, (a.w * c.w - b.w * z.w) * ks);
+      *reinterpret_cast<float4*>(h + half + p0) = make_float4((b.x * c.x + a.x * z.x) * ks, (b.y * c.y + a.y * z.y) * ks,
+                                                              (b.z * c.z + a.z * z.z) * ks, (b.w * c.w + a.w * z.w) * ks);
+    } else {
+      const int d0 = pairs ? 2 * p0 : p0, d1 = pairs ? 2 * p0 + 1 : p0 + half;
+      const float a = h[d0], b = h[d1];
+      h[d0] = (a * co[p0] - b * si[p0]) * ks;
+      h[d1] = (b * co[p0] + a * si[p0]) * ks;
+    }
+  }
+  const int rest = dim - 2 * half;  // coordinates that are not rotated
+  if (rest > 0 && rot.k_scale != 1.0f)
+    for (int i = threadIdx.x; i < heads * rest; i += blockDim.x) row[(heads + i / rest) * dim + 2 * half + i % rest] *= rot.k_scale;
+}
 // Fill shared memory from global memory with U loads of a thread in flight before the first is used: the tiles of these
 // kernels are small and each CTA waits for them once, so the loop is bound by load latency, not by bandwidth.
 template <int U, typename Load, typename Store>
@@ -448,9 +496,10 @@ constexpr int kLinCols = 32;
 constexpr int kLinThreads = 128;
 constexpr int kLinParallelFrom = 2 * kLinChunk;  // steps whose longest entry has more tokens take the chunk-parallel kernels
 
+template <bool SILU>
 __global__ void __launch_bounds__(kLinThreads)
-linear_attention_kernel(int heads, int dim, int vdim, const float* __restrict__ decay, const float* __restrict__ proj,
-                        float* __restrict__ state, const int32_t* __restrict__ ent_first,
+linear_attention_kernel(int heads, int dim, int vdim, const float* __restrict__ decay, LinearRot rot,
+                        const float* __restrict__ proj, int stride, float* __restrict__ state, const int32_t* __restrict__ ent_first,
                         const int32_t* __restrict__ ent_count, const int32_t* __restrict__ ent_seq,
                         const int32_t* __restrict__ ent_pos0, float* __restrict__ o) {
   extern __shared__ float sm[];
@@ -474,19 +523,34 @@ linear_attention_kernel(int heads, int dim, int vdim, const float* __restrict__ 
                  [&](int i) { return (!fresh && i % kLinCols < cols) ? sg[static_cast<size_t>(i / kLinCols) * vdim + c0 + i % kLinCols] : 0.f; },
                  [&](int i, float v) { Ss[i] = v; });
   const int qn = heads * dim, vn = heads * vdim;
-  const int stride = 2 * qn + 2 * vn;
+  const bool turned = !SILU && (rot.rope.dims > 0 || rot.k_scale != 1.0f);
   for (int base = 0; base < count; base += kLinChunk) {
     const int n = min(kLinChunk, count - base);
     __syncthreads();  // the previous chunk's tiles are no longer read; Ss / pw are written
     const float* rows = proj + static_cast<size_t>(first + base) * stride;
     staged_fill<8>(n * dim, [&](int i) { return rows[static_cast<size_t>(i / dim) * stride + h * dim + i % dim]; },
-                   [&](int i, float v) { Qs[(i / dim) * dp + i % dim] = siluf(v); });
+                   [&](int i, float v) { Qs[(i / dim) * dp + i % dim] = lin_act<SILU>(v); });
     staged_fill<8>(n * dim, [&](int i) { return rows[static_cast<size_t>(i / dim) * stride + qn + h * dim + i % dim]; },
-                   [&](int i, float v) { Ks[(i / dim) * dp + i % dim] = siluf(v); });
+                   [&](int i, float v) { Ks[(i / dim) * dp + i % dim] = lin_act<SILU>(v); });
     staged_fill<8>(n * kLinCols,
                    [&](int i) { return i % kLinCols < cols ? rows[static_cast<size_t>(i / kLinCols) * stride + 2 * qn + h * vdim + c0 + i % kLinCols] : 0.f; },
-                   [&](int i, float v) { Vs[i] = siluf(v); });
+                   [&](int i, float v) { Vs[i] = lin_act<SILU>(v); });
     __syncthreads();
+    if (turned) {
+      const int half = rot.rope.dims / 2, rest = dim - 2 * half;
+      const bool pairs = rot.rope.pairing == KLLM_SEQ_ROPE_PAIRS;
+      for (int i = tid; i < n * half; i += kLinThreads) {
+        const int r = i / half, p = i % half;
+        float co, si;
+        rope_turn(rot.rope, p, ent_pos0[e] + base + r, co, si);
+        const int d0 = r * dp + (pairs ? 2 * p : p), d1 = r * dp + (pairs ? 2 * p + 1 : p + half);
+        const float q0 = Qs[d0], q1 = Qs[d1], k0 = Ks[d0], k1 = Ks[d1];
+        Qs[d0] = q0 * co - q1 * si, Qs[d1] = q1 * co + q0 * si;
+        Ks[d0] = (k0 * co - k1 * si) * rot.k_scale, Ks[d1] = (k1 * co + k0 * si) * rot.k_scale;
+      }
+      for (int i = tid; i < n * rest; i += kLinThreads) Ks[(i / rest) * dp + 2 * half + i % rest] *= rot.k_scale;
+      __syncthreads();
+    }
     for (int i = tid; i < n * n; i += kLinThreads) {  // decayed scores inside the chunk
       const int r = i / n, j = i % n;
       float acc = 0.f;
@@ -532,8 +596,10 @@ __host__ __device__ inline int lin_dp(int dim) { return ((dim + 3) & ~3) + 4; } 
 
 // A thread keeps 8 consecutive key coordinates of one value column: two 16-byte broadcast loads and one column load
 // feed 8 multiply-adds.
+template <bool SILU>
 __global__ void __launch_bounds__(kLinThreads)
 linear_chunk_sums_kernel(int heads, int dim, int vdim, const float* __restrict__ decay, const float* __restrict__ proj,
+                         int stride,
                          const int32_t* __restrict__ ent_first, const int32_t* __restrict__ ent_count,
                          float* __restrict__ sums) {
   extern __shared__ __align__(16) float sm[];
@@ -549,18 +615,18 @@ linear_chunk_sums_kernel(int heads, int dim, int vdim, const float* __restrict__
   float* Vs = Ks + kLinChunk * dp;      // [chunk][kLinCols]
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const float llog = logf(decay[h]);
-  const int qn = heads * dim, vn = heads * vdim, stride = 2 * qn + 2 * vn;
+  const int qn = heads * dim;
   const float* rows = proj + static_cast<size_t>(first + base) * stride;
   staged_fill<8>(n * d8,
                  [&](int i) { return i % d8 < dim ? rows[static_cast<size_t>(i / d8) * stride + qn + h * dim + i % d8] : 0.f; },
                  [&](int i, float v) {
                    const int j = i / d8;
                    const float w = n - 1 - j == 0 ? 1.0f : expf(llog * static_cast<float>(n - 1 - j));
-                   Ks[j * dp + i % d8] = siluf(v) * w;
+                   Ks[j * dp + i % d8] = lin_act<SILU>(v) * w;
                  });
   staged_fill<8>(n * kLinCols,
                  [&](int i) { return i % kLinCols < cols ? rows[static_cast<size_t>(i / kLinCols) * stride + 2 * qn + h * vdim + c0 + i % kLinCols] : 0.f; },
-                 [&](int i, float v) { Vs[i] = siluf(v); });
+                 [&](int i, float v) { Vs[i] = lin_act<SILU>(v); });
   __syncthreads();
   float* out = sums + (chunk_slot(first, base, e) * heads + h) * dim * vdim;
   for (int d0 = warp * 8; d0 < d8; d0 += (kLinThreads / 32) * 8) {
@@ -618,8 +684,10 @@ __global__ void linear_scan_kernel(int heads, int dim, int vdim, const float* __
 constexpr int kLinAs = kLinChunk + 4;
 
 constexpr int kLinOutThreads = 256, kLinOutWarps = kLinOutThreads / 32;
+template <bool SILU>
 __global__ void __launch_bounds__(kLinOutThreads)
 linear_chunk_out_kernel(int heads, int dim, int vdim, const float* __restrict__ decay, const float* __restrict__ proj,
+                        int stride,
                         const int32_t* __restrict__ ent_first, const int32_t* __restrict__ ent_count,
                         const float* __restrict__ sums, float* __restrict__ o) {
   extern __shared__ __align__(16) float sm[];
@@ -644,18 +712,18 @@ linear_chunk_out_kernel(int heads, int dim, int vdim, const float* __restrict__ 
   staged_fill<8>(d4 * kLinCols,
                  [&](int i) { return (i / kLinCols < dim && i % kLinCols < cols) ? sb[static_cast<size_t>(i / kLinCols) * vdim + c0 + i % kLinCols] : 0.f; },
                  [&](int i, float v) { Ss[i] = v; });
-  const int qn = heads * dim, vn = heads * vdim, stride = 2 * qn + 2 * vn;
+  const int qn = heads * dim, vn = heads * vdim;
   const float* rows = proj + static_cast<size_t>(first + base) * stride;
-  // silu(0) = 0: rows and coordinates past the chunk load as zeros
+  // the activation of 0 is 0: rows and coordinates past the chunk load as zeros
   staged_fill<8>(kLinChunk * d4,
                  [&](int i) { return (i / d4 < n && i % d4 < dim) ? rows[static_cast<size_t>(i / d4) * stride + h * dim + i % d4] : 0.f; },
-                 [&](int i, float v) { Qs[(i / d4) * dp + i % d4] = siluf(v); });
+                 [&](int i, float v) { Qs[(i / d4) * dp + i % d4] = lin_act<SILU>(v); });
   staged_fill<8>(kLinChunk * d4,
                  [&](int i) { return (i / d4 < n && i % d4 < dim) ? rows[static_cast<size_t>(i / d4) * stride + qn + h * dim + i % d4] : 0.f; },
-                 [&](int i, float v) { Ks[(i / d4) * dp + i % d4] = siluf(v); });
+                 [&](int i, float v) { Ks[(i / d4) * dp + i % d4] = lin_act<SILU>(v); });
   staged_fill<8>(kLinChunk * kLinCols,
                  [&](int i) { return (i / kLinCols < n && i % kLinCols < cols) ? rows[static_cast<size_t>(i / kLinCols) * stride + 2 * qn + h * vdim + c0 + i % kLinCols] : 0.f; },
-                 [&](int i, float v) { Vs[i] = siluf(v); });
+                 [&](int i, float v) { Vs[i] = lin_act<SILU>(v); });
   __syncthreads();
   constexpr int R = kLinChunk / kLinOutWarps;  // rows per thread
   {  // decayed scores inside the chunk: lane = key j, rows warp + 8 k
@@ -709,18 +777,34 @@ linear_chunk_out_kernel(int heads, int dim, int vdim, const float* __restrict__ 
   }
 }
 
-template <typename AT>
-__global__ void linear_out_kernel(int qn, int vn, const float* __restrict__ o, const float* __restrict__ proj,
-                                  const float* __restrict__ norm_w, float eps, AT* __restrict__ out) {
+__device__ __forceinline__ float lin_gate(int act, float g) { return act == KLLM_SEQ_GATEACT_SILU ? siluf(g) : sigmoidf(g); }
+
+// One CTA per token.  ROW: one norm over the row; HEAD: a warp per head, each by its own root mean square.
+template <typename AT, bool HEAD>
+__global__ void linear_out_kernel(int heads, int dim, int vdim, const float* __restrict__ o, const float* __restrict__ proj,
+                                  int stride, const float* __restrict__ norm_w, int gate_act, float eps, AT* __restrict__ out) {
   __shared__ float red[33];
-  const int t = blockIdx.x;
+  const int t = blockIdx.x, vn = heads * vdim;
   const float* row = o + static_cast<size_t>(t) * vn;
-  const float* g = proj + static_cast<size_t>(t) * (2 * qn + 2 * vn) + 2 * qn + vn;
-  float ss = 0.f;
-  for (int i = threadIdx.x; i < vn; i += blockDim.x) ss += row[i] * row[i];
-  const float rinv = 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(vn) + eps);
-  for (int i = threadIdx.x; i < vn; i += blockDim.x)
-    out[static_cast<size_t>(t) * vn + i] = from_f<AT>(row[i] * rinv * norm_w[i] * sigmoidf(g[i]));
+  const float* g = proj + static_cast<size_t>(t) * stride + 2 * heads * dim + vn;
+  AT* dst = out + static_cast<size_t>(t) * vn;
+  if constexpr (HEAD) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+    for (int h = warp; h < heads; h += nw) {
+      float ss = 0.f;
+      for (int d = lane; d < vdim; d += 32) ss = fmaf(row[h * vdim + d], row[h * vdim + d], ss);
+      const float rinv = 1.0f / sqrtf(warp_sum(ss) / static_cast<float>(vdim) + eps);
+      for (int d = lane; d < vdim; d += 32) {
+        const int i = h * vdim + d;
+        dst[i] = from_f<AT>(row[i] * rinv * lin_gate(gate_act, g[i]));
+      }
+    }
+  } else {
+    float ss = 0.f;
+    for (int i = threadIdx.x; i < vn; i += blockDim.x) ss += row[i] * row[i];
+    const float rinv = 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(vn) + eps);
+    for (int i = threadIdx.x; i < vn; i += blockDim.x) dst[i] = from_f<AT>(row[i] * rinv * norm_w[i] * lin_gate(gate_act, g[i]));
+  }
 }
 
 // ---- activations ---------------------------------------------------------------------------------------------------------------
@@ -842,52 +926,91 @@ size_t linear_attention_scratch_bytes(int heads, int dim, int vdim, int T, int n
   return (static_cast<size_t>(T) / kLinChunk + n_entries + 1) * heads * dim * vdim * sizeof(float);
 }
 
-int launch_linear_attention(int heads, int dim, int vdim, const float* decay, const float* proj, float* state, int n_entries,
-                            const int32_t* ent_first, const int32_t* ent_count, const int32_t* ent_seq,
-                            const int32_t* ent_pos0, int max_count, float* scratch, float* o, cudaStream_t s) {
-  const size_t smem = (2 * static_cast<size_t>(kLinChunk) * (dim + 1) + kLinChunk * kLinCols + kLinChunk * (kLinChunk + 1) +
-                       static_cast<size_t>(dim) * kLinCols + kLinChunk + 1) * sizeof(float);
-  if (smem > 200 * 1024) return KLLM_E_UNSUPPORTED;
-  static size_t configured = 0;
-  if (smem > 48 * 1024 && smem > configured) {
-    const cudaError_t e = cudaFuncSetAttribute(linear_attention_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                                               static_cast<int>(smem));
-    if (e != cudaSuccess) return cuda_rc(e);
-    configured = smem;
-  }
+static LinearRot linear_rot(const kllm_seq_linear& m) {
+  return LinearRot{RopeArgs{m.rope_dims, m.rope_base, m.rope_freq, 1.0f, m.rope_pairing}, m.k_scale == 0.f ? 1.0f : m.k_scale};
+}
+
+int launch_linear_rotate(const kllm_seq_linear& m, float* proj, int row, const int32_t* tok_pos, int T, cudaStream_t s) {
+  const LinearRot rot = linear_rot(m);
+  const int half = m.rope_dims / 2;
+  const size_t smem = 2 * static_cast<size_t>(half) * sizeof(float);
+  const bool vec = m.rope_pairing == KLLM_SEQ_ROPE_HALVES && half % 4 == 0 && m.dim % 4 == 0 && row % 4 == 0 &&
+                   (reinterpret_cast<uintptr_t>(proj) & 15) == 0;
+  if (vec) linear_rotate_kernel<4><<<T, 256, smem, s>>>(m.heads, m.dim, rot, proj, row, tok_pos);
+  else linear_rotate_kernel<1><<<T, 256, smem, s>>>(m.heads, m.dim, rot, proj, row, tok_pos);
+  return done();
+}
+
+template <bool SILU>
+static int linear_attention_t(const kllm_seq_linear& m, const float* proj, int row, float* state, int n_entries,
+                              const int32_t* ent_first, const int32_t* ent_count, const int32_t* ent_seq,
+                              const int32_t* ent_pos0, int max_count, float* scratch, float* o, cudaStream_t s) {
+  const int heads = m.heads, dim = m.dim, vdim = m.vdim;
+  const float* decay = m.decay;
   if (max_count > kLinParallelFrom && scratch != nullptr) {  // long entries: chunks in parallel
     const size_t smem_out = (2 * static_cast<size_t>(kLinChunk) * lin_dp(dim) + kLinChunk * kLinCols + kLinChunk * kLinAs +
                              static_cast<size_t>((dim + 3) & ~3) * kLinCols + kLinChunk + 4) * sizeof(float);
     static size_t configured_out = 0;
     if (smem_out > 48 * 1024 && smem_out > configured_out) {
-      cudaError_t e = cudaFuncSetAttribute(linear_chunk_out_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize,
+      cudaError_t e = cudaFuncSetAttribute(linear_chunk_out_kernel<SILU>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                                            static_cast<int>(smem_out));
       if (e == cudaSuccess)
-        e = cudaFuncSetAttribute(linear_chunk_sums_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, static_cast<int>(smem_out));
+        e = cudaFuncSetAttribute(linear_chunk_sums_kernel<SILU>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                 static_cast<int>(smem_out));
       if (e != cudaSuccess) return cuda_rc(e);
       configured_out = smem_out;
     }
     const int n_slices = (vdim + kLinCols - 1) / kLinCols, chunks = (max_count + kLinChunk - 1) / kLinChunk;
     const dim3 grid(chunks * n_slices, heads, n_entries);
     const size_t smem_sums = (static_cast<size_t>(kLinChunk) * lin_dp(dim) + kLinChunk * kLinCols) * sizeof(float);
-    linear_chunk_sums_kernel<<<grid, kLinThreads, smem_sums, s>>>(heads, dim, vdim, decay, proj, ent_first, ent_count, scratch);
+    linear_chunk_sums_kernel<SILU><<<grid, kLinThreads, smem_sums, s>>>(heads, dim, vdim, decay, proj, row, ent_first, ent_count,
+                                                                       scratch);
     count_launch();
     const dim3 sgrid((dim * vdim + 127) / 128, heads, n_entries);
     linear_scan_kernel<<<sgrid, 128, 0, s>>>(heads, dim, vdim, decay, state, ent_first, ent_count, ent_seq, ent_pos0, scratch);
     count_launch();
-    linear_chunk_out_kernel<<<grid, kLinOutThreads, smem_out, s>>>(heads, dim, vdim, decay, proj, ent_first, ent_count, scratch, o);
+    linear_chunk_out_kernel<SILU><<<grid, kLinOutThreads, smem_out, s>>>(heads, dim, vdim, decay, proj, row, ent_first, ent_count,
+                                                                        scratch, o);
     return done();
   }
+  const size_t smem = (2 * static_cast<size_t>(kLinChunk) * (dim + 1) + kLinChunk * kLinCols + kLinChunk * (kLinChunk + 1) +
+                       static_cast<size_t>(dim) * kLinCols + kLinChunk + 1) * sizeof(float);
+  if (smem > 200 * 1024) return KLLM_E_UNSUPPORTED;
+  static size_t configured = 0;
+  if (smem > 48 * 1024 && smem > configured) {
+    const cudaError_t e = cudaFuncSetAttribute(linear_attention_kernel<SILU>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                               static_cast<int>(smem));
+    if (e != cudaSuccess) return cuda_rc(e);
+    configured = smem;
+  }
   const dim3 grid((vdim + kLinCols - 1) / kLinCols, heads, n_entries);
-  linear_attention_kernel<<<grid, kLinThreads, smem, s>>>(heads, dim, vdim, decay, proj, state, ent_first, ent_count, ent_seq,
-                                                         ent_pos0, o);
+  linear_attention_kernel<SILU><<<grid, kLinThreads, smem, s>>>(heads, dim, vdim, decay, linear_rot(m), proj, row, state, ent_first,
+                                                               ent_count, ent_seq, ent_pos0, o);
   return done();
 }
 
-int launch_linear_out(int dtype, int heads, int dim, int vdim, const float* o, const float* proj, const float* norm_w, float eps,
-                      void* out, int T, cudaStream_t s) {
-  KLLM_SEQ_DISPATCH(dtype, (linear_out_kernel<AT><<<T, 128, 0, s>>>(heads * dim, heads * vdim, o, proj, norm_w, eps,
-                                                                   static_cast<AT*>(out))));
+bool linear_attention_rotates(const kllm_seq_linear& m, int max_count) {
+  return m.qkv_act == KLLM_SEQ_QKV_PLAIN && max_count > kLinParallelFrom && (m.rope_dims > 0 || (m.k_scale != 0.f && m.k_scale != 1.0f));
+}
+
+int launch_linear_attention(const kllm_seq_linear& m, const float* proj, int row, float* state, int n_entries,
+                            const int32_t* ent_first, const int32_t* ent_count, const int32_t* ent_seq,
+                            const int32_t* ent_pos0, int max_count, float* scratch, float* o, cudaStream_t s) {
+  if (m.qkv_act == KLLM_SEQ_QKV_PLAIN)
+    return linear_attention_t<false>(m, proj, row, state, n_entries, ent_first, ent_count, ent_seq, ent_pos0, max_count, scratch, o, s);
+  return linear_attention_t<true>(m, proj, row, state, n_entries, ent_first, ent_count, ent_seq, ent_pos0, max_count, scratch, o, s);
+}
+
+int launch_linear_out(int dtype, const kllm_seq_linear& m, const float* o, const float* proj, int row, float eps, void* out, int T,
+                      cudaStream_t s) {
+  if (m.out_norm == KLLM_SEQ_OUTNORM_HEAD) {
+    const int threads = T <= 64 ? 512 : 128;
+    KLLM_SEQ_DISPATCH(dtype, (linear_out_kernel<AT, true><<<T, threads, 0, s>>>(m.heads, m.dim, m.vdim, o, proj, row, nullptr, m.gate_act,
+                                                                               eps, static_cast<AT*>(out))));
+    return done();
+  }
+  KLLM_SEQ_DISPATCH(dtype, (linear_out_kernel<AT, false><<<T, 128, 0, s>>>(m.heads, m.dim, m.vdim, o, proj, row, m.out_norm_w,
+                                                                          m.gate_act, eps, static_cast<AT*>(out))));
   return done();
 }
 

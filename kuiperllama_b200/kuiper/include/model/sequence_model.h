@@ -105,6 +105,9 @@ class SequenceModel : public base::NoCopyable {
   float logit_scale_ = 1.0f;
   float embed_scale_ = 1.0f;    // the embedding rows are multiplied by it
   float logit_softcap_ = 0.0f;  // logits <- cap * tanh(logits / cap); 0: none
+  const void* bigram_ = nullptr;  // bigram embedding (kllm_seq_desc.bigram), or none
+  int32_t bigram_buckets_ = 0;
+  int64_t bigram_mul_prev_ = 0, bigram_mul_cur_ = 0;
   int32_t streams_ = 0;         // residual streams joined by hyper-connections; 0: one plain residual
 
  private:

@@ -161,6 +161,7 @@ base::Status SequenceModel::init(const std::string& dir, const SequenceOptions& 
   d.max_tokens = options.max_tokens, d.max_seqs = options.max_seqs, d.page_tokens = options.page_tokens;
   d.embed_norm = embed_norm_, d.logit_scale = logit_scale_;
   d.embed_scale = embed_scale_, d.logit_softcap = logit_softcap_, d.streams = streams_;
+  d.bigram = bigram_, d.bigram_buckets = bigram_buckets_, d.bigram_mul_prev = bigram_mul_prev_, d.bigram_mul_cur = bigram_mul_cur_;
   d.run_embed = run_embed_.size() == run_layer_.size() ? run_embed_.data() : nullptr;
   return engine_status(kllm_seq_create(&d, nullptr, &engine_), "kllm_seq_create");
 }

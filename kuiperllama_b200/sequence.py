@@ -9,7 +9,7 @@ from __future__ import annotations
 
 import ctypes
 import math
-from ctypes import POINTER, c_float, c_int32, c_void_p
+from ctypes import POINTER, c_float, c_int32, c_int64, c_void_p
 from dataclasses import dataclass
 
 F32, BF16 = 0, 1
@@ -28,7 +28,7 @@ class Attention(ctypes.Structure):
                 ("in_bias", c_void_p), ("conv_taps", c_int32), ("conv_w", c_void_p), ("rope_dims", c_int32),
                 ("rope_base", c_float), ("rope_pairing", c_int32), ("values_are_keys", c_int32),
                 ("rope_freq", c_void_p), ("rope_mag", c_float), ("differential", c_int32), ("diff_lambda", c_float),
-                ("diff_out_scale", c_float), ("out_bias", c_void_p), ("v_blend", c_int32), ("v_lambda", c_float)]
+                ("diff_out_scale", c_float), ("out_bias", c_void_p), ("v_blend", c_int32), ("v_lambda", c_float), ("chunk", c_int32)]
 
 
 class Moe(ctypes.Structure):
@@ -50,12 +50,14 @@ class Latent(ctypes.Structure):
 
 class Linear(ctypes.Structure):
     _fields_ = [("heads", c_int32), ("dim", c_int32), ("vdim", c_int32), ("decay", c_void_p), ("w_in", c_void_p),
-                ("out_norm_w", c_void_p), ("w_out", c_void_p)]
+                ("out_norm_w", c_void_p), ("w_out", c_void_p), ("qkv_act", c_int32), ("rope_dims", c_int32),
+                ("rope_base", c_float), ("rope_pairing", c_int32), ("rope_freq", c_void_p), ("k_scale", c_float),
+                ("out_norm", c_int32), ("gate_act", c_int32)]
 
 
 class Dense(ctypes.Structure):
     _fields_ = [("ff", c_int32), ("act", c_int32), ("act_a", c_float), ("act_b", c_float), ("up", c_void_p),
-                ("down", c_void_p)]
+                ("down", c_void_p), ("up_bias", c_void_p), ("down_bias", c_void_p)]
 
 
 class Ssm(ctypes.Structure):
@@ -96,7 +98,8 @@ class Desc(ctypes.Structure):
                 ("run_add", POINTER(c_int32)), ("run_vectors", c_void_p), ("embed", c_void_p), ("final_norm", Norm),
                 ("head", c_void_p), ("max_tokens", c_int32), ("max_seqs", c_int32), ("page_tokens", c_int32),
                 ("embed_norm", Norm), ("run_embed", POINTER(c_int32)), ("logit_scale", c_float), ("embed_scale", c_float),
-                ("logit_softcap", c_float), ("streams", c_int32)]
+                ("logit_softcap", c_float), ("streams", c_int32), ("bigram", c_void_p), ("bigram_buckets", c_int32),
+                ("bigram_mul_prev", c_int64), ("bigram_mul_cur", c_int64)]
 
 
 class SeqError(RuntimeError):
