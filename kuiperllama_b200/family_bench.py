@@ -1,8 +1,9 @@
-"""`bench.py --family fobolorn | kikunex | vurazen | bukuvik | bifazen`: prefill and decode throughput of a batched family (sequence-batch
+"""`bench.py --family fobolorn | kikunex | vurazen | bukuvik | bifazen | mobatar`: prefill and decode throughput of a batched family (sequence-batch
 engine) at sizes that resemble a real model's layers, random weights, beside the closest existing model at equal width,
 heads, active feed-forward size and number of layer runs: Fobolorn beside the Llama family of the single-sequence decoder,
 Kikunex beside Fobolorn, Vurazen beside Kikunex, Bukuvik beside Vurazen, Bifazen beside Kikunex (its latent attention) and
-Fobolorn (its attention).
+Fobolorn (its attention), Mobatar beside Bifazen (its attention), Kikunex (its linear attention) and Fobolorn (causal
+attention).
 
 What is timed.  A step is the call a server makes: kllm_seq_step() with token ids in host memory and the greedy ids
 read back to host memory, blocking -- so every number here is end to end.  Between timed steps a buffer larger than
@@ -20,7 +21,7 @@ import statistics
 import time
 from pathlib import Path
 
-from .sequence import BF16, BifazenShape, BukuvikShape, F32, FobolornShape, KikunexShape, SeqEngine, VurazenShape, load_seq_library
+from .sequence import BF16, BifazenShape, BukuvikShape, F32, FobolornShape, KikunexShape, MobatarShape, SeqEngine, VurazenShape, load_seq_library
 
 ROOT = Path(__file__).resolve().parent.parent
 
@@ -133,6 +134,65 @@ def bifazen_decode_bytes(shape, B, ctx, es):
             "experts": sum(3 * (f or 0) * W for _, f in shape.pattern) * es,
             "attention": shape.state_bytes_per_step(B, ctx, es) +
             sum(shape.heads * shape.vdim * shape.kv_rank for m, _ in shape.pattern if m == "latent") * es,
+            "head": shape.vocab * W * es}
+
+
+# the sizes of BIFAZEN's layers: same width, heads, key/value rank, window and feed-forward in the latent layers, the heads of
+# SIZES over 4 key heads in the causal ones; a pair is a chunked attention of those heads (chunks of 768)
+# beside a retention with the square states of KIKUNEX_SIZES; six layer runs
+_MOBATAR_DIMS = {"s": (1024, 32000, 2048, 16, 4, 64, 64, 16, 4, 64, 64, 768, 16, 64, 64, 16, 64, 32, 64, 128, 512),
+                 "m": (2048, 32000, 4096, 16, 4, 128, 128, 16, 4, 128, 128, 768, 16, 128, 128, 16, 128, 64, 128, 256, 512),
+                 "debug": (256, 4096, 512, 4, 2, 32, 32, 4, 2, 32, 32, 96, 4, 32, 32, 4, 32, 16, 32, 64, 96)}
+
+
+def mobatar_shape(size, kinds, again, tag):
+    w, v, ff, *rest = _MOBATAR_DIMS[size]
+    pattern = tuple(({"A": "attention", "P": "parallel", "L": "latent"}[k], ff) for k in kinds)
+    return MobatarShape(f"mobatar-{size}{tag}", w, v, pattern, tuple(again), *rest)
+
+
+def kikunex_linear_shape(size):
+    """Kikunex with linear attention and a dense feed-forward in all of six layers."""
+    import dataclasses
+    base = KIKUNEX_SIZES[size]
+    return dataclasses.replace(base, name=base.name + "-linear", pattern=(("lightning", "dense"),) * 6, loop=(0, 0, 1))
+
+
+def chunk_pairs(T, chunk):
+    full, rest = divmod(T, chunk)
+    return full * chunk * (chunk + 1) / 2 + rest * (rest + 1) / 2
+
+
+def mobatar_costs(shape, prompt_len):
+    """FLOPs of a prompt step by phase class of the engine's profile: latents in their per-head form (their expansion is counted
+    with the preparation, where the engine runs it), the retention as the recurrence it is (k v^T, the decayed sum, S^T q)."""
+    W, T = shape.width, prompt_len
+    kinds = shape.run_kinds()
+    win = min(shape.window, T)
+    per = {"latent": 2 * (T * win - win * (win - 1) / 2) * shape.l_heads * (shape.l_dim + shape.rot_dim + shape.l_vdim),
+           "attention": T * (T + 1) * shape.heads * (shape.dim + shape.vdim),
+           "parallel": 2 * chunk_pairs(T, shape.chunk) * shape.c_heads * (shape.c_dim + shape.c_vdim) +
+           4 * T * shape.r_heads * shape.r_dim * shape.r_vdim}
+    return {"in_proj": 2 * T * W * sum(shape.n_in(m) for m, _ in kinds),
+            "qk_prepare": 2 * T * sum(shape.expand_elems(m) for m, _ in kinds),
+            "attention": sum(per[m] for m, _ in kinds),
+            "out_proj": 2 * T * W * sum(shape.n_out(m) for m, _ in kinds),
+            "experts": 2 * T * sum(3 * (f or 0) * W for _, f in kinds),
+            "head": 2 * shape.vocab * W}
+
+
+def mobatar_decode_bytes(shape, B, ctx, es):
+    """Bytes a decode step must move, by phase class: weights once per step, keys and values in reach, states."""
+    W = shape.width
+    kinds = shape.run_kinds()
+    n_sub = sum(2 if f else 1 for _, f in kinds)
+    latent = [1 for m, _ in kinds if m == "latent"]
+    return {"norm": n_sub * B * W * 4 * 4,
+            "in_proj": sum(shape.n_in(m) for m, _ in kinds) * W * es,
+            "out_proj": sum(shape.n_out(m) for m, _ in kinds) * W * es,
+            "qk_prepare": len(latent) * shape.l_heads * shape.l_dim * shape.kv_rank * es,
+            "experts": sum(3 * (f or 0) * W for _, f in kinds) * es,
+            "attention": shape.state_bytes_per_step(B, ctx, es) + len(latent) * shape.l_heads * shape.l_vdim * shape.kv_rank * es,
             "head": shape.vocab * W * es}
 
 
@@ -315,7 +375,8 @@ def bench_engine(torch, shape, dtype, prompt_len, ctx, batches, steps, warm, flu
     vura = isinstance(shape, VurazenShape)
     buku = isinstance(shape, BukuvikShape)
     bifa = isinstance(shape, BifazenShape)
-    phase_flops = (bifazen_costs if bifa else bukuvik_costs if buku else vurazen_costs if vura else kikunex_costs if kiku else
+    moba = isinstance(shape, MobatarShape)
+    phase_flops = (mobatar_costs if moba else bifazen_costs if bifa else bukuvik_costs if buku else vurazen_costs if vura else kikunex_costs if kiku else
                    fobolorn_costs)(shape, prompt_len)
     flops = sum(phase_flops.values())
     out["prefill"] = {"tokens": prompt_len, "tok_s": prompt_len / sec, "ms": sec * 1e3, "launches": launches,
@@ -346,10 +407,10 @@ def bench_engine(torch, shape, dtype, prompt_len, ctx, batches, steps, warm, flu
         # bytes a step must read: the active weights (distinct experts per token, an upper bound when tokens share
         # experts) and the cached keys / values
         W = shape.width
-        if vura or buku or bifa:
-            phase_bytes = (bifazen_decode_bytes if bifa else bukuvik_decode_bytes if buku else vurazen_decode_bytes)(shape, B, ctx, es)
+        if vura or buku or bifa or moba:
+            phase_bytes = (mobatar_decode_bytes if moba else bifazen_decode_bytes if bifa else bukuvik_decode_bytes if buku else vurazen_decode_bytes)(shape, B, ctx, es)
             bytes_step = shape.weight_elems_per_step(B) * es + \
-                (shape.state_bytes_per_step(B, ctx, es) + phase_bytes["norm"] if bifa else phase_bytes["attention"])
+                (shape.state_bytes_per_step(B, ctx, es) + phase_bytes["norm"] if bifa or moba else phase_bytes["attention"])
             out["decode"][str(B)] = {
                 "batch": B, "context": ctx, "tok_s": B / sec, "ms_per_step": sec * 1e3, "launches": launches,
                 "bytes_per_step": bytes_step, "frac_of_hbm_peak": bytes_step / sec / 1e9 / hbm, "phase_ms": ph,
@@ -501,6 +562,8 @@ def run(args, emit):
         return run_bukuvik(args, emit, torch, sizes, steps, warm, flush, hbm, tf, src)
     if args.family == "bifazen":
         return run_bifazen(args, emit, torch, sizes, steps, warm, flush, hbm, tf, src)
+    if args.family == "mobatar":
+        return run_mobatar(args, emit, torch, sizes, steps, warm, flush, hbm, tf, src)
     line = {"family": "fobolorn", "metric": "prefill_and_decode_tokens_per_s", "n_gpus": 1, "steps": steps, "warmup": warm,
             "data": "synthetic", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": src},
             "config": {"l2": "a 256 MiB buffer is written between timed steps", "timing": "wall clock around the blocking "
@@ -595,6 +658,32 @@ def run_bifazen(args, emit, torch, sizes, steps, warm, flush, hbm, tf, src):
                   "kikunex_latent": kikunex_latent_shape(name), "bifazen_attention": bifazen_shape(name, "AAAAAA", "-attention"),
                   "fobolorn": SIZES[name]}
         entry = {"shape": dict(shapes["bifazen"].__dict__)}
+        for key, shape in shapes.items():
+            entry[key] = [bench_engine(torch, shape, dtype, prompt, ctx, [1, 8], steps, warm, flush, hbm, tf)
+                          for dtype in (BF16, F32)]
+        line["sizes"][name] = entry
+    emit(line)
+
+
+def run_mobatar(args, emit, torch, sizes, steps, warm, flush, hbm, tf, src):
+    """Mobatar (its three kinds of layer mixed, two of them run again; and each kind alone) beside its closest existing models on
+    the same engine at equal width, heads and layer runs: Bifazen's attention (normed over whole projections, a window of
+    512) and Kikunex's linear attention for the two halves of a pair, Bifazen's latent layers for the latent ones and
+    Fobolorn for the causal attention."""
+    line = {"family": "mobatar", "metric": "prefill_and_decode_tokens_per_s", "n_gpus": 1, "steps": steps, "warmup": warm,
+            "data": "synthetic", "peaks": {"hbm_gbs": hbm, "bf16_tflops": tf, "source": src},
+            "config": {"l2": "a 256 MiB buffer is written between timed steps", "timing": "wall clock around the blocking "
+                       "step call (token ids from host memory, greedy ids back to host memory); phases by CUDA events"},
+            "sizes": {}}
+    for name in sizes:
+        ctx, prompt = (256, 512) if name == "debug" else (1024, 2048)
+        shapes = {"mobatar": mobatar_shape(name, "APLP", (0, 1), ""),
+                  "mobatar_parallel": mobatar_shape(name, "PPPPPP", (), "-parallel"),
+                  "bifazen_attention": bifazen_shape(name, "AAAAAA", "-attention"), "kikunex_linear": kikunex_linear_shape(name),
+                  "mobatar_latent": mobatar_shape(name, "LLLLLL", (), "-latent"),
+                  "bifazen_latent": bifazen_shape(name, "LLLLLL", "-latent"),
+                  "mobatar_attention": mobatar_shape(name, "AAAAAA", (), "-attention"), "fobolorn": SIZES[name]}
+        entry = {"shape": dict(shapes["mobatar"].__dict__)}
         for key, shape in shapes.items():
             entry[key] = [bench_engine(torch, shape, dtype, prompt, ctx, [1, 8], steps, warm, flush, hbm, tf)
                           for dtype in (BF16, F32)]

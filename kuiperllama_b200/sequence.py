@@ -2,7 +2,7 @@
 device memory, the engine and every kernel are the product library's.  Like the rest of this package it has no
 fallback: without libkllm_seq.so (or libkllm_b200.so, which carries the same symbols) it raises.
 
-`FobolornShape` / `KikunexShape` / `VurazenShape` / `BukuvikShape` / `BifazenShape` + `SeqEngine` build a random-weight model of a family directly in device memory
+`FobolornShape` / `KikunexShape` / `VurazenShape` / `BukuvikShape` / `BifazenShape` / `MobatarShape` + `SeqEngine` build a random-weight model of a family directly in device memory
 (no model folder), for measurements at sizes that resemble a real model's layers.
 """
 from __future__ import annotations
@@ -493,8 +493,91 @@ class BifazenShape:
         return total
 
 
+@dataclass
+class MobatarShape:
+    """A Mobatar model: `pattern` lists the layers with weights of their own ("attention" | "parallel" | "latent", feed-forward
+    size or None), `again` the layers that run once more after them."""
+    name: str
+    width: int
+    vocab: int
+    pattern: tuple
+    again: tuple
+    heads: int           # causal attention
+    kv_heads: int
+    dim: int
+    vdim: int
+    c_heads: int         # chunked attention of a pair
+    c_kv_heads: int
+    c_dim: int
+    c_vdim: int
+    chunk: int
+    r_heads: int         # retention of a pair
+    r_dim: int
+    r_vdim: int
+    l_heads: int         # latent attention
+    l_dim: int
+    rot_dim: int
+    l_vdim: int
+    kv_rank: int
+    window: int
+    buckets: int = 65537
+    eps: float = 1e-5
+
+    @property
+    def layers(self):
+        return len(self.pattern)
+
+    def run_order(self):
+        return [(i, -1, 0) for i in list(range(self.layers)) + list(self.again)]
+
+    @property
+    def runs(self):
+        return len(self.run_order())
+
+    def run_kinds(self):
+        return [self.pattern[i] for i, _, _ in self.run_order()]
+
+    def attn_in(self, kind):
+        if kind == "attention":
+            return (self.heads + self.kv_heads) * self.dim + self.kv_heads * self.vdim
+        return (self.c_heads + self.c_kv_heads) * self.c_dim + self.c_kv_heads * self.c_vdim + self.c_heads
+
+    def n_in(self, kind):
+        if kind == "latent":
+            return self.l_heads * (self.l_dim + self.rot_dim) + self.kv_rank + self.rot_dim
+        return self.attn_in(kind) + (2 * self.r_heads * (self.r_dim + self.r_vdim) if kind == "parallel" else 0)
+
+    def n_out(self, kind):
+        return {"latent": self.l_heads * self.l_vdim, "attention": self.heads * self.vdim,
+                "parallel": self.c_heads * self.c_vdim + self.r_heads * self.r_vdim}[kind]
+
+    def expand_elems(self, kind):
+        return self.l_heads * (self.l_dim + self.l_vdim) * self.kv_rank if kind == "latent" else 0
+
+    def weight_elems_per_step(self, batch):
+        return self.vocab * self.width + sum((self.n_in(m) + self.n_out(m)) * self.width + self.expand_elems(m) +
+                                             3 * (f or 0) * self.width for m, f in self.run_kinds())
+
+    def flops_per_token(self):
+        return 2 * self.weight_elems_per_step(1)
+
+    def state_bytes_per_step(self, batch, ctx, es):
+        """Cache and state a decode step touches: keys and values in reach, the window's latents, the retention's state (read
+        and written)."""
+        total = 0
+        for m, _ in self.run_kinds():
+            if m == "latent":
+                total += batch * min(ctx, self.window) * (self.kv_rank + self.rot_dim) * es
+            elif m == "attention":
+                total += batch * ctx * self.kv_heads * (self.dim + self.vdim) * es
+            else:
+                total += batch * (ctx % self.chunk + 1) * self.c_kv_heads * (self.c_dim + self.c_vdim) * es
+                total += batch * 2 * self.r_heads * self.r_dim * self.r_vdim * 4
+        return total
+
+
 class SeqEngine:
-    """A random-weight model (Fobolorn, Kikunex, Vurazen, Bukuvik or Bifazen, by the shape's class) in device memory behind the engine's C-ABI."""
+    """A random-weight model (Fobolorn, Kikunex, Vurazen, Bukuvik, Bifazen or Mobatar, by the shape's class) in device memory behind the engine's C-ABI."""
 
     def __init__(self, shape, dtype=BF16, max_tokens=4096, max_seqs=16, page=0, seed=1):
         import torch
@@ -512,6 +595,9 @@ class SeqEngine:
             return
         if isinstance(shape, BifazenShape):
             self._init_bifazen(shape, dtype, max_tokens, max_seqs, page, seed)
+            return
+        if isinstance(shape, MobatarShape):
+            self._init_mobatar(shape, dtype, max_tokens, max_seqs, page, seed)
             return
         td = torch.bfloat16 if dtype == BF16 else torch.float32
         g = torch.Generator(device="cuda").manual_seed(seed)
@@ -943,6 +1029,100 @@ class SeqEngine:
         d.embed = rnd(shape.vocab, W, std=1.0).data_ptr()
         d.final_norm = norm()
         d.head = d.embed  # the classifier is the embedding table
+        d.max_tokens, d.max_seqs, d.page_tokens = max_tokens, max_seqs, page
+        self._desc = (d, layers, run_layer, run_add, run_embed)
+        self.handle = c_void_p()
+        torch.cuda.synchronize()
+        _check(self.lib, self.lib.kllm_seq_create(ctypes.byref(d), None, ctypes.byref(self.handle)), "kllm_seq_create")
+
+    def _init_mobatar(self, shape, dtype, max_tokens, max_seqs, page, seed):
+        torch = self.torch
+        td = torch.bfloat16 if dtype == BF16 else torch.float32
+        g = torch.Generator(device="cuda").manual_seed(seed)
+        keep = self._keep = []
+        W = shape.width
+
+        def rnd(*dims, std, t=td, mean=0.0):
+            x = (torch.randn(*dims, device="cuda", generator=g) * std + mean).to(t).contiguous()
+            keep.append(x)
+            return x
+
+        def f32(*dims, std, mean=0.0):
+            return rnd(*dims, std=std, t=torch.float32, mean=mean)
+
+        def host(values):
+            x = torch.tensor(values, dtype=torch.float32, device="cuda")
+            keep.append(x)
+            return x.data_ptr()
+
+        def freq(dims, base):
+            return host([base ** (-2.0 * i / dims) for i in range(dims // 2)])
+
+        def norm():
+            return Norm(f32(W, std=0.1, mean=1.0).data_ptr(), None, 1)
+
+        def attention(a, kind, heads, kv_heads, dim, vdim, w_in):
+            a.heads, a.kv_heads, a.dim, a.vdim, a.scale = heads, kv_heads, dim, vdim, dim ** -0.5
+            a.rope_dims, a.rope_base, a.rope_freq = dim, 5e5, freq(dim, 5e5)
+            a.w_in = w_in
+            a.w_out = rnd(W, heads * vdim, std=(heads * vdim) ** -0.5).data_ptr()
+
+        layers = (Layer * shape.layers)()
+        for L, (mix, ff) in zip(layers, shape.pattern):
+            L.pre_mixer, L.pre_ff = Norm(None, None, 2), Norm(None, None, 2)
+            L.post_mixer = norm()
+            w_in = rnd(shape.n_in(mix), W, std=W ** -0.5)
+            if mix == "attention":
+                L.mixer_kind = 1
+                attention(L.attn, mix, shape.heads, shape.kv_heads, shape.dim, shape.vdim, w_in.data_ptr())
+                L.attn.qk_norm, L.attn.sink = 2, host([0.0] * shape.heads)
+            elif mix == "parallel":
+                L.mixer_kind, L.mixer2_kind, L.mixer_scale, L.mixer2_scale = 1, 3, 0.75, 1.25
+                a, r = L.attn, L.linear
+                attention(a, mix, shape.c_heads, shape.c_kv_heads, shape.c_dim, shape.c_vdim, w_in.data_ptr())
+                a.qk_norm, a.gate, a.chunk = 3, 1, shape.chunk
+                a.q_norm_w = f32(shape.c_heads * shape.c_dim, std=0.1, mean=1.0).data_ptr()
+                a.k_norm_w = f32(shape.c_kv_heads * shape.c_dim, std=0.1, mean=1.0).data_ptr()
+                r.heads, r.dim, r.vdim = shape.r_heads, shape.r_dim, shape.r_vdim
+                r.decay = host([1.0 - 2.0 ** (-5 - i % 8) for i in range(shape.r_heads)])
+                r.w_in = w_in.data_ptr() + shape.attn_in(mix) * W * w_in.element_size()
+                r.w_out = rnd(W, shape.r_heads * shape.r_vdim, std=(shape.r_heads * shape.r_vdim) ** -0.5).data_ptr()
+                r.qkv_act, r.rope_dims, r.rope_base, r.rope_freq = 1, shape.r_dim, 1e4, freq(shape.r_dim, 1e4)
+                r.k_scale, r.out_norm, r.gate_act = shape.r_dim ** -0.5, 1, 1
+            else:
+                L.mixer_kind = 2
+                a = L.latent
+                a.heads, a.dim, a.rot_dim, a.vdim = shape.l_heads, shape.l_dim, shape.rot_dim, shape.l_vdim
+                a.q_rank, a.kv_rank, a.window, a.gate = 0, shape.kv_rank, shape.window, 0
+                a.scale, a.rope_dims, a.rope_base, a.rope_pairing = (shape.l_dim + shape.rot_dim) ** -0.5, shape.rot_dim, 1e5, 1
+                a.rope_freq = freq(shape.rot_dim, 1e5)
+                a.w_in = w_in.data_ptr()
+                a.kv_norm_w = f32(shape.kv_rank, std=0.05, mean=1.0).data_ptr()
+                ukv = rnd(shape.l_heads * (shape.l_dim + shape.l_vdim), shape.kv_rank, std=shape.kv_rank ** -0.5)
+                a.w_uk = ukv.data_ptr()
+                a.w_uv = ukv.data_ptr() + shape.l_heads * shape.l_dim * shape.kv_rank * ukv.element_size()
+                a.w_out = rnd(W, shape.l_heads * shape.l_vdim, std=(shape.l_heads * shape.l_vdim) ** -0.5).data_ptr()
+            L.ff_kind = 2 if ff else 0
+            if ff:
+                L.post_ff = norm()
+                d = L.dense
+                d.ff, d.act, d.act_a, d.act_b = ff, 4, 4.0, 1.702
+                d.up = rnd(2 * ff, W, std=W ** -0.5).data_ptr()
+                d.down = rnd(W, ff, std=ff ** -0.5).data_ptr()
+                d.up_bias, d.down_bias = f32(2 * ff, std=0.1).data_ptr(), f32(W, std=0.1).data_ptr()
+        order = shape.run_order()
+        run_layer = (c_int32 * len(order))(*[i for i, _, _ in order])
+        run_add = (c_int32 * len(order))(*[p for _, p, _ in order])
+        run_embed = (c_int32 * len(order))(*[x for _, _, x in order])
+        d = Desc()
+        d.dtype, d.width, d.vocab, d.norm_eps = dtype, W, shape.vocab, shape.eps
+        d.n_layers, d.layers = shape.layers, layers
+        d.n_runs, d.run_layer, d.run_add, d.run_embed = len(order), run_layer, run_add, run_embed
+        d.embed = rnd(shape.vocab, W, std=1.0).data_ptr()
+        d.bigram = rnd(shape.buckets + 1, W, std=1.0).data_ptr()
+        d.bigram_buckets, d.bigram_mul_prev, d.bigram_mul_cur = shape.buckets, 31337, 7919
+        d.final_norm = norm()
+        d.head = rnd(shape.vocab, W, std=W ** -0.5).data_ptr()
         d.max_tokens, d.max_seqs, d.page_tokens = max_tokens, max_seqs, page
         self._desc = (d, layers, run_layer, run_add, run_embed)
         self.handle = c_void_p()

@@ -202,3 +202,108 @@ def greedy(config, weights, prompt, n_new):
     for _ in range(n_new):
         seq.append(int(np.argmax(forward(config, weights, seq)[0][-1])))
     return seq[len(prompt):]
+
+
+# ---- small configurations and random weights for the tests ---------------------------------------------------------------
+def rotation(dims, base=1000.0, scaling=None):
+    r = {"dims": dims, "base": base}
+    if scaling:
+        r["scaling"] = dict(scaling)
+    return r
+
+
+BANDS = {"factor": 5.0, "low": 1.0, "high": 3.0, "original": 60}
+
+
+def sink_mixer(heads=4, kv_heads=2, dim=12, vdim=10, rot_dims=8, base=1000.0, scaling=BANDS, scale=0.35):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale,
+            "rot": rotation(rot_dims, base, scaling)}
+
+
+def chunk_mixer(heads=4, kv_heads=2, dim=10, vdim=6, chunk=13, rot_dims=6, base=300.0, factor=3.0, scale=None):
+    return {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "mask": {"size": chunk},
+            "scale": dim ** -0.5 if scale is None else scale, "rot": rotation(rot_dims, base, {"factor": factor})}
+
+
+def retention_mixer(heads=3, dim=8, vdim=7, rot_dims=6, base=500.0, decay=None):
+    if decay is None:
+        decay = [(0.9, 0.99, 0.75, 0.998, 1.0)[i % 5] for i in range(heads)]
+    return {"heads": heads, "dim": dim, "vdim": vdim, "decay": list(decay), "rot": rotation(rot_dims, base)}
+
+
+def parallel_mixer(left=None, right=None, left_scale=0.75, right_scale=1.5):
+    return {"left": left or chunk_mixer(), "right": right or retention_mixer(), "left_scale": left_scale,
+            "right_scale": right_scale}
+
+
+def latent_mixer(heads=3, dim=10, rot_dim=6, vdim=7, kv_rank=20, window=14, base=1000.0, scale=None):
+    return {"heads": heads, "dim": dim, "rot_dim": rot_dim, "vdim": vdim, "kv_rank": kv_rank, "mask": {"size": window},
+            "rot": rotation(rot_dim, base), "scale": (dim + rot_dim) ** -0.5 if scale is None else scale}
+
+
+def make_config(width=48, vocab=61, layers=(), eps=3e-6, buckets=37, mul_prev=11, mul_cur=5):
+    """layers: (mixer, (ff size, limit) or None), the mixer's kind read off its keys; or the number of an earlier layer whose
+    weights run again."""
+    out = []
+    for spec in layers:
+        if isinstance(spec, int):
+            out.append(dict(out[spec], weights_of=spec))
+            continue
+        mixer, ff = spec
+        kind = "latent_attention" if "kv_rank" in mixer else "parallel" if "left" in mixer else "attention"
+        out.append({"type": kind, "mixer": mixer, "mlp": {"kind": "dense", "ff": ff[0], "limit": ff[1]} if ff else None})
+    return {"architecture": "Mobatar", "vocab": vocab, "width": width, "norm": {"eps": eps}, "layers": out,
+            "embedding": {"bigram": {"buckets": buckets, "mul_prev": mul_prev, "mul_cur": mul_cur}}}
+
+
+def make_weights(cfg, seed=0, sharp=1.0):
+    """Random bf16-representable weights.  `sharp` multiplies the query weights of the softmax attentions that do not
+    unit-norm their queries (the norm weights of those that norm them): > 1 makes the softmax peaky, so that single keys
+    (those at an edge too) carry the output."""
+    from seq_util import bf16_round
+    rng = np.random.default_rng(seed)
+    W, V = cfg["width"], cfg["vocab"]
+
+    def rnd(*shape, std=1.0, mean=0.0):
+        return bf16_round(mean + std * rng.standard_normal(shape))
+
+    def fan(rows, cols, gain=1.0):
+        return rnd(rows, cols, std=gain * cols ** -0.5)
+
+    w = {"embed": rnd(V, W, std=0.7), "bigram": rnd(cfg["embedding"]["bigram"]["buckets"] + 1, W, std=0.7),
+         "final.norm": rnd(W, std=0.2), "head": fan(V, W)}
+    for i, L in enumerate(cfg["layers"]):
+        if L.get("weights_of") is not None:
+            continue
+        p, m = f"l{i}.", L["mixer"]
+        q = p + "mix."
+        w[p + "norm1"] = rnd(W, std=0.2)
+        if L["type"] == "latent_attention":
+            H = m["heads"]
+            w[q + "q"] = fan(H * (m["dim"] + m["rot_dim"]), W, sharp)
+            w[q + "dkv"] = fan(m["kv_rank"] + m["rot_dim"], W, 1.5)
+            w[q + "dkv.norm"] = rnd(m["kv_rank"], mean=1.0, std=0.2)
+            w[q + "uk"] = fan(H * m["dim"], m["kv_rank"], 1.5)
+            w[q + "uv"] = fan(H * m["vdim"], m["kv_rank"])
+            w[q + "o"] = fan(W, H * m["vdim"])
+        else:
+            a, r = (m["left"], m["right"]) if L["type"] == "parallel" else (m, None)
+            lp = q + "left." if r else q
+            H, G = a["heads"], a["kv_heads"]
+            w[lp + "q"], w[lp + "k"] = fan(H * a["dim"], W), fan(G * a["dim"], W)
+            w[lp + "v"], w[lp + "o"] = fan(G * a["vdim"], W), fan(W, H * a["vdim"])
+            if r:
+                w[lp + "q.norm"] = rnd(H * a["dim"], mean=sharp, std=0.2 * sharp)
+                w[lp + "k.norm"] = rnd(G * a["dim"], mean=1.5, std=0.3)
+                w[lp + "g"] = fan(H, W, 2.0)
+                rp, R = q + "right.", r["heads"]
+                w[rp + "q"], w[rp + "k"] = fan(R * r["dim"], W), fan(R * r["dim"], W)
+                w[rp + "v"], w[rp + "g"] = fan(R * r["vdim"], W), fan(R * r["vdim"], W)
+                w[rp + "o"] = fan(W, R * r["vdim"])
+        if L.get("mlp"):
+            ff = L["mlp"]["ff"]
+            w[p + "norm2"] = rnd(W, std=0.2)
+            for n, rows, cols in (("gate", ff, W), ("up", ff, W), ("down", W, ff)):
+                w[p + "mlp." + n] = fan(rows, cols)
+                w[p + "mlp." + n + ".b"] = rnd(rows, std=0.3)
+    return w

@@ -1,7 +1,9 @@
-"""Drive bin/trace_run (the product's own entry: registry -> scheduler -> sequence-batch engine) from the tests."""
+"""Drive bin/trace_run (the product's own entry: registry -> scheduler -> sequence-batch engine) from the tests: model
+folders, traces of steps, comparisons of rows of logits."""
 from __future__ import annotations
 
 import json
+import struct
 import subprocess
 import tempfile
 from pathlib import Path
@@ -55,3 +57,53 @@ def rel_err(got, ref):
     d = d - d.mean(-1, keepdims=True)
     spread = (ref - ref.mean(-1, keepdims=True)).std()
     return float(np.sqrt((d ** 2).mean(-1)).max() / spread)
+
+
+def row_errors(got, ref):
+    """rel_err of every row on its own."""
+    return np.array([rel_err(got[i:i + 1], ref[i:i + 1]) for i in range(len(ref))])
+
+
+def assert_rows(got, ref, tol):
+    assert len(got) == len(ref)
+    err = row_errors(got, ref)
+    assert err.max() < tol, f"first bad position {int(np.argmax(err >= tol))} of {len(ref)}, worst {err.max():.3g}"
+
+
+def single(rid, tokens, end=False):
+    """One step per token."""
+    steps = [{"entries": [{"id": rid, "tokens": [x], "want": [0]}]} for x in tokens]
+    if end and steps:
+        steps[-1]["end"] = [rid]
+    return steps
+
+
+def random_tokens(n, vocab, seed):
+    return [int(t) for t in np.random.default_rng(seed).integers(0, vocab, n)]
+
+
+def bf16_round(a):
+    """Round float64 values to the nearest bfloat16 (ties to even); the result is exactly representable."""
+    u = np.asarray(a, dtype=np.float32).view(np.uint32).astype(np.uint64)
+    u = (u + 0x7fff + ((u >> 16) & 1)) & 0xffff0000
+    return u.astype(np.uint32).view(np.float32).astype(np.float64)
+
+
+def write_model(folder, cfg, weights):
+    """config.json and model.safetensors (bfloat16) in `folder`."""
+    folder = Path(folder)
+    folder.mkdir(parents=True, exist_ok=True)
+    (folder / "config.json").write_text(json.dumps(cfg))
+    header, blobs, at = {}, [], 0
+    for name, a in weights.items():
+        u = np.ascontiguousarray(a, dtype=np.float32).view(np.uint32)
+        assert not (u & 0xffff).any(), f"{name} is not bf16-representable"
+        raw = (u >> 16).astype("<u2").tobytes()
+        header[name] = {"dtype": "BF16", "shape": list(np.shape(a)), "data_offsets": [at, at + len(raw)]}
+        blobs.append(raw)
+        at += len(raw)
+    head = json.dumps(header).encode()
+    head += b" " * (-len(head) % 8)
+    with open(folder / "model.safetensors", "wb") as f:
+        f.write(struct.pack("<Q", len(head)) + head + b"".join(blobs))
+    return folder
