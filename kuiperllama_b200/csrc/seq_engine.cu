@@ -145,6 +145,7 @@ struct kllm_seq_engine {
   DevBuf idx, x, h, proj, q, gates, att, y, y2, ws, top_idx, top_w, sgate, inter, pairs_out, sort, sorted_a, sorted_inter, hw, logits, amax;
   DevBuf lat_c, lat_kr, lat_kp, lat_vp, lat_q, lat_k, lat_v;  // a prompt step's latents expanded into per-head keys / values
   DevBuf x0, hn, qf, qa, ol;  // embedding output; fp32 normed rows ahead of a token shift; latent / linear attention scratch
+  DevBuf proj2, q2, att2, ws2;  // what a second mixer works in beside the first
   DevBuf y3, y4;              // outputs of a second mixer and of a feed-forward that runs beside the mixer
   DevBuf xs, vfirst;          // residual streams [T][streams][width]; the values of the step that later layers blend with
   DevBuf rec_a, rec_b, rec_c; // fp32 scratch of the selective scan (filtered rows, low-rank rows) and the delta rule (prepared rows)
@@ -161,6 +162,8 @@ struct kllm_seq_engine {
   };
   std::map<std::tuple<int, int, int, int>, Graph> graphs;
   bool own_stream = false;
+  cudaStream_t side = nullptr;  // a pair's second mixer runs here, between `fork` and `join`
+  cudaEvent_t fork = nullptr, join = nullptr;
   bool use_graphs = true;
   // per-phase device times of one step (kllm_seq_profile): an event after every phase, read after the step's sync
   float* prof_out = nullptr;
@@ -196,6 +199,9 @@ struct kllm_seq_engine {
     if (logits_pinned) cudaFreeHost(logits_pinned);
     for (cudaEvent_t ev : prof_events) cudaEventDestroy(ev);
     for (auto& g : graphs) if (g.second.exec) cudaGraphExecDestroy(g.second.exec);
+    if (fork) cudaEventDestroy(fork);
+    if (join) cudaEventDestroy(join);
+    if (side) cudaStreamDestroy(side);
     if (own_stream && stream) cudaStreamDestroy(stream);
   }
 };
@@ -214,6 +220,17 @@ static AttnShape attn_shape(const kllm_seq_attention& A) {
 static int attn_proj_rows(const kllm_seq_attention& A) {
   const AttnShape s = attn_shape(A);
   return s.heads * A.dim + s.kv_heads * A.dim + (A.values_are_keys ? 0 : A.kv_heads * A.vdim) + gate_floats(s);
+}
+
+static int linear_proj_rows(const kllm_seq_linear& A) { return 2 * A.heads * (A.dim + A.vdim); }
+
+// A pair whose linear attention's input rows follow the attention's in memory: how many rows those are (0: not stacked)
+static int stacked_rows(const kllm_seq_desc& d, const kllm_seq_layer& L) {
+  if (L.mixer_kind != KLLM_SEQ_MIXER_ATTENTION || L.mixer2_kind != KLLM_SEQ_MIXER_LINEAR || L.attn.values_are_keys || L.attn.in_bias)
+    return 0;
+  const int rows = attn_proj_rows(L.attn);
+  const char* end = static_cast<const char*>(L.attn.w_in) + static_cast<size_t>(rows) * d.width * elt(d.dtype);
+  return end == static_cast<const char*>(L.linear.w_in) ? rows : 0;
 }
 
 static LatentShape latent_shape(const kllm_seq_latent& A) {
@@ -471,7 +488,7 @@ extern "C" int kllm_seq_create(const kllm_seq_desc* desc, void* stream, kllm_seq
         e->max_gates = std::max(e->max_gates, a.heads);
       } else if (kind == KLLM_SEQ_MIXER_LINEAR) {
         const kllm_seq_linear& a = L.linear;
-        e->max_proj = std::max(e->max_proj, 2 * a.heads * (a.dim + a.vdim));
+        e->max_proj = std::max(e->max_proj, linear_proj_rows(a));
         e->max_ol = std::max(e->max_ol, a.heads * a.vdim);
         e->max_att = std::max(e->max_att, a.heads * a.vdim);
       } else if (kind == KLLM_SEQ_MIXER_SSM) {
@@ -505,6 +522,14 @@ extern "C" int kllm_seq_create(const kllm_seq_desc* desc, void* stream, kllm_seq
       e->max_ff = std::max(e->max_ff, L.moe.top * L.moe.ff);
       e->max_sff = std::max(e->max_sff, L.moe.shared_ff);
     }
+  }
+  for (const kllm_seq_layer& L : e->layers)
+    if (const int n1 = stacked_rows(e->d, L)) e->max_proj = std::max(e->max_proj, n1 + linear_proj_rows(L.linear));
+  if (e->any_mixer2 && (cudaStreamCreateWithFlags(&e->side, cudaStreamNonBlocking) != cudaSuccess ||
+                        cudaEventCreateWithFlags(&e->fork, cudaEventDisableTiming) != cudaSuccess ||
+                        cudaEventCreateWithFlags(&e->join, cudaEventDisableTiming) != cudaSuccess)) {
+    delete e;
+    return KLLM_E_NODEVICE;
   }
   *out = e;
   return 0;
@@ -685,7 +710,12 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
   if (e->max_qf > 0) RC(e->qf.reserve(Ts * e->max_qf * 4));
   if (e->max_qa > 0) RC(e->qa.reserve(Ts * e->max_qa * 4));
   if (e->max_ol > 0) RC(e->ol.reserve(Ts * e->max_ol * 4));
-  if (e->any_mixer2) RC(e->y3.reserve(Ts * W * 4));
+  if (e->any_mixer2) {
+    RC(e->y3.reserve(Ts * W * 4));
+    RC(e->proj2.reserve(Ts * e->max_proj * 4));
+    RC(e->q2.reserve(Ts * std::max(1, e->max_q) * es));
+    RC(e->att2.reserve(Ts * e->max_att * es));
+  }
   if (e->any_parallel_ff) RC(e->y4.reserve(Ts * W * 4));
   if (e->max_rec_a > 0) RC(e->rec_a.reserve(Ts * e->max_rec_a * 4));
   if (e->max_rec_b > 0) RC(e->rec_b.reserve(Ts * e->max_rec_b * 4));
@@ -712,6 +742,7 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
     if (L.mixer_kind == KLLM_SEQ_MIXER_SSD || L.mixer2_kind == KLLM_SEQ_MIXER_SSD)
       ws_bytes = std::max(ws_bytes, ssd_scan_scratch_bytes(L.ssd, T, n_entries, max_count));
   RC(e->ws.reserve(ws_bytes));
+  if (e->any_mixer2) RC(e->ws2.reserve(ws_bytes));
   const bool grouped = T >= kGroupedMinTokens;
   if (e->max_top > 0) {
     RC(e->top_idx.reserve(Ts * e->max_top * 4));
@@ -775,38 +806,53 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
     e->mark(phase);
     return 0;
   };
+  // What a mixer works in.  The two mixers of a pair have buffers of their own, so that they can run side by side; `row` != 0
+  // says that the input projection is already in `proj`, its rows `row` floats apart.
+  struct MixerRoom {
+    float* proj;
+    int row;
+    void *q, *att;
+    float* ws;
+    cudaStream_t st;
+  };
   // one mixer of layer L (run r): reads the normed rows in e->h, writes its output rows to `yout`
-  auto run_mixer = [&](const kllm_seq_layer& L, int kind, int r, float* yout) -> int {
+  auto run_mixer = [&](const kllm_seq_layer& L, int kind, int r, const MixerRoom& room, float* yout) -> int {
+    float* const proj = room.proj;
+    const cudaStream_t st = room.st;
+    const bool main = st == e->stream;  // phases are marked on the engine's stream only
+    auto mark = [&](int phase) {
+      if (main) e->mark(phase);
+    };
     if (kind == KLLM_SEQ_MIXER_ATTENTION) {
       const kllm_seq_attention& A = L.attn;
       const AttnShape shape = attn_shape(A);
       const PagedKV kv{e->k_pool[r], e->v_pool[r], e->table_dev, e->table_stride, e->page, shape.kv_heads * A.dim,
                        A.kv_heads * A.vdim};
-      const int n_proj = attn_proj_rows(A);
+      const int n_proj = attn_proj_rows(A), row = room.row > 0 ? room.row : n_proj;
       // the filtered form adds its bias in its own preparation
-      RC(gemm(dtype, e->h.p, A.w_in, proj, T, W, n_proj, st, A.values_are_keys ? nullptr : A.in_bias));
-      e->mark(KLLM_SEQ_PHASE_IN_PROJ);
+      if (room.row == 0) RC(gemm(dtype, e->h.p, A.w_in, proj, T, W, n_proj, st, A.values_are_keys ? nullptr : A.in_bias));
+      mark(KLLM_SEQ_PHASE_IN_PROJ);
       if (A.values_are_keys) {
         const AttnPrep prep{std::max(1, A.conv_taps), A.conv_w, e->attn_conv[r], A.in_bias, A.rope_dims, A.rope_pairing,
                             A.rope_base};
-        RC(launch_qk_conv_prepare(dtype, shape, prep, proj, step_rows, e->q.p, kv, T, st));
+        RC(launch_qk_conv_prepare(dtype, shape, prep, proj, step_rows, room.q, kv, T, st));
       } else {
         const RopeArgs rope{A.rope_dims, A.rope_base, A.rope_freq, A.rope_mag, A.rope_pairing};
-        RC(launch_qk_prepare(dtype, shape, rope, proj, A.q_norm_w, A.k_norm_w, d.norm_eps, d_seq, d_pos, e->q.p,
+        RC(launch_qk_prepare(dtype, shape, rope, proj, row, A.q_norm_w, A.k_norm_w, d.norm_eps, d_seq, d_pos, room.q,
                              static_cast<float*>(e->gates.p), kv,
                              ValueBlend{A.v_blend, A.v_lambda, static_cast<float*>(e->vfirst.p)}, T, st));
       }
-      e->mark(KLLM_SEQ_PHASE_QK_PREPARE);
-      RC(launch_attention(dtype, shape, e->q.p, static_cast<const float*>(e->gates.p), kv, n_entries, d_first, d_count,
+      mark(KLLM_SEQ_PHASE_QK_PREPARE);
+      RC(launch_attention(dtype, shape, room.q, static_cast<const float*>(e->gates.p), kv, n_entries, d_first, d_count,
                           d_eseq, d_pos0, max_count, max_ctx, attn_splits(A),
-                          static_cast<float*>(e->ws.p), e->att.p, T, d_seq, d_pos, st));
+                          room.ws, room.att, T, d_seq, d_pos, st));
       if (A.differential)
-        RC(launch_diff_merge(dtype, shape, attn_splits(A), static_cast<const float*>(e->ws.p),
-                             static_cast<const float*>(e->gates.p), A.diff_lambda, A.diff_out_scale, d.norm_eps, e->att.p, T,
+        RC(launch_diff_merge(dtype, shape, attn_splits(A), room.ws,
+                             static_cast<const float*>(e->gates.p), A.diff_lambda, A.diff_out_scale, d.norm_eps, room.att, T,
                              st));
-      e->mark(KLLM_SEQ_PHASE_ATTENTION);
-      RC(gemm(dtype, e->att.p, A.w_out, yout, T, A.heads * A.vdim, W, st, A.out_bias));
-      e->mark(KLLM_SEQ_PHASE_OUT_PROJ);
+      mark(KLLM_SEQ_PHASE_ATTENTION);
+      RC(gemm(dtype, room.att, A.w_out, yout, T, A.heads * A.vdim, W, st, A.out_bias));
+      mark(KLLM_SEQ_PHASE_OUT_PROJ);
     } else if (kind == KLLM_SEQ_MIXER_LATENT) {
       const kllm_seq_latent& A = L.latent;
       const LatentShape ls = latent_shape(A);
@@ -815,12 +861,12 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
       float* gates = A.gate ? static_cast<float*>(e->gates.p) : nullptr;
       const int n_proj = latent_proj_rows(ls);
       RC(gemm(dtype, e->h.p, A.w_in, proj, T, W, n_proj, st));
-      e->mark(KLLM_SEQ_PHASE_IN_PROJ);
+      mark(KLLM_SEQ_PHASE_IN_PROJ);
       // the queries: expanded from their own latent, or rows of the input projection
       const float* queries = A.q_rank > 0 ? static_cast<const float*>(e->qf.p) : proj;
       const int q_row = A.q_rank > 0 ? A.heads * (A.dim + A.rot_dim) : n_proj;
       auto expand_queries = [&]() -> int {
-        return A.q_rank > 0 ? gemm(dtype, e->q.p, A.w_uq, static_cast<float*>(e->qf.p), T, A.q_rank, q_row, st) : 0;
+        return A.q_rank > 0 ? gemm(dtype, room.q, A.w_uq, static_cast<float*>(e->qf.p), T, A.q_rank, q_row, st) : 0;
       };
       // Prompt steps whose sequences all start here: the step's own latents are all the keys there are, so they are
       // expanded into per-head keys and values (two products) and the tensor-core attention runs on those rows.  Every
@@ -838,7 +884,7 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
         RC(e->lat_q.reserve(Ts * A.heads * dqk * es));
         RC(e->lat_k.reserve(Ts * A.heads * dqk * es));
         RC(e->lat_v.reserve(Ts * A.heads * A.vdim * es));
-        RC(launch_latent_prepare(dtype, ls, proj, A.q_norm_w, A.kv_norm_w, d.norm_eps, d_seq, d_pos, e->q.p, gates, kv,
+        RC(launch_latent_prepare(dtype, ls, proj, A.q_norm_w, A.kv_norm_w, d.norm_eps, d_seq, d_pos, room.q, gates, kv,
                                  e->lat_c.p, static_cast<float*>(e->lat_kr.p), T, st));
         RC(expand_queries());
         float* kp = static_cast<float*>(e->lat_kp.p);
@@ -847,98 +893,104 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
         RC(launch_latent_pack(dtype, ls, queries, q_row, kp, stacked ? kn + vn : kn, static_cast<const float*>(e->lat_kr.p),
                               stacked ? kp + kn : static_cast<const float*>(e->lat_vp.p), stacked ? kn + vn : vn, d_pos,
                               e->lat_q.p, e->lat_k.p, e->lat_v.p, T, st));
-        e->mark(KLLM_SEQ_PHASE_QK_PREPARE);
+        mark(KLLM_SEQ_PHASE_QK_PREPARE);
         const PagedKV rows{e->lat_k.p, e->lat_v.p, nullptr, 0, 1, A.heads * dqk, A.heads * A.vdim};
         RC(launch_attention(dtype, eshape, e->lat_q.p, gates, rows, n_entries, d_first, d_count, d_eseq, d_pos0, max_count,
-                            max_ctx, 1, static_cast<float*>(e->ws.p), e->att.p, T, d_seq, d_pos, st));
-        e->mark(KLLM_SEQ_PHASE_ATTENTION);
-        RC(gemm(dtype, e->att.p, A.w_out, yout, T, A.heads * A.vdim, W, st));
-        e->mark(KLLM_SEQ_PHASE_OUT_PROJ);
+                            max_ctx, 1, room.ws, room.att, T, d_seq, d_pos, st));
+        mark(KLLM_SEQ_PHASE_ATTENTION);
+        RC(gemm(dtype, room.att, A.w_out, yout, T, A.heads * A.vdim, W, st));
+        mark(KLLM_SEQ_PHASE_OUT_PROJ);
       } else {
-      RC(launch_latent_prepare(dtype, ls, proj, A.q_norm_w, A.kv_norm_w, d.norm_eps, d_seq, d_pos, e->q.p, gates, kv, nullptr,
+      RC(launch_latent_prepare(dtype, ls, proj, A.q_norm_w, A.kv_norm_w, d.norm_eps, d_seq, d_pos, room.q, gates, kv, nullptr,
                                nullptr, T, st));
       RC(expand_queries());
       RC(launch_latent_absorb(dtype, ls, queries, q_row, A.w_uk, d_pos, static_cast<float*>(e->qa.p), T, st));
-      e->mark(KLLM_SEQ_PHASE_QK_PREPARE);
+      mark(KLLM_SEQ_PHASE_QK_PREPARE);
       // one shared key/value "head": keys [latent | rotated part], values the latent itself
       // steps of single tokens merge the key splits and apply W_uv in one kernel
       const bool fused_merge = single && T <= 32;
       const AttnShape shape{A.heads, 1, krow, A.kv_rank, A.scale, 0.f, 0, 0, A.gate, A.window, A.sink, 1, 1, fused_merge ? 1 : 0};
       const int lsplits = reach_splits(A.window);
       RC(launch_attention(dtype, shape, e->qa.p, gates, kv, n_entries, d_first, d_count, d_eseq, d_pos0, max_count, max_ctx,
-                          lsplits, static_cast<float*>(e->ws.p), e->ol.p, T, d_seq, d_pos, st));
+                          lsplits, room.ws, e->ol.p, T, d_seq, d_pos, st));
       if (fused_merge)
-        RC(launch_latent_merge_expand(dtype, ls, lsplits, static_cast<const float*>(e->ws.p), gates, A.sink, A.w_uv,
-                                      e->att.p, T, st));
+        RC(launch_latent_merge_expand(dtype, ls, lsplits, room.ws, gates, A.sink, A.w_uv,
+                                      room.att, T, st));
       else
-        RC(launch_latent_expand(dtype, ls, static_cast<const float*>(e->ol.p), A.w_uv, e->att.p, T, st));
-      e->mark(KLLM_SEQ_PHASE_ATTENTION);
-      RC(gemm(dtype, e->att.p, A.w_out, yout, T, A.heads * A.vdim, W, st));
-      e->mark(KLLM_SEQ_PHASE_OUT_PROJ);
+        RC(launch_latent_expand(dtype, ls, static_cast<const float*>(e->ol.p), A.w_uv, room.att, T, st));
+      mark(KLLM_SEQ_PHASE_ATTENTION);
+      RC(gemm(dtype, room.att, A.w_out, yout, T, A.heads * A.vdim, W, st));
+      mark(KLLM_SEQ_PHASE_OUT_PROJ);
       }
     } else if (kind == KLLM_SEQ_MIXER_LINEAR) {
       const kllm_seq_linear& A = L.linear;
-      const int row = 2 * A.heads * (A.dim + A.vdim);
-      RC(gemm(dtype, e->h.p, A.w_in, proj, T, W, row, st));
-      e->mark(KLLM_SEQ_PHASE_IN_PROJ);
+      const int n_proj = linear_proj_rows(A), row = room.row > 0 ? room.row : n_proj;
+      if (room.row == 0) RC(gemm(dtype, e->h.p, A.w_in, proj, T, W, n_proj, st));
+      mark(KLLM_SEQ_PHASE_IN_PROJ);
+      if (single && linear_token_usable(A)) {
+        RC(launch_linear_token(dtype, A, proj, row, e->linear_state[r], d_seq, d_pos, d.norm_eps, room.att, T, st));
+      } else {
       if (linear_attention_rotates(A, max_count)) {
         RC(launch_linear_rotate(A, proj, row, d_pos, T, st));
-        e->mark(KLLM_SEQ_PHASE_QK_PREPARE);
+        mark(KLLM_SEQ_PHASE_QK_PREPARE);
       }
       RC(launch_linear_attention(A, proj, row, e->linear_state[r], n_entries, d_first, d_count, d_eseq, d_pos0, max_count,
-                                 static_cast<float*>(e->ws.p), static_cast<float*>(e->ol.p), st));
-      RC(launch_linear_out(dtype, A, static_cast<const float*>(e->ol.p), proj, row, d.norm_eps, e->att.p, T, st));
-      e->mark(KLLM_SEQ_PHASE_ATTENTION);
-      RC(gemm(dtype, e->att.p, A.w_out, yout, T, A.heads * A.vdim, W, st));
-      e->mark(KLLM_SEQ_PHASE_OUT_PROJ);
+                                 room.ws, static_cast<float*>(e->ol.p), st));
+      RC(launch_linear_out(dtype, A, static_cast<const float*>(e->ol.p), proj, row, d.norm_eps, room.att, T, st));
+      }
+      mark(KLLM_SEQ_PHASE_ATTENTION);
+      RC(gemm(dtype, room.att, A.w_out, yout, T, A.heads * A.vdim, W, st));
+      mark(KLLM_SEQ_PHASE_OUT_PROJ);
     } else if (kind == KLLM_SEQ_MIXER_SSM) {
       const kllm_seq_ssm& A = L.ssm;
       float* uc = static_cast<float*>(e->rec_a.p);
       float* low = static_cast<float*>(e->rec_b.p);
       RC(gemm(dtype, e->h.p, A.w_in, proj, T, W, 2 * A.inner, st));
-      e->mark(KLLM_SEQ_PHASE_IN_PROJ);
-      RC(launch_ssm_conv(dtype, A, proj, e->ssm_conv[r], step_rows, uc, e->att.p, T, st));
-      RC(gemm(dtype, e->att.p, A.w_x, low, T, A.inner, A.dt_rank + 2 * A.state, st));
-      e->mark(KLLM_SEQ_PHASE_QK_PREPARE);
+      mark(KLLM_SEQ_PHASE_IN_PROJ);
+      RC(launch_ssm_conv(dtype, A, proj, e->ssm_conv[r], step_rows, uc, room.att, T, st));
+      RC(gemm(dtype, room.att, A.w_x, low, T, A.inner, A.dt_rank + 2 * A.state, st));
+      mark(KLLM_SEQ_PHASE_QK_PREPARE);
       RC(launch_ssm_scan(dtype, A, proj, uc, low, e->ssm_state[r], step_rows, d_eseq, max_count, T,
-                         static_cast<float*>(e->ws.p), e->att.p, st));
-      e->mark(KLLM_SEQ_PHASE_ATTENTION);
-      RC(gemm(dtype, e->att.p, A.w_out, yout, T, A.inner, W, st));
-      e->mark(KLLM_SEQ_PHASE_OUT_PROJ);
+                         room.ws, room.att, st));
+      mark(KLLM_SEQ_PHASE_ATTENTION);
+      RC(gemm(dtype, room.att, A.w_out, yout, T, A.inner, W, st));
+      mark(KLLM_SEQ_PHASE_OUT_PROJ);
     } else if (kind == KLLM_SEQ_MIXER_SSD) {
       const kllm_seq_ssd& A = L.ssd;
       float* xbc = static_cast<float*>(e->rec_a.p);
       float* yr = static_cast<float*>(e->rec_b.p);
       RC(gemm(dtype, e->h.p, A.w_in, proj, T, W, ssd_proj_row(A), st));
-      e->mark(KLLM_SEQ_PHASE_IN_PROJ);
+      mark(KLLM_SEQ_PHASE_IN_PROJ);
       RC(launch_ssd_conv(A, proj, e->ssd_conv[r], step_rows, xbc, T, st));
-      e->mark(KLLM_SEQ_PHASE_QK_PREPARE);
-      RC(launch_ssd_scan(A, proj, xbc, e->ssd_state[r], step_rows, d_eseq, max_count, T, static_cast<float*>(e->ws.p), yr, st));
-      RC(launch_ssd_out(dtype, A, yr, proj, d.norm_eps, e->att.p, T, st));
-      e->mark(KLLM_SEQ_PHASE_ATTENTION);
-      RC(gemm(dtype, e->att.p, A.w_out, yout, T, ssd_inner(A), W, st));
-      e->mark(KLLM_SEQ_PHASE_OUT_PROJ);
+      mark(KLLM_SEQ_PHASE_QK_PREPARE);
+      RC(launch_ssd_scan(A, proj, xbc, e->ssd_state[r], step_rows, d_eseq, max_count, T, room.ws, yr, st));
+      RC(launch_ssd_out(dtype, A, yr, proj, d.norm_eps, room.att, T, st));
+      mark(KLLM_SEQ_PHASE_ATTENTION);
+      RC(gemm(dtype, room.att, A.w_out, yout, T, ssd_inner(A), W, st));
+      mark(KLLM_SEQ_PHASE_OUT_PROJ);
     } else {
       const kllm_seq_delta& A = L.delta;
       float* prep = static_cast<float*>(e->rec_a.p);
       float* o = static_cast<float*>(e->rec_b.p);
       const int n_proj = 2 * A.kv_heads * A.dim + A.heads * A.vdim + A.heads + A.decay_rank + A.gate_rank;
       RC(gemm(dtype, e->h.p, A.w_in, proj, T, W, n_proj, st));
-      e->mark(KLLM_SEQ_PHASE_IN_PROJ);
+      mark(KLLM_SEQ_PHASE_IN_PROJ);
       // the second low-rank projections of the decays and the gates: one product on the low-rank rows in the compute type
       float* low2 = static_cast<float*>(e->rec_c.p);
-      RC(launch_delta_low(dtype, A, proj, e->q.p, T, st));
-      RC(gemm(dtype, e->q.p, A.w_low2, low2, T, A.decay_rank + A.gate_rank, A.heads * (A.dim + A.vdim), st));
+      RC(launch_delta_low(dtype, A, proj, room.q, T, st));
+      RC(gemm(dtype, room.q, A.w_low2, low2, T, A.decay_rank + A.gate_rank, A.heads * (A.dim + A.vdim), st));
       RC(launch_delta_prepare(A, proj, low2, e->delta_conv[r], step_rows, prep, T, st));
-      e->mark(KLLM_SEQ_PHASE_QK_PREPARE);
-      RC(launch_delta_rule(A, prep, e->delta_state[r], step_rows, d_eseq, max_count, T, static_cast<float*>(e->ws.p), o, st));
-      RC(launch_delta_out(dtype, A, o, prep, d.norm_eps, e->att.p, T, st));
-      e->mark(KLLM_SEQ_PHASE_ATTENTION);
-      RC(gemm(dtype, e->att.p, A.w_out, yout, T, A.heads * A.vdim, W, st));
-      e->mark(KLLM_SEQ_PHASE_OUT_PROJ);
+      mark(KLLM_SEQ_PHASE_QK_PREPARE);
+      RC(launch_delta_rule(A, prep, e->delta_state[r], step_rows, d_eseq, max_count, T, room.ws, o, st));
+      RC(launch_delta_out(dtype, A, o, prep, d.norm_eps, room.att, T, st));
+      mark(KLLM_SEQ_PHASE_ATTENTION);
+      RC(gemm(dtype, room.att, A.w_out, yout, T, A.heads * A.vdim, W, st));
+      mark(KLLM_SEQ_PHASE_OUT_PROJ);
     }
     return 0;
   };
+  const MixerRoom room1{proj, 0, e->q.p, e->att.p, static_cast<float*>(e->ws.p), st};
+  const MixerRoom room2{static_cast<float*>(e->proj2.p), 0, e->q2.p, e->att2.p, static_cast<float*>(e->ws2.p), st};
   // the feed-forward of layer L on the rows in e->h: its output goes to `yout`, a shared expert's (when it did not ride
   // along with the routed ones) to y2 with *shared_out set; the router has already run
   auto run_ff = [&](const kllm_seq_layer& L, float* yout, bool* shared_out) -> int {
@@ -1030,7 +1082,7 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
       const kllm_seq_layer& L = e->layers[e->run_layer[r]];
       RC(launch_streams(boundary(open, &L.hyper_mixer, nw(L.pre_mixer), e->h.p), st));
       e->mark(KLLM_SEQ_PHASE_NORM);
-      RC(run_mixer(L, L.mixer_kind, r, y));
+      RC(run_mixer(L, L.mixer_kind, r, room1, y));
       open = &L.hyper_mixer;
       if (L.ff_kind != KLLM_SEQ_FF_NONE) {
         RC(launch_streams(boundary(open, &L.hyper_ff, nw(L.pre_ff), e->h.p), st));
@@ -1058,8 +1110,34 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
     const kllm_seq_layer& L = e->layers[e->run_layer[r]];
     if (!pre_done) RC(launch_pre(ResidNormArgs{}, r, KLLM_SEQ_PHASE_NORM));
     pre_done = false;
-    RC(run_mixer(L, L.mixer_kind, r, y));
-    if (L.mixer2_kind != 0) RC(run_mixer(L, L.mixer2_kind, r, y3));
+    if (L.mixer2_kind == 0) {
+      RC(run_mixer(L, L.mixer_kind, r, room1, y));
+    } else {
+      // The two mixers read the same rows and meet in the sum: the second runs on a stream of its own beside the first.  Input
+      // projections that are stacked in memory are one product ahead of both.
+      MixerRoom a1 = room1, a2 = room2;
+      if (const int n1 = stacked_rows(d, L); n1 > 0) {
+        const int row = n1 + linear_proj_rows(L.linear);
+        RC(gemm(dtype, e->h.p, L.attn.w_in, a1.proj, T, W, row, st));
+        e->mark(KLLM_SEQ_PHASE_IN_PROJ);
+        a1.row = a2.row = row, a2.proj = a1.proj + n1;
+      }
+      // (other kinds of mixer share the recurrences' scratch rows; phases are timed one after the other)
+      const bool beside = L.mixer_kind == KLLM_SEQ_MIXER_ATTENTION && e->prof_out == nullptr;
+      if (beside) {
+        a2.st = e->side;
+        CU(cudaEventRecord(e->fork, st));
+        CU(cudaStreamWaitEvent(e->side, e->fork, 0));
+      }
+      const int rc1 = run_mixer(L, L.mixer_kind, r, a1, y);
+      const int rc2 = rc1 == 0 ? run_mixer(L, L.mixer2_kind, r, a2, y3) : 0;
+      if (beside) {  // join even when a launch failed: nothing of this step may still run when the call returns
+        CU(cudaEventRecord(e->join, e->side));
+        CU(cudaStreamWaitEvent(st, e->join, 0));
+      }
+      RC(rc1);
+      RC(rc2);
+    }
     // what the mixers add to x: c1 y (+ c3 y3)
     ResidNormArgs mixed{};
     mixed.y1 = y;

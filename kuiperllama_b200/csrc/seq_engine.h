@@ -167,7 +167,7 @@ struct ResidNormArgs {
 };
 int launch_resid_norm(const ResidNormArgs& a, cudaStream_t s);
 
-// qkvg: [T, heads*dim + kv_heads*dim + (kv_heads / v_share)*vdim + gate_floats()] fp32 (projection output).
+// qkvg: [T, heads*dim + kv_heads*dim + (kv_heads / v_share)*vdim + gate_floats()] fp32 (projection output), rows `stride` floats apart.
 // Writes q [T, heads, dim] (compute type; head norm, rotation, temperature applied), the key / value rows into the pages,
 // and the gates sigmoid(.) [T, gate_floats()] fp32.  qk_norm KLLM_SEQ_QKNORM_WEIGHTED norms before the rotation,
 // KLLM_SEQ_QKNORM_UNIT after it.  With v_share > 1 the projection's query rows are head by head [map 0 | map 1 ...] and q
@@ -181,7 +181,7 @@ struct ValueBlend {
   float lambda;
   float* rows;   // [T, value row] fp32
 };
-int launch_qk_prepare(int dtype, const AttnShape& a, const RopeArgs& rope, const float* qkvg, const float* qnorm_w,
+int launch_qk_prepare(int dtype, const AttnShape& a, const RopeArgs& rope, const float* qkvg, int stride, const float* qnorm_w,
                       const float* knorm_w, float eps, const int32_t* tok_seq, const int32_t* tok_pos, void* q, float* gates,
                       const PagedKV& kv, const ValueBlend& blend, int T, cudaStream_t s);
 // Differential attention: joins the key splits of both maps of every head (a.no_merge left them in `ws`), then
@@ -267,6 +267,11 @@ size_t linear_attention_scratch_bytes(int heads, int dim, int vdim, int T, int n
 int launch_linear_attention(const kllm_seq_linear& m, const float* proj, int row, float* state, int n_entries,
                             const int32_t* ent_first, const int32_t* ent_count, const int32_t* ent_seq,
                             const int32_t* ent_pos0, int max_count, float* scratch, float* o, cudaStream_t s);
+// Steps of single tokens whose heads are normed one by one: recurrence, norm, gate and conversion in one kernel (out [T, heads *
+// vdim] in the compute type).
+bool linear_token_usable(const kllm_seq_linear& m);
+int launch_linear_token(int dtype, const kllm_seq_linear& m, const float* proj, int row, float* state, const int32_t* tok_seq,
+                        const int32_t* tok_pos, float eps, void* out, int T, cudaStream_t s);
 // out[t] = norm(o[t]) * act(gate rows of proj[t]) in the compute type
 int launch_linear_out(int dtype, const kllm_seq_linear& m, const float* o, const float* proj, int row, float eps, void* out, int T,
                       cudaStream_t s);

@@ -14,6 +14,7 @@
 
 #include <cfloat>
 #include <cstdint>
+#include <initializer_list>
 
 #include "seq_engine.h"
 #include "seq_merge.cuh"
@@ -457,6 +458,102 @@ __global__ void resid_norm_kernel(ResidNormArgs a) {
   route_token(a.router, buf, buf + W, r, W);
 }
 
+// The same step for rows whose columns fit the CTA's registers (NV 16-byte vectors per thread) and that neither route nor shift
+// nor norm the addends one by one: every load of the row is in flight before the first reduction, the sums go through shared
+// memory once each, and nothing else does.
+template <int NV>
+__device__ __forceinline__ void reg_stats(const float4 (&v)[NV], int n4, int W, int kind, float eps, float* red, float& mean,
+                                          float& rstd) {
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  const float inv_w = 1.0f / static_cast<float>(W);
+  mean = 0.f;
+  if (kind == KLLM_SEQ_NORM_LAYER) {
+    float s = 0.f;
+#pragma unroll
+    for (int k = 0; k < NV; ++k)
+      if (static_cast<int>(threadIdx.x + k * blockDim.x) < n4) s += (v[k].x + v[k].y) + (v[k].z + v[k].w);
+    s = warp_sum(s);
+    if (lane == 0) red[warp] = s;
+    __syncthreads();
+    s = 0.f;
+    for (int i = 0; i < nw; ++i) s += red[i];
+    mean = s * inv_w;
+  }
+  float q = 0.f;
+#pragma unroll
+  for (int k = 0; k < NV; ++k)
+    if (static_cast<int>(threadIdx.x + k * blockDim.x) < n4) {
+      const float a = v[k].x - mean, b = v[k].y - mean, c = v[k].z - mean, d = v[k].w - mean;
+      q = fmaf(a, a, fmaf(b, b, fmaf(c, c, fmaf(d, d, q))));
+    }
+  q = warp_sum(q);
+  if (lane == 0) red[32 + warp] = q;
+  __syncthreads();
+  q = 0.f;
+  for (int i = 0; i < nw; ++i) q += red[32 + i];
+  rstd = 1.0f / sqrtf(q * inv_w + eps);
+}
+__device__ __forceinline__ float4 scaled(float c, const float4& a) { return make_float4(c * a.x, c * a.y, c * a.z, c * a.w); }
+__device__ __forceinline__ void add_scaled(float4& s, float c, const float4& a) {
+  s.x = fmaf(c, a.x, s.x), s.y = fmaf(c, a.y, s.y), s.z = fmaf(c, a.z, s.z), s.w = fmaf(c, a.w, s.w);
+}
+__device__ __forceinline__ float4 normed4(const float4& v, float mean, float rstd, const float* w, const float* b, int i) {
+  const float4 g = *reinterpret_cast<const float4*>(w + i);
+  const float4 o = b ? *reinterpret_cast<const float4*>(b + i) : make_float4(0.f, 0.f, 0.f, 0.f);
+  return make_float4((v.x - mean) * rstd * g.x + o.x, (v.y - mean) * rstd * g.y + o.y, (v.z - mean) * rstd * g.z + o.z,
+                     (v.w - mean) * rstd * g.w + o.w);
+}
+__device__ __forceinline__ void put4(float* dst, const float4& v) { *reinterpret_cast<float4*>(dst) = v; }
+__device__ __forceinline__ void put4(__nv_bfloat16* dst, const float4& v) {
+  const __nv_bfloat162 a = __floats2bfloat162_rn(v.x, v.y), b = __floats2bfloat162_rn(v.z, v.w);
+  *reinterpret_cast<uint2*>(dst) = make_uint2(*reinterpret_cast<const uint32_t*>(&a), *reinterpret_cast<const uint32_t*>(&b));
+}
+
+template <typename AT, int NV>
+__global__ void __launch_bounds__(512) resid_rows_kernel(ResidNormArgs a) {
+  __shared__ float red_post[64], red_pre[64];
+  const int W = a.width, n4 = W / 4, r = blockIdx.x;
+  const size_t src = static_cast<size_t>(a.rows ? a.rows[r] : r) * W, dst = static_cast<size_t>(r) * W;
+  auto at = [](const float* p, size_t i) { return *reinterpret_cast<const float4*>(p + i); };
+  float4 x[NV], u[NV];
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = (threadIdx.x + k * blockDim.x) * 4;
+    x[k] = u[k] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (i >= W) continue;
+    x[k] = at(a.x, src + i);
+    if (a.y1) u[k] = scaled(a.c1, at(a.y1, src + i));
+    if (a.y1 && a.y3) add_scaled(u[k], a.c3, at(a.y3, src + i));
+    if (a.y1 && a.y2) add_scaled(u[k], a.s2 ? a.s2[r] : 1.0f, at(a.y2, src + i));
+    if (a.y1 && a.y4) add_scaled(u[k], a.c4, at(a.y4, src + i));
+  }
+  const bool post = a.y1 != nullptr && a.post.w != nullptr;
+  float mean = 0.f, rstd = 1.0f;
+  if (post) reg_stats<NV>(u, n4, W, a.post.kind, a.eps, red_post, mean, rstd);
+  const bool changes = !a.rows && (a.y1 != nullptr || a.add != nullptr || a.add_rows != nullptr);
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = (threadIdx.x + k * blockDim.x) * 4;
+    if (i >= W) continue;
+    add_scaled(x[k], 1.0f, post ? normed4(u[k], mean, rstd, a.post.w, a.post.b, i) : u[k]);
+    if (a.add_rows) add_scaled(x[k], 1.0f, at(a.add_rows, src + i));
+    if (a.add) add_scaled(x[k], 1.0f, at(a.add, i));
+    if (changes) put4(a.x + dst + i, x[k]);
+  }
+  if (a.out == nullptr) return;
+  const bool plain = a.pre.kind == KLLM_SEQ_NORM_NONE;
+  if (!plain) {
+    if (a.pre.w == nullptr) return;
+    reg_stats<NV>(x, n4, W, a.pre.kind, a.eps, red_pre, mean, rstd);
+  }
+  AT* out = static_cast<AT*>(a.out) + dst;
+#pragma unroll
+  for (int k = 0; k < NV; ++k) {
+    const int i = (threadIdx.x + k * blockDim.x) * 4;
+    if (i < W) put4(out + i, plain ? x[k] : normed4(x[k], mean, rstd, a.pre.w, a.pre.b, i));
+  }
+}
+
 // One CTA per row; the CTA of an entry's first row also moves the entry's last h into the state (it alone touches it).
 template <typename AT>
 __global__ void token_shift_kernel(const float* __restrict__ h, const float* __restrict__ mu, float* __restrict__ state,
@@ -497,7 +594,7 @@ __device__ __forceinline__ AT* page_row(AT* base, const PagedKV& kv, int seq, in
 // it), temperature -- and leaves as a query row or as the key row of the token's page.  Angles, cos and sin are fp32.
 // One norm over all query rows (and one over all key rows) takes its two sums of squares over the CTA first.
 template <typename AT>
-__global__ void qk_prepare_kernel(AttnShape a, RopeArgs rope, const float* __restrict__ qkvg,
+__global__ void qk_prepare_kernel(AttnShape a, RopeArgs rope, const float* __restrict__ qkvg, int stride,
                                   const float* __restrict__ qnorm_w, const float* __restrict__ knorm_w, float eps,
                                   const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ tok_pos,
                                   AT* __restrict__ q, float* __restrict__ gates, PagedKV kv, ValueBlend blend) {
@@ -506,7 +603,6 @@ __global__ void qk_prepare_kernel(AttnShape a, RopeArgs rope, const float* __res
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
   const int maps = v_share_of(a);
   const int qn = a.heads * a.dim, kn = a.kv_heads * a.dim, vn = a.kv_heads / maps * a.vdim, gn = gate_floats(a);
-  const int stride = qn + kn + vn + gn;
   const float* row = qkvg + static_cast<size_t>(t) * stride;
   const int seq = tok_seq[t], pos = tok_pos[t];
   float temp = 1.0f;
@@ -577,6 +673,102 @@ __global__ void qk_prepare_kernel(AttnShape a, RopeArgs rope, const float* __res
     gates[static_cast<size_t>(t) * gn + i] = 1.0f / (1.0f + expf(-row[qn + kn + vn + i]));
 }
 
+// The same with 16-byte accesses for head sizes that are multiples of 4 and halves paired (or no rotation): G lanes share a head,
+// a lane owns four coordinates of its first half and the four they turn with (or four that do not turn).  The angles of the
+// token's position are taken once, into shared memory; all heads read them from there.
+template <typename AT, int G>
+__global__ void __launch_bounds__(512)
+qk_turn_kernel(AttnShape a, RopeArgs rope, const float* __restrict__ qkvg, int stride, const float* __restrict__ qnorm_w,
+               const float* __restrict__ knorm_w, float eps, const int32_t* __restrict__ tok_seq,
+               const int32_t* __restrict__ tok_pos, AT* __restrict__ q, float* __restrict__ gates, PagedKV kv) {
+  extern __shared__ __align__(16) float turn[];  // [half] cos, [half] sin
+  __shared__ float red[2][32];
+  const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
+  const int qn = a.heads * a.dim, kn = a.kv_heads * a.dim, vn = a.kv_heads * a.vdim, gn = gate_floats(a);
+  const float* row = qkvg + static_cast<size_t>(t) * stride;
+  const int seq = tok_seq[t], pos = tok_pos[t];
+  const int half = rope.dims / 2;
+  float* co = turn;
+  float* si = turn + half;
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    const float freq = rope.freq ? rope.freq[i] : powf(rope.base, -2.0f * static_cast<float>(i) / static_cast<float>(rope.dims));
+    const float ang = static_cast<float>(pos) * freq;
+    co[i] = cosf(ang) * rope.mag, si[i] = sinf(ang) * rope.mag;
+  }
+  const bool whole = a.qk_norm == KLLM_SEQ_QKNORM_PROJECTION, weighted = whole || a.qk_norm == KLLM_SEQ_QKNORM_WEIGHTED;
+  float sq = 0.f, sk = 0.f;
+  if (whole) {
+    for (int i = threadIdx.x * 4; i < qn + kn; i += blockDim.x * 4) {
+      const float4 v = *reinterpret_cast<const float4*>(row + i);
+      const float ss = fmaf(v.x, v.x, fmaf(v.y, v.y, fmaf(v.z, v.z, v.w * v.w)));
+      if (i < qn) sq += ss;
+      else sk += ss;
+    }
+    sq = warp_sum(sq), sk = warp_sum(sk);
+    if (lane == 0) red[0][warp] = sq, red[1][warp] = sk;
+  }
+  __syncthreads();
+  float rq = 1.0f, rk = 1.0f;
+  if (whole) {
+    sq = 0.f, sk = 0.f;
+    for (int i = 0; i < nw; ++i) sq += red[0][i], sk += red[1][i];
+    rq = 1.0f / sqrtf(sq / static_cast<float>(qn) + eps);
+    rk = 1.0f / sqrtf(sk / static_cast<float>(kn) + eps);
+  }
+  const float temp = a.temp_every > 0 ? 1.0f + a.temp_coef * logf(static_cast<float>((pos + 1) / a.temp_every) + 1.0f) : 1.0f;
+  AT* krow = page_row(static_cast<AT*>(kv.k), kv, seq, pos, a.kv_heads, a.dim);
+  AT* vrow = page_row(static_cast<AT*>(kv.v), kv, seq, pos, a.kv_heads, a.vdim);
+  const float inv_dim = 1.0f / static_cast<float>(a.dim);
+  const int pairs = half / 4, rest = (a.dim - 2 * half) / 4;  // units of a head: pairs of quads, then quads
+  const int gl = threadIdx.x % G, group = threadIdx.x / G, groups = blockDim.x / G;
+  // the quads of this lane: first coordinate of each (-1: none)
+  const bool turns = gl < pairs;
+  const int d0 = turns ? 4 * gl : (gl - pairs < rest ? 2 * half + 4 * (gl - pairs) : -1), d1 = turns ? half + 4 * gl : -1;
+  const int total = a.heads + a.kv_heads;
+  for (int u0 = 0; u0 < total; u0 += groups) {  // every lane of a warp walks the same rounds: the shuffles need them all
+    const int u = u0 + group;
+    const bool live = u < total, is_q = u < a.heads;
+    const float* src = row + (is_q ? u * a.dim : qn + (u - a.heads) * a.dim);
+    float4 x = make_float4(0.f, 0.f, 0.f, 0.f), y = x;
+    if (live && d0 >= 0) x = *reinterpret_cast<const float4*>(src + d0);
+    if (live && d1 >= 0) y = *reinterpret_cast<const float4*>(src + d1);
+    auto head_ss = [&]() {
+      float ss = fmaf(x.x, x.x, fmaf(x.y, x.y, fmaf(x.z, x.z, x.w * x.w))) + fmaf(y.x, y.x, fmaf(y.y, y.y, fmaf(y.z, y.z, y.w * y.w)));
+#pragma unroll
+      for (int o = G / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(kAll, ss, o);
+      return ss;
+    };
+    float rinv = is_q ? rq : rk;
+    if (a.qk_norm == KLLM_SEQ_QKNORM_WEIGHTED) rinv = 1.0f / sqrtf(head_ss() * inv_dim + eps);
+    if (weighted && live) {
+      const float* w = (is_q ? qnorm_w : knorm_w) + (whole ? (is_q ? u : u - a.heads) * a.dim : 0);
+      if (d0 >= 0) {
+        const float4 g = *reinterpret_cast<const float4*>(w + d0);
+        x = make_float4(x.x * rinv * g.x, x.y * rinv * g.y, x.z * rinv * g.z, x.w * rinv * g.w);
+      }
+      if (d1 >= 0) {
+        const float4 g = *reinterpret_cast<const float4*>(w + d1);
+        y = make_float4(y.x * rinv * g.x, y.y * rinv * g.y, y.z * rinv * g.z, y.w * rinv * g.w);
+      }
+    }
+    if (turns) {
+      const float4 c = *reinterpret_cast<const float4*>(co + d0), z = *reinterpret_cast<const float4*>(si + d0);
+      const float4 n = make_float4(x.x * c.x - y.x * z.x, x.y * c.y - y.y * z.y, x.z * c.z - y.z * z.z, x.w * c.w - y.w * z.w);
+      y = make_float4(y.x * c.x + x.x * z.x, y.y * c.y + x.y * z.y, y.z * c.z + x.z * z.z, y.w * c.w + x.w * z.w);
+      x = n;
+    }
+    float post = is_q ? temp : 1.0f;
+    if (a.qk_norm == KLLM_SEQ_QKNORM_UNIT) post *= 1.0f / sqrtf(head_ss() * inv_dim + eps);
+    if (!live) continue;
+    AT* dst = is_q ? q + (static_cast<size_t>(t) * a.heads + u) * a.dim : krow + (u - a.heads) * a.dim;
+    if (d0 >= 0) put4(dst + d0, scaled(post, x));
+    if (d1 >= 0) put4(dst + d1, scaled(post, y));
+  }
+  for (int i = threadIdx.x * 4; i < vn; i += blockDim.x * 4) put4(vrow + i, *reinterpret_cast<const float4*>(row + qn + kn + i));
+  for (int i = threadIdx.x; i < gn; i += blockDim.x)
+    gates[static_cast<size_t>(t) * gn + i] = 1.0f / (1.0f + expf(-row[qn + kn + vn + i]));
+}
+
 // The same for heads without rotation, temperature or maps, normed over the whole projection or not at all: nothing is done
 // per head then, so the row is walked straight through, V columns at a time -- sums of squares, then query rows out, key and
 // value rows into the page, gates.
@@ -599,14 +791,14 @@ template <> __device__ __forceinline__ void get_cols<4>(const float* src, float*
 template <> __device__ __forceinline__ void get_cols<1>(const float* src, float* v) { v[0] = *src; }
 
 template <typename AT, int V>
-__global__ void qk_rows_kernel(AttnShape a, const float* __restrict__ qkvg, const float* __restrict__ qnorm_w,
+__global__ void qk_rows_kernel(AttnShape a, const float* __restrict__ qkvg, int stride, const float* __restrict__ qnorm_w,
                                const float* __restrict__ knorm_w, float eps, const int32_t* __restrict__ tok_seq,
                                const int32_t* __restrict__ tok_pos, AT* __restrict__ q, float* __restrict__ gates, PagedKV kv,
                                ValueBlend blend) {
   __shared__ float red[2][32];
   const int t = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
   const int qn = a.heads * a.dim, kn = a.kv_heads * a.dim, vn = a.kv_heads * a.vdim, gn = gate_floats(a);
-  const float* row = qkvg + static_cast<size_t>(t) * (qn + kn + vn + gn);
+  const float* row = qkvg + static_cast<size_t>(t) * stride;
   const int seq = tok_seq[t], pos = tok_pos[t];
   AT* krow = page_row(static_cast<AT*>(kv.k), kv, seq, pos, a.kv_heads, a.dim);
   AT* vrow = page_row(static_cast<AT*>(kv.v), kv, seq, pos, a.kv_heads, a.vdim);
@@ -1311,6 +1503,25 @@ int launch_resid_norm(const ResidNormArgs& a, cudaStream_t s) {
   if (smem > 200 * 1024) return KLLM_E_UNSUPPORTED;
   if (a.router.w_router && (a.router.top > a.router.experts || a.router.experts <= 0 || a.router.top <= 0 || !a.pre.w))
     return KLLM_E_INVALID;
+  auto aligned = [](std::initializer_list<const void*> ps) {
+    uintptr_t bits = 0;
+    for (const void* p : ps) bits |= reinterpret_cast<uintptr_t>(p);
+    return (bits & 15) == 0;
+  };
+  if (!a.router.w_router && !a.shift.mu && !a.out_f32 && !a.n1.w && !a.n3.w && a.width % 4 == 0 && a.width <= 512 * 16 &&
+      aligned({a.x, a.y1, a.y2, a.y3, a.y4, a.add, a.add_rows, a.post.w, a.post.b, a.pre.w, a.pre.b, a.out})) {
+    // few rows: as many threads as the row has vectors; many: 256 threads and the row's vectors in each thread's registers
+    const int n4 = a.width / 4;
+    int threads = std::min((n4 + 31) / 32 * 32, a.T <= 64 ? 512 : 256);
+    const int nv = (n4 + threads - 1) / threads;
+    if (nv > 4) threads = 512;
+#define KLLM_RESID_ROWS(N) KLLM_SEQ_DISPATCH(a.dtype, (resid_rows_kernel<AT, N><<<a.T, threads, 0, s>>>(a)))
+    if (nv <= 1) KLLM_RESID_ROWS(1);
+    else if (nv <= 2) KLLM_RESID_ROWS(2);
+    else KLLM_RESID_ROWS(4);
+#undef KLLM_RESID_ROWS
+    return done();
+  }
   const int threads = a.width >= 1024 ? 256 : 128;
   if (smem > 48 * 1024) {
     KLLM_SEQ_DISPATCH(a.dtype, (cudaFuncSetAttribute(resid_norm_kernel<AT>, cudaFuncAttributeMaxDynamicSharedMemorySize,
@@ -1320,7 +1531,7 @@ int launch_resid_norm(const ResidNormArgs& a, cudaStream_t s) {
   return done();
 }
 
-int launch_qk_prepare(int dtype, const AttnShape& a, const RopeArgs& rope_, const float* qkvg, const float* qnorm_w,
+int launch_qk_prepare(int dtype, const AttnShape& a, const RopeArgs& rope_, const float* qkvg, int stride, const float* qnorm_w,
                       const float* knorm_w, float eps, const int32_t* tok_seq, const int32_t* tok_pos, void* q, float* gates,
                       const PagedKV& kv, const ValueBlend& blend, int T, cudaStream_t s) {
   RopeArgs rope = rope_;
@@ -1331,14 +1542,29 @@ int launch_qk_prepare(int dtype, const AttnShape& a, const RopeArgs& rope_, cons
   if (rope.dims == 0 && a.temp_every == 0 && v_share_of(a) == 1 &&
       (a.qk_norm == KLLM_SEQ_QKNORM_PROJECTION || a.qk_norm == KLLM_SEQ_QKNORM_NONE)) {
     const int qn = a.heads * a.dim, kn = a.kv_heads * a.dim, vn = a.kv_heads * a.vdim;
-    const bool vec = qn % 4 == 0 && kn % 4 == 0 && vn % 4 == 0 && gate_floats(a) % 4 == 0;
+    const bool vec = qn % 4 == 0 && kn % 4 == 0 && vn % 4 == 0 && stride % 4 == 0 && (reinterpret_cast<uintptr_t>(qkvg) & 15) == 0;
     const int threads = T <= 16 ? 512 : 256;
     if (vec)
-      KLLM_SEQ_DISPATCH(dtype, (qk_rows_kernel<AT, 4><<<T, threads, 0, s>>>(a, qkvg, qnorm_w, knorm_w, eps, tok_seq, tok_pos,
+      KLLM_SEQ_DISPATCH(dtype, (qk_rows_kernel<AT, 4><<<T, threads, 0, s>>>(a, qkvg, stride, qnorm_w, knorm_w, eps, tok_seq, tok_pos,
                                                                             static_cast<AT*>(q), gates, kv, blend)));
     else
-      KLLM_SEQ_DISPATCH(dtype, (qk_rows_kernel<AT, 1><<<T, threads, 0, s>>>(a, qkvg, qnorm_w, knorm_w, eps, tok_seq, tok_pos,
+      KLLM_SEQ_DISPATCH(dtype, (qk_rows_kernel<AT, 1><<<T, threads, 0, s>>>(a, qkvg, stride, qnorm_w, knorm_w, eps, tok_seq, tok_pos,
                                                                             static_cast<AT*>(q), gates, kv, blend)));
+    return done();
+  }
+  const int half = rope.dims / 2, units = half / 4 + (a.dim - rope.dims) / 4;
+  if (v_share_of(a) == 1 && blend.mode == KLLM_SEQ_VBLEND_NONE && a.dim % 4 == 0 && half % 4 == 0 && a.vdim % 4 == 0 &&
+      (rope.dims == 0 || rope.pairing == KLLM_SEQ_ROPE_HALVES) && units <= 32 && stride % 4 == 0 &&
+      (reinterpret_cast<uintptr_t>(qkvg) & 15) == 0) {
+    const int threads = T <= 64 ? 512 : 256;
+    const size_t smem = std::max<size_t>(16, 2 * static_cast<size_t>(half) * sizeof(float));
+#define KLLM_QK_TURN(G)                                                                                                   \
+  KLLM_SEQ_DISPATCH(dtype, (qk_turn_kernel<AT, G><<<T, threads, smem, s>>>(a, rope, qkvg, stride, qnorm_w, knorm_w, eps, tok_seq, \
+                                                                          tok_pos, static_cast<AT*>(q), gates, kv)))
+    if (units <= 8) KLLM_QK_TURN(8);
+    else if (units <= 16) KLLM_QK_TURN(16);
+    else KLLM_QK_TURN(32);
+#undef KLLM_QK_TURN
     return done();
   }
   // a warp per head: few tokens get as many warps as there are query and key heads (at most 16: the kernel's registers
@@ -1346,7 +1572,7 @@ int launch_qk_prepare(int dtype, const AttnShape& a, const RopeArgs& rope_, cons
   int warps = T <= 64 ? std::min(16, std::max(4, a.heads + a.kv_heads)) : 4;
   warps = std::max(1, std::min(warps, 48 * 1024 / (4 * a.dim)));
   const size_t smem = static_cast<size_t>(warps) * a.dim * sizeof(float);
-  KLLM_SEQ_DISPATCH(dtype, (qk_prepare_kernel<AT><<<T, 32 * warps, smem, s>>>(a, rope, qkvg, qnorm_w, knorm_w, eps, tok_seq,
+  KLLM_SEQ_DISPATCH(dtype, (qk_prepare_kernel<AT><<<T, 32 * warps, smem, s>>>(a, rope, qkvg, stride, qnorm_w, knorm_w, eps, tok_seq,
                                                                              tok_pos, static_cast<AT*>(q), gates, kv, blend)));
   return done();
 }

@@ -777,6 +777,103 @@ linear_chunk_out_kernel(int heads, int dim, int vdim, const float* __restrict__ 
   }
 }
 
+// One token per entry (decode steps), heads normed one by one: a CTA per (head, token) reads the head's state once, 16 bytes per
+// lane, writes it back, and has the head's whole output -- its norm, the gate and the conversion follow in place.  A thread owns
+// V columns and every slices-th row; kLinTokenLoads rows of it are in flight before the projections are read.
+constexpr int kLinTokenLoads = 8;
+template <typename AT, int V>
+__global__ void __launch_bounds__(512)
+linear_token_kernel(int heads, int dim, int vdim, const float* __restrict__ decay, LinearRot rot, int silu,
+                    const float* __restrict__ proj, int stride, int gate_act, float eps, float* __restrict__ state,
+                    const int32_t* __restrict__ tok_seq, const int32_t* __restrict__ tok_pos, AT* __restrict__ out) {
+  extern __shared__ __align__(16) float sm[];
+  __shared__ float red[33];
+  const int h = blockIdx.x, t = blockIdx.y, tid = threadIdx.x;
+  const int dp = (dim + 3) & ~3, units = vdim / V, slices = blockDim.x / units;
+  float* qs = sm;                         // [dp]
+  float* ks = qs + dp;                    // [dp]
+  float* vs = ks + dp;                    // [vdim, padded to 4]
+  float* part = vs + ((vdim + 3) & ~3);   // [slices][vdim]
+  const int pos = tok_pos[t];
+  const bool fresh = pos == 0;
+  float* S = state + (static_cast<size_t>(tok_seq[t]) * heads + h) * dim * vdim;
+  const int c = (tid % units) * V, sl = tid / units;
+  const bool works = sl < slices;
+  float s[kLinTokenLoads][V];
+  auto fetch = [&](int d0) {
+#pragma unroll
+    for (int u = 0; u < kLinTokenLoads; ++u) {
+      const int d = d0 + u * slices;
+#pragma unroll
+      for (int z = 0; z < V; ++z) s[u][z] = 0.f;
+      if (!works || fresh || d >= dim) continue;
+      if constexpr (V == 4) {
+        const float4 f = *reinterpret_cast<const float4*>(S + static_cast<size_t>(d) * vdim + c);
+        s[u][0] = f.x, s[u][1] = f.y, s[u][2] = f.z, s[u][3] = f.w;
+      } else {
+        s[u][0] = S[static_cast<size_t>(d) * vdim + c];
+      }
+    }
+  };
+  fetch(sl);
+  const float* row = proj + static_cast<size_t>(t) * stride;
+  const float *q = row + h * dim, *k = q + heads * dim, *v = row + 2 * heads * dim + h * vdim;
+  const int half = rot.rope.dims / 2;
+  const bool pairs = rot.rope.pairing == KLLM_SEQ_ROPE_PAIRS;
+  auto act = [&](float x) { return silu ? siluf(x) : x; };
+  for (int i = tid; i < half; i += blockDim.x) {
+    float co, si;
+    rope_turn(rot.rope, i, pos, co, si);
+    const int d0 = pairs ? 2 * i : i, d1 = pairs ? 2 * i + 1 : i + half;
+    const float q0 = q[d0], q1 = q[d1], k0 = k[d0], k1 = k[d1];
+    qs[d0] = q0 * co - q1 * si, qs[d1] = q1 * co + q0 * si;
+    ks[d0] = (k0 * co - k1 * si) * rot.k_scale, ks[d1] = (k1 * co + k0 * si) * rot.k_scale;
+  }
+  for (int d = 2 * half + tid; d < dim; d += blockDim.x) qs[d] = act(q[d]), ks[d] = act(k[d]) * rot.k_scale;
+  for (int i = tid; i < vdim; i += blockDim.x) vs[i] = act(v[i]);
+  __syncthreads();
+  const float lam = decay[h];
+  if (works) {
+    float acc[V], vc[V];
+#pragma unroll
+    for (int z = 0; z < V; ++z) acc[z] = 0.f, vc[z] = vs[c + z];
+    for (int d0 = sl; d0 < dim; d0 += kLinTokenLoads * slices) {
+      if (d0 != sl) fetch(d0);
+#pragma unroll
+      for (int u = 0; u < kLinTokenLoads; ++u) {
+        const int d = d0 + u * slices;
+        if (d >= dim) break;
+        const float kd = ks[d], qd = qs[d];
+#pragma unroll
+        for (int z = 0; z < V; ++z) {
+          s[u][z] = fmaf(lam, s[u][z], kd * vc[z]);
+          acc[z] = fmaf(qd, s[u][z], acc[z]);
+        }
+        float* dst = S + static_cast<size_t>(d) * vdim + c;
+        if constexpr (V == 4) *reinterpret_cast<float4*>(dst) = make_float4(s[u][0], s[u][1], s[u][2], s[u][3]);
+        else *dst = s[u][0];
+      }
+    }
+#pragma unroll
+    for (int z = 0; z < V; ++z) part[sl * vdim + c + z] = acc[z];
+  }
+  __syncthreads();
+  float ss = 0.f;
+  for (int i = tid; i < vdim; i += blockDim.x) {
+    float o = 0.f;
+    for (int p = 0; p < slices; ++p) o += part[p * vdim + i];
+    vs[i] = o;
+    ss = fmaf(o, o, ss);
+  }
+  const float rinv = 1.0f / sqrtf(block_sum(ss, red) / static_cast<float>(vdim) + eps);
+  const float* g = row + 2 * heads * dim + heads * vdim + h * vdim;
+  for (int i = tid; i < vdim; i += blockDim.x) {
+    const float z = g[i];
+    const float gate = gate_act == KLLM_SEQ_GATEACT_SILU ? siluf(z) : sigmoidf(z);
+    out[(static_cast<size_t>(t) * heads + h) * vdim + i] = from_f<AT>(vs[i] * rinv * gate);
+  }
+}
+
 __device__ __forceinline__ float lin_gate(int act, float g) { return act == KLLM_SEQ_GATEACT_SILU ? siluf(g) : sigmoidf(g); }
 
 // One CTA per token.  ROW: one norm over the row; HEAD: a warp per head, each by its own root mean square.
@@ -999,6 +1096,34 @@ int launch_linear_attention(const kllm_seq_linear& m, const float* proj, int row
   if (m.qkv_act == KLLM_SEQ_QKV_PLAIN)
     return linear_attention_t<false>(m, proj, row, state, n_entries, ent_first, ent_count, ent_seq, ent_pos0, max_count, scratch, o, s);
   return linear_attention_t<true>(m, proj, row, state, n_entries, ent_first, ent_count, ent_seq, ent_pos0, max_count, scratch, o, s);
+}
+
+bool linear_token_usable(const kllm_seq_linear& m) {
+  const int units = m.vdim % 4 == 0 ? m.vdim / 4 : m.vdim;
+  return m.out_norm == KLLM_SEQ_OUTNORM_HEAD && units <= 256;
+}
+
+int launch_linear_token(int dtype, const kllm_seq_linear& m, const float* proj, int row, float* state, const int32_t* tok_seq,
+                        const int32_t* tok_pos, float eps, void* out, int T, cudaStream_t s) {
+  const bool vec = m.vdim % 4 == 0;
+  const int units = vec ? m.vdim / 4 : m.vdim;
+  int threads = 128;
+  while (threads < 512 && (threads < units || threads / units * kLinTokenLoads < m.dim)) threads *= 2;
+  const size_t smem = (2 * static_cast<size_t>((m.dim + 3) & ~3) + ((m.vdim + 3) & ~3) + static_cast<size_t>(threads / units) * m.vdim) *
+                      sizeof(float);
+  if (T > 65535 || smem > 48 * 1024) return KLLM_E_UNSUPPORTED;
+  const dim3 grid(m.heads, T);
+  const LinearRot rot = linear_rot(m);
+  const int silu = m.qkv_act == KLLM_SEQ_QKV_SILU;
+  if (vec)
+    KLLM_SEQ_DISPATCH(dtype, (linear_token_kernel<AT, 4><<<grid, threads, smem, s>>>(m.heads, m.dim, m.vdim, m.decay, rot, silu, proj, row,
+                                                                                    m.gate_act, eps, state, tok_seq, tok_pos,
+                                                                                    static_cast<AT*>(out))));
+  else
+    KLLM_SEQ_DISPATCH(dtype, (linear_token_kernel<AT, 1><<<grid, threads, smem, s>>>(m.heads, m.dim, m.vdim, m.decay, rot, silu, proj, row,
+                                                                                    m.gate_act, eps, state, tok_seq, tok_pos,
+                                                                                    static_cast<AT*>(out))));
+  return done();
 }
 
 int launch_linear_out(int dtype, const kllm_seq_linear& m, const float* o, const float* proj, int row, float eps, void* out, int T,

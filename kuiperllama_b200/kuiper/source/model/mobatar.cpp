@@ -112,7 +112,7 @@ base::Status MobatarModel::build_attention(const json::Value& c, const Safetenso
     return bad(p, "tensor shapes do not fit the configuration");
   if (st = upload_f32(qnorm, qn, &a->q_norm_w); !st) return st;
   if (st = upload_f32(knorm, kn, &a->k_norm_w); !st) return st;
-  return upload_compute({q, k, v, g}, width_, &a->w_in);
+  return base::error::Success();  // the input projection is stacked with the other mixer's
 }
 
 base::Status MobatarModel::build_retention(const json::Value& c, const SafetensorsFile& w, const std::string& p,
@@ -137,8 +137,7 @@ base::Status MobatarModel::build_retention(const json::Value& c, const Safetenso
   if (!shaped(q, qn, width_) || !shaped(k, qn, width_) || !shaped(v, vn, width_) || !shaped(g, vn, width_) ||
       !shaped(o, width_, vn))
     return bad(p, "tensor shapes do not fit the configuration");
-  if (st = upload_compute({q, k, v, g}, width_, &a->w_in); !st) return st;
-  return upload_compute({o}, vn, &a->w_out);
+  return upload_compute({o}, vn, &a->w_out);  // the input projection is stacked with the other mixer's
 }
 
 base::Status MobatarModel::build_latent(const json::Value& c, const SafetensorsFile& w, const std::string& p, kllm_seq_latent* a) {
@@ -251,6 +250,15 @@ base::Status MobatarModel::build(const json::Value& config, const SafetensorsFil
       L.mixer2_scale = static_cast<float>(get_number(mc, "right_scale"));
       if (st = build_attention(mc.at("left"), w, p + "mix.left.", true, &L.attn); !st) return st;
       if (st = build_retention(mc.at("right"), w, p + "mix.right.", &L.linear); !st) return st;
+      // one tensor holds both input projections, so that a step runs them as one product
+      std::vector<const StTensor*> in;
+      for (const char* n : {"left.q", "left.k", "left.v", "left.g", "right.q", "right.k", "right.v", "right.g"})
+        in.push_back(need(w, p + "mix." + n, &st));
+      if (!st) return st;
+      if (st = upload_compute(in, width_, &L.attn.w_in); !st) return st;
+      const int64_t left = int64_t(L.attn.heads + L.attn.kv_heads) * L.attn.dim + int64_t(L.attn.kv_heads) * L.attn.vdim + L.attn.heads;
+      const size_t es = compute_ == ComputeType::kBFloat16 ? 2 : 4;
+      L.linear.w_in = static_cast<const char*>(L.attn.w_in) + static_cast<size_t>(left) * width_ * es;
     } else if (type == "latent_attention") {
       L.mixer_kind = KLLM_SEQ_MIXER_LATENT;
       if (st = build_latent(mc, w, p + "mix.", &L.latent); !st) return st;
