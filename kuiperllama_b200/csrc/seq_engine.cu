@@ -731,7 +731,9 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
     }
   for (const kllm_seq_layer& L : e->layers)  // the chunk sums of linear attention share the attention workspace
     if (L.mixer_kind == KLLM_SEQ_MIXER_LINEAR || L.mixer2_kind == KLLM_SEQ_MIXER_LINEAR)
-      ws_bytes = std::max(ws_bytes, linear_attention_scratch_bytes(L.linear.heads, L.linear.dim, L.linear.vdim, T, n_entries, max_count));
+      ws_bytes = std::max(ws_bytes, linear_mma_usable(dtype, L.linear, max_count)
+                                        ? linear_mma_scratch_bytes(L.linear, T, n_entries)
+                                        : linear_attention_scratch_bytes(L.linear.heads, L.linear.dim, L.linear.vdim, T, n_entries, max_count));
   for (const kllm_seq_layer& L : e->layers)  // and so do the segments of the selective scan
     if (L.mixer_kind == KLLM_SEQ_MIXER_SSM || L.mixer2_kind == KLLM_SEQ_MIXER_SSM)
       ws_bytes = std::max(ws_bytes, ssm_scan_scratch_bytes(L.ssm, T, n_entries, max_count));
@@ -927,17 +929,25 @@ extern "C" int kllm_seq_step(kllm_seq_engine* e, int32_t n_entries, const int32_
       const int n_proj = linear_proj_rows(A), row = room.row > 0 ? room.row : n_proj;
       if (room.row == 0) RC(gemm(dtype, e->h.p, A.w_in, proj, T, W, n_proj, st));
       mark(KLLM_SEQ_PHASE_IN_PROJ);
+      const bool by_head = A.out_norm == KLLM_SEQ_OUTNORM_HEAD;
+      float* o = static_cast<float*>(e->ol.p);
+      bool normed = true;  // the recurrence's kernel has also normed, gated and converted its output
       if (single && linear_token_usable(A)) {
         RC(launch_linear_token(dtype, A, proj, row, e->linear_state[r], d_seq, d_pos, d.norm_eps, room.att, T, st));
+      } else if (linear_mma_usable(dtype, A, max_count)) {
+        RC(launch_linear_mma(A, proj, row, e->linear_state[r], n_entries, d_first, d_count, d_eseq, d_pos0, max_count, T, d.norm_eps,
+                             room.ws, by_head ? nullptr : o, room.att, st));
+        normed = by_head;
       } else {
-      if (linear_attention_rotates(A, max_count)) {
-        RC(launch_linear_rotate(A, proj, row, d_pos, T, st));
-        mark(KLLM_SEQ_PHASE_QK_PREPARE);
+        if (linear_attention_rotates(A, max_count)) {
+          RC(launch_linear_rotate(A, proj, row, d_pos, T, st));
+          mark(KLLM_SEQ_PHASE_QK_PREPARE);
+        }
+        RC(launch_linear_attention(A, proj, row, e->linear_state[r], n_entries, d_first, d_count, d_eseq, d_pos0, max_count, room.ws,
+                                   o, st));
+        normed = false;
       }
-      RC(launch_linear_attention(A, proj, row, e->linear_state[r], n_entries, d_first, d_count, d_eseq, d_pos0, max_count,
-                                 room.ws, static_cast<float*>(e->ol.p), st));
-      RC(launch_linear_out(dtype, A, static_cast<const float*>(e->ol.p), proj, row, d.norm_eps, room.att, T, st));
-      }
+      if (!normed) RC(launch_linear_out(dtype, A, o, proj, row, d.norm_eps, room.att, T, st));
       mark(KLLM_SEQ_PHASE_ATTENTION);
       RC(gemm(dtype, room.att, A.w_out, yout, T, A.heads * A.vdim, W, st));
       mark(KLLM_SEQ_PHASE_OUT_PROJ);

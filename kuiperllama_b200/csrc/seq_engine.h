@@ -267,6 +267,14 @@ size_t linear_attention_scratch_bytes(int heads, int dim, int vdim, int T, int n
 int launch_linear_attention(const kllm_seq_linear& m, const float* proj, int row, float* state, int n_entries,
                             const int32_t* ent_first, const int32_t* ent_count, const int32_t* ent_seq,
                             const int32_t* ent_pos0, int max_count, float* scratch, float* o, cudaStream_t s);
+// bf16 steps with long entries and head sizes that are multiples of 16 up to 128: the whole of it -- activation or rotation,
+// recurrence and, unless `o` is given, the norm of each head, the gate and the conversion to `out` -- on the tensor cores
+// (seq_linear_mma.cu).
+bool linear_mma_usable(int dtype, const kllm_seq_linear& m, int max_count);
+size_t linear_mma_scratch_bytes(const kllm_seq_linear& m, int T, int n_entries);
+int launch_linear_mma(const kllm_seq_linear& m, const float* proj, int row, float* state, int n_entries, const int32_t* ent_first,
+                      const int32_t* ent_count, const int32_t* ent_seq, const int32_t* ent_pos0, int max_count, int T, float eps,
+                      void* scratch, float* o, void* out, cudaStream_t s);
 // Steps of single tokens whose heads are normed one by one: recurrence, norm, gate and conversion in one kernel (out [T, heads *
 // vdim] in the compute type).
 bool linear_token_usable(const kllm_seq_linear& m);

@@ -16,6 +16,7 @@
 #include <cstdint>
 
 #include "seq_engine.h"
+#include "seq_linear.cuh"
 #include "seq_merge.cuh"
 
 namespace kllm {
@@ -427,15 +428,6 @@ latent_merge_expand_kernel(LatentShape a, int splits, const float* __restrict__ 
 // the activation rotates q and k and scales k: steps of short entries do it on the rows in shared memory (`rot`), steps of long
 // ones in place in the projection, before the chunk kernels read them (linear_rotate_kernel).
 template <bool SILU> __device__ __forceinline__ float lin_act(float v) { return SILU ? siluf(v) : v; }
-struct LinearRot {
-  RopeArgs rope;   // dims == 0: none
-  float k_scale;
-};
-__device__ __forceinline__ void rope_turn(const RopeArgs& r, int i, int pos, float& co, float& si) {
-  const float f = r.freq ? r.freq[i] : powf(r.base, -2.0f * static_cast<float>(i) / static_cast<float>(r.dims));
-  const float a = static_cast<float>(pos) * f;
-  co = cosf(a), si = sinf(a);
-}
 
 // One CTA per token: the angles of its position once, then every q and k head, V pairs at a time.
 template <int V>
@@ -1021,10 +1013,6 @@ int launch_latent_expand(int dtype, const LatentShape& a, const float* ol, const
 size_t linear_attention_scratch_bytes(int heads, int dim, int vdim, int T, int n_entries, int max_count) {
   if (max_count <= kLinParallelFrom) return 0;
   return (static_cast<size_t>(T) / kLinChunk + n_entries + 1) * heads * dim * vdim * sizeof(float);
-}
-
-static LinearRot linear_rot(const kllm_seq_linear& m) {
-  return LinearRot{RopeArgs{m.rope_dims, m.rope_base, m.rope_freq, 1.0f, m.rope_pairing}, m.k_scale == 0.f ? 1.0f : m.k_scale};
 }
 
 int launch_linear_rotate(const kllm_seq_linear& m, float* proj, int row, const int32_t* tok_pos, int T, cudaStream_t s) {

@@ -564,6 +564,37 @@ def test_bfloat16_prompts_on_the_tensor_cores(tmp_path, kind, dim, vdim, reach):
     assert_loosely(np.concatenate(logits[2:]), logits[0][200:])
 
 
+@pytest.mark.parametrize("dim,vdim,rot_dims", [(16, 16, 16), (48, 96, 24), (64, 112, 36), (80, 32, 6), (128, 128, 128)])
+def test_retention_of_long_entries_on_the_tensor_cores(tmp_path, monkeypatch, dim, vdim, rot_dims):
+    """bf16 steps with long entries: entries around multiples of the chunk beside short ones, a second portion that starts from
+    the first one's state, decays from nothing to none -- against the float64 restatement, and closely against the same run on
+    the fp32 kernels (both round the same projections)."""
+    right = RET(heads=5, dim=dim, vdim=vdim, rot_dims=rot_dims, base=2000.0, decay=[0.0, 0.6, 0.97, 0.9995, 1.0])
+    cfg = mo.make_config(width=64, vocab=80, layers=[(PAR(CHUNK(), right, 0.0, 1.0), None)])
+    w = mo.make_weights(cfg, seed=61)
+    d = write_model(tmp_path, cfg, w)
+    sizes = {"a": (63, 70), "b": (64, 65), "c": (129, 2), "d": (5, 192), "e": (200, 1)}
+    reqs = {k: toks(sum(n), cfg["vocab"], 62 + i) for i, (k, n) in enumerate(sizes.items())}
+    steps, at = [], {k: 0 for k in sizes}
+    for part in range(2):
+        steps.append({"entries": [{"id": k, "tokens": reqs[k][at[k]:at[k] + n[part]], "want": list(range(n[part]))}
+                                  for k, n in sizes.items()]})
+        at = {k: n[0] for k, n in sizes.items()}
+    steps.append({"entries": [{"id": k, "tokens": [7], "want": [0]} for k in sizes]})
+    logits, _ = run_trace(d, steps, dtype="bfloat16")
+    monkeypatch.setenv("KLLM_SEQ_LINEAR_MMA", "0")
+    plain, _ = run_trace(d, steps, dtype="bfloat16")
+    for got, want in zip(logits, plain):
+        assert row_errors(got, want).max() < 1e-2
+    for k, n in sizes.items():
+        ref = ref_logits(cfg, w, reqs[k] + [7])
+        rows, i = [], list(sizes).index(k)
+        for part in range(2):
+            b = sum(sizes[x][part] for x in list(sizes)[:i])
+            rows.append(logits[part][b:b + n[part]])
+        assert_loosely(np.concatenate(rows + [logits[2][i:i + 1]]), ref)
+
+
 @pytest.mark.parametrize("dtype", ["float32", "bfloat16"])
 def test_sizes_that_fit_no_vector(tmp_path, dtype):
     """Odd sizes everywhere: no 16-byte vector load, no tensor-core tile and no warp-sized loop fits."""
