@@ -273,8 +273,10 @@ struct RowsOut {
   float eps;
 };
 
-// Grid: (chunk, head, entry).  Warp w: rows 16 (w % 4) .. + 15 of the chunk, half w / 4 of the value columns.
-__global__ void __launch_bounds__(kThreads)
+// Grid: (chunk, head, entry).  Warp w: rows 16 (w % 4) .. + 15 of the chunk, half w / 4 of the value columns.  Beside the queries
+// two tiles of shared memory take turns: keys, the upper and the lower rows of the state, values -- each is on its way while
+// the one before it is multiplied, and two CTAs fit an SM.
+__global__ void __launch_bounds__(kThreads, 2)
 linear_rows_kernel(int heads, int dim, int vdim, const float* __restrict__ decay, Planes in, const int32_t* __restrict__ ent_first,
                    const int32_t* __restrict__ ent_count, const __nv_bfloat16* __restrict__ before_hi,
                    const __nv_bfloat16* __restrict__ before_lo, RowsOut ro) {
@@ -286,24 +288,24 @@ linear_rows_kernel(int heads, int dim, int vdim, const float* __restrict__ decay
   const ChunkAt c = chunk_at(first, count, e, blockIdx.x);
   const int ldq = dim + 8, ldv = vdim + 8, qn = heads * dim;
   const uint32_t q_sm = static_cast<uint32_t>(__cvta_generic_to_shared(raw)), k_sm = q_sm + 2 * kChunk * ldq * 2;
-  const uint32_t v_sm = k_sm + 2 * kChunk * ldq * 2, s_sm = v_sm + 2 * kChunk * ldv * 2;
+  const uint32_t tile = 2 * kChunk * max(ldq, ldv) * 2, v_sm = k_sm + tile;  // v_sm: the second tile
   const int t0 = first + c.base;
+  const int upper = (dim / 16 + 1) / 2 * 16;  // rows of the state in its first part
+  auto load_state = [&](uint32_t dst, int d0, int d1) {
+    const int chunks = vdim / 8;
+    const size_t at0 = (c.slot * heads + h) * dim * vdim;
+    for (int i = threadIdx.x; i < (d1 - d0) * chunks; i += kThreads) {
+      const int d = i / chunks, col = (i % chunks) * 8;
+      const size_t at = at0 + static_cast<size_t>(d0 + d) * vdim + col;
+      cp_async16(dst + (d * ldv + col) * 2, before_hi + at, true);
+      cp_async16(dst + ((kChunk + d) * ldv + col) * 2, before_lo + at, true);
+    }
+    cp_async_commit();
+  };
   load_rows(q_sm, ldq, in, h * dim, dim, t0, c.off);
   load_rows(k_sm, ldq, in, qn + h * dim, dim, t0, c.off);
   cp_async_commit();
-  {
-    const int chunks = vdim / 8;
-    const size_t at0 = (c.slot * heads + h) * dim * vdim;
-    for (int i = threadIdx.x; i < dim * chunks; i += kThreads) {
-      const int d = i / chunks, col = (i % chunks) * 8;
-      const size_t at = at0 + static_cast<size_t>(d) * vdim + col;
-      cp_async16(s_sm + (d * ldv + col) * 2, before_hi + at, true);
-      cp_async16(s_sm + ((dim + d) * ldv + col) * 2, before_lo + at, true);
-    }
-  }
-  cp_async_commit();
-  load_rows(v_sm, ldv, in, 3 * qn + h * vdim, vdim, t0, c.off);
-  cp_async_commit();
+  load_state(v_sm, 0, upper);
   if (threadIdx.x <= kChunk) pw[threadIdx.x] = decay_power(logf(decay[h]), threadIdx.x);
 
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, mi = lane >> 3, gq = lane >> 2, t4 = lane & 3;
@@ -313,7 +315,7 @@ linear_rows_kernel(int heads, int dim, int vdim, const float* __restrict__ decay
   column_half(vdim, hf, p0, np);
   const uint32_t qa = q_sm + ((mt * 16 + (lane & 15)) * ldq + (lane >> 4) * 8) * 2;
 
-  cp_async_wait<2>();
+  cp_async_wait<1>();
   __syncthreads();
   // scores of the rows against the chunk's tokens up to the row tile's last
   float s[kChunk / 8][4];
@@ -347,23 +349,32 @@ linear_rows_kernel(int heads, int dim, int vdim, const float* __restrict__ decay
   for (int p = 0; p < kPairs; ++p)
 #pragma unroll
     for (int z = 0; z < 4; ++z) acc[p][0][z] = acc[p][1][z] = 0.f;
-  cp_async_wait<1>();
-  __syncthreads();
-  for (int ks = 0; ks < dim / 16; ++ks) {
-    uint32_t ah[4], al[4];
-    ldmatrix_x4(qa + ks * 32, ah[0], ah[1], ah[2], ah[3]);
-    ldmatrix_x4(qa + ks * 32 + kChunk * ldq * 2, al[0], al[1], al[2], al[3]);
-    const uint32_t sa = s_sm + ((ks * 16 + (mi & 1) * 8 + (lane & 7)) * ldv + p0 * 16 + (mi >> 1) * 8) * 2;
+  cp_async_wait<0>();
+  __syncthreads();  // the upper rows are in; the keys are no longer read
+  load_state(k_sm, upper, dim);
+  auto times_state = [&](uint32_t part, int ks0, int ks1) {
+    for (int ks = ks0; ks < ks1; ++ks) {
+      uint32_t ah[4], al[4];
+      ldmatrix_x4(qa + ks * 32, ah[0], ah[1], ah[2], ah[3]);
+      ldmatrix_x4(qa + ks * 32 + kChunk * ldq * 2, al[0], al[1], al[2], al[3]);
+      const uint32_t sa = part + (((ks - ks0) * 16 + (mi & 1) * 8 + (lane & 7)) * ldv + p0 * 16 + (mi >> 1) * 8) * 2;
 #pragma unroll
-    for (int p = 0; p < kPairs; ++p) {
-      if (p >= np) break;
-      uint32_t bh[4], bl[4];
-      ldmatrix_x4_trans(sa + p * 32, bh[0], bh[1], bh[2], bh[3]);
-      ldmatrix_x4_trans(sa + p * 32 + dim * ldv * 2, bl[0], bl[1], bl[2], bl[3]);
-      mma_split(acc[p][0], ah, al, bh[0], bh[1], bl[0], bl[1]);
-      mma_split(acc[p][1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+      for (int p = 0; p < kPairs; ++p) {
+        if (p >= np) break;
+        uint32_t bh[4], bl[4];
+        ldmatrix_x4_trans(sa + p * 32, bh[0], bh[1], bh[2], bh[3]);
+        ldmatrix_x4_trans(sa + p * 32 + kChunk * ldv * 2, bl[0], bl[1], bl[2], bl[3]);
+        mma_split(acc[p][0], ah, al, bh[0], bh[1], bl[0], bl[1]);
+        mma_split(acc[p][1], ah, al, bh[2], bh[3], bl[2], bl[3]);
+      }
     }
-  }
+  };
+  times_state(v_sm, 0, upper / 16);
+  cp_async_wait<0>();
+  __syncthreads();  // the lower rows are in; the upper ones are no longer read
+  load_rows(v_sm, ldv, in, 3 * qn + h * vdim, vdim, t0, c.off);
+  cp_async_commit();
+  times_state(k_sm, upper / 16, dim / 16);
   const float fA = pw[max(0, rA - c.off + 1)], fB = pw[max(0, rB - c.off + 1)];
 #pragma unroll
   for (int p = 0; p < kPairs; ++p)
@@ -495,7 +506,7 @@ int launch_linear_mma(const kllm_seq_linear& m, const float* proj, int row, floa
 #undef KLLM_LINEAR_SPLIT
   if (int rc = launched()) return rc;
   const size_t rows_k = 2 * static_cast<size_t>(kChunk) * (m.dim + 8) * 2, rows_v = 2 * static_cast<size_t>(kChunk) * (m.vdim + 8) * 2;
-  const size_t smem_sums = rows_k + rows_v, smem_rows = 2 * rows_k + rows_v + 2 * static_cast<size_t>(m.dim) * (m.vdim + 8) * 2;
+  const size_t smem_sums = rows_k + rows_v, smem_rows = rows_k + 2 * std::max(rows_k, rows_v);
   static size_t configured_sums = 0, configured_rows = 0;
   if (int rc = allow_smem(linear_sums_kernel, smem_sums, &configured_sums)) return rc;
   if (int rc = allow_smem(linear_rows_kernel, smem_rows, &configured_rows)) return rc;
