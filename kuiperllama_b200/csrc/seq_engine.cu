@@ -7,7 +7,7 @@
 // sequence takes pages as it grows (lowest free number first, so freed pages are the next to be used again) and
 // returns them at close.  The table rows of the step's sequences are copied to the device before the kernels run.
 //
-// State.  Beside the pages, every layer run owns per-slot recurrent state in fp32: the last mixer input of a layer with a
+// State.  A slot keeps its sequence's last token (bigram embedding).  Beside the pages, every layer run owns per-slot recurrent state in fp32: the last mixer input of a layer with a
 // token shift, the matrix state of linear attention, of the delta rule and of the duality mixer, the diagonal state of
 // the selective scan, and the last taps - 1 inputs of every short convolution.  A sequence of length 0 reads zeros instead of its slot's
 // memory, so slots are reused without clearing.  A run of attention through a latent keeps one row per token in its pool
@@ -25,7 +25,9 @@
 //                              bf16 prompts that start their sequences, per-head keys and values of the step's own
 //                              latents (two products) and the tensor-core attention
 //                  linear:     gemm (q | k | v | gate rows), the decayed-state recurrence (one kernel for short entries,
-//                              chunk sums / scan / chunk outputs for long ones), output norm and gate
+//                              chunk sums / scan / chunk outputs for long ones, on the tensor cores in bf16), output norm and
+//                              gate -- in the recurrence's own kernel for single tokens and on the tensor cores when the heads
+//                              are normed one by one.  A retention is the form that rotates q and k instead of activating them
 //                  attention behind a filter (values = keys): gemm (q | k rows), qk_conv_prepare (bias, short convolution,
 //                              keys as they are into the value pages, rotation, queries / keys out), attention with window,
 //                              kept first tokens, capped scores and sink
@@ -40,10 +42,11 @@
 //                  an attention may also rotate its queries and keys (frequencies from a table), norm them after the
 //                  rotation, gate every output element, and run as a DIFFERENTIAL attention: two maps per head over the
 //                  same values, joined by diff_merge
-//                  or be normed over the whole query / key projections, and blend their values with those an earlier layer of
+//                  or see only its own chunk of the sequence, be normed over the whole query / key projections, and blend their values with those an earlier layer of
 //                  the step kept; a latent attention may project its queries directly
 //                  a layer may run two mixers of different kinds on the same rows; their outputs join x with a weight each,
-//                  each after an RMS norm of its own when the layer names one
+//                  each after an RMS norm of its own when the layer names one.  Beside an attention the second mixer runs on a
+//                  stream of its own, in buffers of its own; stacked input projections are one product ahead of both
 //     gemm         output projection
 //     resid_norm   x += N_post(y);  h = N_pre_ff(x);  router on h (softmax or sigmoid with groups): same kernel, the row
 //                  is still in shared memory

@@ -1,7 +1,7 @@
-// Kernels of the sequence-batch engine other than the matrix products: embedding rows (with their norm), the fused
+// Kernels of the sequence-batch engine other than the matrix products: embedding rows (with bigram rows and their norm), the fused
 // residual / norm step (layer norm or RMS norm; token shift for single-token steps; router), the token shift over longer
 // entries, query-key preparation with the scatter into the paged cache, causal paged attention (prompt tiles and single
-// decode rows through the same kernel, keys split over CTAs, optional window, sink and fp32 queries), the softmax and the
+// decode rows through the same kernel, keys split over CTAs, optional window or chunks, sink and fp32 queries), the softmax and the
 // grouped sigmoid router with top-k selection, and the routed experts one (token, expert) pair at a time for steps of a
 // few tokens.  The mixers with other kinds of memory (latents, recurrent state) are in seq_mixers.cu.
 //
@@ -458,50 +458,30 @@ __global__ void resid_norm_kernel(ResidNormArgs a) {
   route_token(a.router, buf, buf + W, r, W);
 }
 
-// The same step for rows whose columns fit the CTA's registers (NV 16-byte vectors per thread) and that neither route nor shift
-// nor norm the addends one by one: every load of the row is in flight before the first reduction, the sums go through shared
-// memory once each, and nothing else does.
+// The same step for RMS norms (or none) and rows whose columns fit the CTA's registers (NV 16-byte vectors per thread), which
+// neither route nor shift nor norm the addends one by one: every load of the row is in flight before the first reduction, each
+// sum goes through shared memory once, and nothing else does.
 template <int NV>
-__device__ __forceinline__ void reg_stats(const float4 (&v)[NV], int n4, int W, int kind, float eps, float* red, float& mean,
-                                          float& rstd) {
+__device__ __forceinline__ float reg_rstd(const float4 (&v)[NV], int W, float eps, float* red) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, nw = blockDim.x >> 5;
-  const float inv_w = 1.0f / static_cast<float>(W);
-  mean = 0.f;
-  if (kind == KLLM_SEQ_NORM_LAYER) {
-    float s = 0.f;
+  float q = 0.f;  // vectors past the row are zero
 #pragma unroll
-    for (int k = 0; k < NV; ++k)
-      if (static_cast<int>(threadIdx.x + k * blockDim.x) < n4) s += (v[k].x + v[k].y) + (v[k].z + v[k].w);
-    s = warp_sum(s);
-    if (lane == 0) red[warp] = s;
-    __syncthreads();
-    s = 0.f;
-    for (int i = 0; i < nw; ++i) s += red[i];
-    mean = s * inv_w;
-  }
-  float q = 0.f;
-#pragma unroll
-  for (int k = 0; k < NV; ++k)
-    if (static_cast<int>(threadIdx.x + k * blockDim.x) < n4) {
-      const float a = v[k].x - mean, b = v[k].y - mean, c = v[k].z - mean, d = v[k].w - mean;
-      q = fmaf(a, a, fmaf(b, b, fmaf(c, c, fmaf(d, d, q))));
-    }
+  for (int k = 0; k < NV; ++k) q = fmaf(v[k].x, v[k].x, fmaf(v[k].y, v[k].y, fmaf(v[k].z, v[k].z, fmaf(v[k].w, v[k].w, q))));
   q = warp_sum(q);
-  if (lane == 0) red[32 + warp] = q;
+  if (lane == 0) red[warp] = q;
   __syncthreads();
   q = 0.f;
-  for (int i = 0; i < nw; ++i) q += red[32 + i];
-  rstd = 1.0f / sqrtf(q * inv_w + eps);
+  for (int i = 0; i < nw; ++i) q += red[i];
+  return 1.0f / sqrtf(q * (1.0f / static_cast<float>(W)) + eps);
 }
 __device__ __forceinline__ float4 scaled(float c, const float4& a) { return make_float4(c * a.x, c * a.y, c * a.z, c * a.w); }
 __device__ __forceinline__ void add_scaled(float4& s, float c, const float4& a) {
   s.x = fmaf(c, a.x, s.x), s.y = fmaf(c, a.y, s.y), s.z = fmaf(c, a.z, s.z), s.w = fmaf(c, a.w, s.w);
 }
-__device__ __forceinline__ float4 normed4(const float4& v, float mean, float rstd, const float* w, const float* b, int i) {
+__device__ __forceinline__ float4 normed4(const float4& v, float rstd, const float* w, const float* b, int i) {
   const float4 g = *reinterpret_cast<const float4*>(w + i);
   const float4 o = b ? *reinterpret_cast<const float4*>(b + i) : make_float4(0.f, 0.f, 0.f, 0.f);
-  return make_float4((v.x - mean) * rstd * g.x + o.x, (v.y - mean) * rstd * g.y + o.y, (v.z - mean) * rstd * g.z + o.z,
-                     (v.w - mean) * rstd * g.w + o.w);
+  return make_float4(v.x * rstd * g.x + o.x, v.y * rstd * g.y + o.y, v.z * rstd * g.z + o.z, v.w * rstd * g.w + o.w);
 }
 __device__ __forceinline__ void put4(float* dst, const float4& v) { *reinterpret_cast<float4*>(dst) = v; }
 __device__ __forceinline__ void put4(__nv_bfloat16* dst, const float4& v) {
@@ -511,8 +491,8 @@ __device__ __forceinline__ void put4(__nv_bfloat16* dst, const float4& v) {
 
 template <typename AT, int NV>
 __global__ void __launch_bounds__(512) resid_rows_kernel(ResidNormArgs a) {
-  __shared__ float red_post[64], red_pre[64];
-  const int W = a.width, n4 = W / 4, r = blockIdx.x;
+  __shared__ float red_post[32], red_pre[32];
+  const int W = a.width, r = blockIdx.x;
   const size_t src = static_cast<size_t>(a.rows ? a.rows[r] : r) * W, dst = static_cast<size_t>(r) * W;
   auto at = [](const float* p, size_t i) { return *reinterpret_cast<const float4*>(p + i); };
   float4 x[NV], u[NV];
@@ -528,14 +508,13 @@ __global__ void __launch_bounds__(512) resid_rows_kernel(ResidNormArgs a) {
     if (a.y1 && a.y4) add_scaled(u[k], a.c4, at(a.y4, src + i));
   }
   const bool post = a.y1 != nullptr && a.post.w != nullptr;
-  float mean = 0.f, rstd = 1.0f;
-  if (post) reg_stats<NV>(u, n4, W, a.post.kind, a.eps, red_post, mean, rstd);
+  float rstd = post ? reg_rstd<NV>(u, W, a.eps, red_post) : 1.0f;
   const bool changes = !a.rows && (a.y1 != nullptr || a.add != nullptr || a.add_rows != nullptr);
 #pragma unroll
   for (int k = 0; k < NV; ++k) {
     const int i = (threadIdx.x + k * blockDim.x) * 4;
     if (i >= W) continue;
-    add_scaled(x[k], 1.0f, post ? normed4(u[k], mean, rstd, a.post.w, a.post.b, i) : u[k]);
+    add_scaled(x[k], 1.0f, post ? normed4(u[k], rstd, a.post.w, a.post.b, i) : u[k]);
     if (a.add_rows) add_scaled(x[k], 1.0f, at(a.add_rows, src + i));
     if (a.add) add_scaled(x[k], 1.0f, at(a.add, i));
     if (changes) put4(a.x + dst + i, x[k]);
@@ -544,13 +523,13 @@ __global__ void __launch_bounds__(512) resid_rows_kernel(ResidNormArgs a) {
   const bool plain = a.pre.kind == KLLM_SEQ_NORM_NONE;
   if (!plain) {
     if (a.pre.w == nullptr) return;
-    reg_stats<NV>(x, n4, W, a.pre.kind, a.eps, red_pre, mean, rstd);
+    rstd = reg_rstd<NV>(x, W, a.eps, red_pre);
   }
   AT* out = static_cast<AT*>(a.out) + dst;
 #pragma unroll
   for (int k = 0; k < NV; ++k) {
     const int i = (threadIdx.x + k * blockDim.x) * 4;
-    if (i < W) put4(out + i, plain ? x[k] : normed4(x[k], mean, rstd, a.pre.w, a.pre.b, i));
+    if (i < W) put4(out + i, plain ? x[k] : normed4(x[k], rstd, a.pre.w, a.pre.b, i));
   }
 }
 
@@ -673,7 +652,7 @@ __global__ void qk_prepare_kernel(AttnShape a, RopeArgs rope, const float* __res
     gates[static_cast<size_t>(t) * gn + i] = 1.0f / (1.0f + expf(-row[qn + kn + vn + i]));
 }
 
-// The same with 16-byte accesses for head sizes that are multiples of 4 and halves paired (or no rotation): G lanes share a head,
+// The same with 16-byte accesses for heads that turn (halves paired) or are unit-normed, sizes multiples of 4: G lanes share a head,
 // a lane owns four coordinates of its first half and the four they turn with (or four that do not turn).  The angles of the
 // token's position are taken once, into shared memory; all heads read them from there.
 template <typename AT, int G>
@@ -1508,7 +1487,8 @@ int launch_resid_norm(const ResidNormArgs& a, cudaStream_t s) {
     for (const void* p : ps) bits |= reinterpret_cast<uintptr_t>(p);
     return (bits & 15) == 0;
   };
-  if (!a.router.w_router && !a.shift.mu && !a.out_f32 && !a.n1.w && !a.n3.w && a.width % 4 == 0 && a.width <= 512 * 16 &&
+  const bool layer_norm = (a.y1 && a.post.w && a.post.kind == KLLM_SEQ_NORM_LAYER) || (a.pre.w && a.pre.kind == KLLM_SEQ_NORM_LAYER);
+  if (!layer_norm && !a.router.w_router && !a.shift.mu && !a.out_f32 && !a.n1.w && !a.n3.w && a.width % 4 == 0 && a.width <= 512 * 16 &&
       aligned({a.x, a.y1, a.y2, a.y3, a.y4, a.add, a.add_rows, a.post.w, a.post.b, a.pre.w, a.pre.b, a.out})) {
     // few rows: as many threads as the row has vectors; many: 256 threads and the row's vectors in each thread's registers
     const int n4 = a.width / 4;
@@ -1553,7 +1533,7 @@ int launch_qk_prepare(int dtype, const AttnShape& a, const RopeArgs& rope_, cons
     return done();
   }
   const int half = rope.dims / 2, units = half / 4 + (a.dim - rope.dims) / 4;
-  if (v_share_of(a) == 1 && blend.mode == KLLM_SEQ_VBLEND_NONE && a.dim % 4 == 0 && half % 4 == 0 && a.vdim % 4 == 0 &&
+  if ((rope.dims > 0 || a.qk_norm == KLLM_SEQ_QKNORM_UNIT) && v_share_of(a) == 1 && blend.mode == KLLM_SEQ_VBLEND_NONE && a.dim % 4 == 0 && half % 4 == 0 && a.vdim % 4 == 0 &&
       (rope.dims == 0 || rope.pairing == KLLM_SEQ_ROPE_HALVES) && units <= 32 && stride % 4 == 0 &&
       (reinterpret_cast<uintptr_t>(qkvg) & 15) == 0) {
     const int threads = T <= 64 ? 512 : 256;

@@ -6,7 +6,8 @@
 //                                dimensions), latent_expand (W_uv on the weighted sum of latents).  Between absorb and expand
 //                                the paged attention kernel of seq_kernels.cu runs with one key/value "head" of
 //                                kv_rank + rot_dim key and kv_rank value dimensions that every query head shares.
-//   linear attention             the decayed-state recurrence, chunk by chunk, and its output norm with the sigmoid gate
+//   linear attention             the decayed-state recurrence, chunk by chunk (activated, or rotated as a retention), and its output
+//                                norm with the gate; single tokens in one kernel.  bf16 steps with long entries: seq_linear_mma.cu
 //   activations                  xIELU and squared ReLU between the two products of a dense feed-forward
 //
 // Positions and angles, norms, gates, decays and the recurrent state are fp32 in both compute types.
