@@ -270,6 +270,7 @@ struct RowsOut {
   __nv_bfloat16* out;     // [T][heads * vdim]: o / rms(o of the head) * act(gate)
   const float* gate;      // gate rows of the projection
   int gate_stride, gate_act;
+  int gate_vec;           // != 0: gate rows can be read 16 bytes at a time
   float eps;
 };
 
@@ -381,7 +382,17 @@ linear_rows_kernel(int heads, int dim, int vdim, const float* __restrict__ decay
 #pragma unroll
     for (int b = 0; b < 2; ++b) acc[p][b][0] *= fA, acc[p][b][1] *= fA, acc[p][b][2] *= fB, acc[p][b][3] *= fB;
   cp_async_wait<0>();
-  __syncthreads();
+  __syncthreads();  // the values are in; the first tile is free: the head's gate rows come in under the last product
+  const bool staged = ro.o == nullptr && ro.gate_vec;
+  if (staged) {
+    const int quads = vdim / 4;
+    for (int i = threadIdx.x; i < kChunk * quads; i += kThreads) {
+      const int r = i / quads, col = (i % quads) * 4;
+      const bool in = r >= c.off;
+      cp_async16(k_sm + (r * ldv + col) * 4, in ? ro.gate + static_cast<size_t>(t0 + r - c.off) * ro.gate_stride + h * vdim + col : ro.gate, in);
+    }
+    cp_async_commit();
+  }
 #pragma unroll
   for (int kk = 0; kk < kChunk / 16; ++kk) {
     if (kk > mt) break;
@@ -427,7 +438,9 @@ linear_rows_kernel(int heads, int dim, int vdim, const float* __restrict__ decay
     }
   qA = quad_sum(qA), qB = quad_sum(qB);
   if (t4 == 0) square[hf][rA] = qA, square[hf][rB] = qB;
+  cp_async_wait<0>();
   __syncthreads();
+  const float* gates = reinterpret_cast<const float*>(raw + (k_sm - q_sm));  // [kChunk][ldv] when they are staged
   const float nA = 1.0f / sqrtf((square[0][rA] + square[1][rA]) / static_cast<float>(vdim) + ro.eps);
   const float nB = 1.0f / sqrtf((square[0][rB] + square[1][rB]) / static_cast<float>(vdim) + ro.eps);
   auto gated = [&](float o, float z) { return o * (ro.gate_act == KLLM_SEQ_GATEACT_SILU ? silu(z) : 1.0f / (1.0f + expf(-z))); };
@@ -442,9 +455,15 @@ linear_rows_kernel(int heads, int dim, int vdim, const float* __restrict__ decay
         if (!(z == 0 ? inA : inB)) continue;
         const size_t t = z == 0 ? tA : tB;
         const float n = z == 0 ? nA : nB;
-        const float* g = ro.gate + t * ro.gate_stride + col;
+        float2 g;
+        if (staged) {
+          g = *reinterpret_cast<const float2*>(gates + (z == 0 ? rA : rB) * ldv + col - h * vdim);
+        } else {
+          const float* src = ro.gate + t * ro.gate_stride + col;
+          g = make_float2(src[0], src[1]);
+        }
         *reinterpret_cast<__nv_bfloat162*>(ro.out + t * vn + col) =
-            __floats2bfloat162_rn(gated(acc[p][b][2 * z] * n, g[0]), gated(acc[p][b][2 * z + 1] * n, g[1]));
+            __floats2bfloat162_rn(gated(acc[p][b][2 * z] * n, g.x), gated(acc[p][b][2 * z + 1] * n, g.y));
       }
     }
   }
@@ -517,7 +536,9 @@ int launch_linear_mma(const kllm_seq_linear& m, const float* proj, int row, floa
   linear_carry_kernel<<<cgrid, 128, 0, s>>>(m.heads, size, m.decay, state, ent_first, ent_count, ent_seq, ent_pos0, sums, before,
                                             before + se);
   if (int rc = launched()) return rc;
-  const RowsOut ro{o, static_cast<__nv_bfloat16*>(out), proj + 2 * m.heads * m.dim + m.heads * m.vdim, row, m.gate_act, eps};
+  const float* gate = proj + 2 * m.heads * m.dim + m.heads * m.vdim;
+  const RowsOut ro{o, static_cast<__nv_bfloat16*>(out), gate, row, m.gate_act,
+                   row % 4 == 0 && (reinterpret_cast<uintptr_t>(gate) & 15) == 0, eps};
   linear_rows_kernel<<<grid, kThreads, smem_rows, s>>>(m.heads, m.dim, m.vdim, m.decay, planes, ent_first, ent_count, before, before + se,
                                                        ro);
   return launched();
